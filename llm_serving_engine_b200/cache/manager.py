@@ -11,7 +11,8 @@ Beyond it:
 * Layers are put into *groups* by what their mixer needs (number of key/value
   heads, head size, window).  Each group has its own pool of pages, its own free
   list and its own block table per request.  A group with a window gives a page
-  back as soon as every key in it lies before the window of the next token.
+  back as soon as every key in it lies before the window of the next token (pages with one
+  of the first keys that a window keeps stay).
 * Mixers that keep a state of fixed size per request get *state slots*: one
   tensor [slots, *shape] per layer; a request takes a slot when it is created
   (the slot is zeroed) and gives it back when it ends.  A model without such a
@@ -20,7 +21,8 @@ Beyond it:
   both are made) gets pages of such rows: [layer in group, 1, page, offset in page, width].
 * A mixer that keeps several things (pages and a state, or states of different shapes) names them
   in a tuple; each member is kept as if it were a layer's only need (its key is (layer, index)),
-  and the layer's view holds the members' views in ``parts``.
+  and the layer's view holds the members' views in ``parts``.  What the layer's arrangement keeps
+  itself stands behind the mixer's members.
 
 Storage layout of a group: [layer in group, 2 (keys, values), page, kv head,
 offset in page, head size]: the tokens of one page and one head are contiguous.
@@ -283,9 +285,10 @@ class CacheManager:
             window = group.need.window
             if window <= 0:
                 continue
-            first_needed = request.length - window + 1   # smallest key the next token reads
+            first_needed = request.length - window + 1   # smallest key the next token reads (kept first keys aside)
             table = request.tables[index]
-            page = request.released[index]
+            kept = -(-getattr(group.need, "keep_first", 0) // self.page_size)     # pages with a key that is read for ever
+            page = max(request.released[index], kept)
             while page < len(table) and (page + 1) * self.page_size <= first_needed:
                 group.pool.free(table[page], request_id)
                 table[page] = -1

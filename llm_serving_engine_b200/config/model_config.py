@@ -68,11 +68,15 @@ class ModelSpec:
     embedding_scale: float = 1.0     # the embedding rows are multiplied by it
     position_table_name: str | None = None   # a learned vector per position [max_position_embeddings, hidden], added to the embedding
     logit_softcap: float = 0.0       # > 0: logits <- cap * tanh(logits / cap)
+    embedding_again: tuple[int, ...] = ()    # positions in ``order`` before which the embedding's output is added once more
+    shared_tensors: dict[str, tuple[int, ...]] = field(default_factory=dict)   # matrices that several layers' parts read, by full name
 
     def __post_init__(self) -> None:
         for index in self.order:
             if not 0 <= index < len(self.layers):
                 raise ConfigError(f"order names layer {index}, model has {len(self.layers)}")
+        if any(not 0 <= position < len(self.order) for position in self.embedding_again):
+            raise ConfigError("embedding_again names a position outside the order")
         for number, layer in enumerate(self.layers):
             if layer.cache_from is not None and not 0 <= layer.cache_from < len(self.layers):
                 raise ConfigError(f"layer {number} reads the cache of unknown layer {layer.cache_from}")

@@ -12,6 +12,8 @@
 //
 //   * window: row i reads keys j with i - j < window only (window <= 0: every key up to i); pages before the window
 //     are never touched (their table entries may have been given back);
+//   * kept first keys (`keep_first` > 0, with a window): keys j < keep_first are read by every row that lies behind them
+//     as well; chunks and tiles that hold neither kept keys nor keys of the window are stepped over;
 //   * cap: s <- cap * tanh(s / cap) before anything else is done with the score (cap <= 0: none);
 //   * weights without a softmax (`head_bias` given): a key's weight is sigmoid(s_ij + head_bias_h), not normalised
 //     over the keys; the output is the plain weighted sum of the values.  The chunks' sums are then added in order
@@ -43,6 +45,11 @@ __device__ __forceinline__ void merge_parts(float& M, float& L, float m, float l
   M = m_new;
 }
 
+// Whether a row that reads keys first_key .. pos and, of those before, the first keep_first has a key in [lo, hi).
+__device__ __forceinline__ bool scored_range_seen(int lo, int hi, int first_key, int keep_first) {
+  return hi > first_key || lo < keep_first;
+}
+
 // The sink joins a finished (M, L): the factor on the outputs is returned.
 __device__ __forceinline__ float add_sink(float M, float& L, float sink) {
   const float m_new = fmaxf(M, sink);
@@ -61,7 +68,7 @@ attention_scored_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
                         const int* __restrict__ segment_of_token, const int* __restrict__ positions,
                         const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink,
                         int n_q, int n_kv, int dk, int dv, int n_values, int page_size, float scale, int num_pages,
-                        int num_segments, float* __restrict__ partials, int max_chunks, int window, float cap,
+                        int num_segments, float* __restrict__ partials, int max_chunks, int window, int keep_first, float cap,
                         const float* __restrict__ head_bias) {
   extern __shared__ float smem[];
   pdl_launch_dependents();
@@ -82,9 +89,9 @@ attention_scored_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
   const int pos = positions[t];
   const int ctx = pos + 1;
   const int first_key = window > 0 ? max(0, ctx - window) : 0;   // the first key the row reads
-  int chunk_lo = first_key / CHUNK, chunk_hi = pos / CHUNK;
+  int chunk_lo = keep_first > 0 ? 0 : first_key / CHUNK, chunk_hi = pos / CHUNK;
   if (SPLIT) {
-    if (zz > chunk_hi || zz < chunk_lo) return;
+    if (zz > chunk_hi || !scored_range_seen(zz * CHUNK, (zz + 1) * CHUNK, first_key, keep_first)) return;
     chunk_lo = chunk_hi = zz;
   }
   const int* bt = block_tables + (size_t)seg * bt_stride;
@@ -125,6 +132,7 @@ attention_scored_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
   const float inv_cap = cap > 0.f ? 1.0f / cap : 0.f;
 
   for (int chunk = chunk_lo; chunk <= chunk_hi; ++chunk) {
+    if (!scored_range_seen(chunk * CHUNK, (chunk + 1) * CHUNK, first_key, keep_first)) continue;
     float acc[GC][DPT];
 #pragma unroll
     for (int g = 0; g < GC; ++g)
@@ -135,12 +143,13 @@ attention_scored_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
     for (int i = 0; i < GC / 4; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
 
     const int tile_end = min(ctx, (chunk + 1) * CHUNK);
-    for (int base = max(chunk * CHUNK, first_key / KT * KT); base < tile_end; base += KT) {
+    for (int base = keep_first > 0 ? chunk * CHUNK : max(chunk * CHUNK, first_key / KT * KT); base < tile_end; base += KT) {
+      if (!scored_range_seen(base, base + KT, first_key, keep_first)) continue;
       __syncthreads();  // previous tile fully consumed (also orders the q_s fill)
       if (tid < KT) {
         const int j = base + tid;
         int slot = -1;
-        if (j < ctx && j >= first_key) {
+        if (j < ctx && (j >= first_key || j < keep_first)) {
           const int page = LSE_CHECKED(bt[j / page_size], 0, num_pages, 0, LSE_CHECK_TABLE_ENTRY);
           slot = page * page_size + (j % page_size);
         }
@@ -264,7 +273,7 @@ __global__ void __launch_bounds__(MAX_D)
 attention_scored_merge_kernel(const float* __restrict__ partials, TO* __restrict__ out,
                               const int* __restrict__ segment_of_token, const int* __restrict__ positions,
                               const float* __restrict__ sink, int n_values, int dv, int max_chunks, int num_segments,
-                              int window, int unnormalised) {
+                              int window, int keep_first, int unnormalised) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, item = blockIdx.y, d = threadIdx.x;
@@ -273,8 +282,9 @@ attention_scored_merge_kernel(const float* __restrict__ partials, TO* __restrict
   const int pos = positions[t];
   const float* src = partials + ((size_t)t * gridDim.y + item) * max_chunks * (dv + 2);
   float total = 0.f, M = -INFINITY, L = 0.f;
-  const int first_chunk = window > 0 ? max(0, pos + 1 - window) / CHUNK : 0;
-  for (int chunk = first_chunk; chunk <= pos / CHUNK; ++chunk) {
+  const int first_key = window > 0 ? max(0, pos + 1 - window) : 0;
+  for (int chunk = keep_first > 0 ? 0 : first_key / CHUNK; chunk <= pos / CHUNK; ++chunk) {
+    if (!scored_range_seen(chunk * CHUNK, (chunk + 1) * CHUNK, first_key, keep_first)) continue;
     const float* part = src + (size_t)chunk * (dv + 2);
     float wa, wb;
     merge_parts(M, L, part[dv], part[dv + 1], wa, wb);
@@ -411,8 +421,8 @@ template <typename T, typename TO>
 int launch_scored(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_tables,
                   int bt_stride, const int* segment_of_token, const int* positions, const float* r1, const float* r2,
                   const float* sink, int tokens, int n_q, int n_kv, int dk, int dv, int n_values, int page_size,
-                  float scale, int num_pages, int num_segments, float* partials, int max_chunks, int window, float cap,
-                  const float* head_bias, cudaStream_t stream) {
+                  float scale, int num_pages, int num_segments, float* partials, int max_chunks, int window, int keep_first,
+                  float cap, const float* head_bias, cudaStream_t stream) {
   const int group = n_q / n_kv;
   const int gchunks = (group + GC - 1) / GC;
   const bool split = partials != nullptr;
@@ -431,14 +441,14 @@ int launch_scored(const void* q, const void* k_cache, const void* v_cache, void*
   if (split) {
     lse_launch(attention_scored_kernel<T, TO, true>, grid, THREADS, smem, stream, (const T*)q, (const T*)k_cache,
                (const T*)v_cache, (TO*)out, block_tables, bt_stride, segment_of_token, positions, r1, r2, sink, n_q, n_kv,
-               dk, dv, n_values, page_size, scale, num_pages, num_segments, partials, max_chunks, window, cap, head_bias);
+               dk, dv, n_values, page_size, scale, num_pages, num_segments, partials, max_chunks, window, keep_first, cap, head_bias);
     lse_launch(attention_scored_merge_kernel<TO>, dim3(tokens, n_q * n_values), ((dv + 31) / 32) * 32, 0, stream,
                (const float*)partials, (TO*)out, segment_of_token, positions, sink, n_values, dv, max_chunks,
-               num_segments, window, (int)(head_bias != nullptr));
+               num_segments, window, keep_first, (int)(head_bias != nullptr));
   } else {
     lse_launch(attention_scored_kernel<T, TO, false>, grid, THREADS, smem, stream, (const T*)q, (const T*)k_cache,
                (const T*)v_cache, (TO*)out, block_tables, bt_stride, segment_of_token, positions, r1, r2, sink, n_q, n_kv,
-               dk, dv, n_values, page_size, scale, num_pages, num_segments, (float*)nullptr, 0, window, cap, head_bias);
+               dk, dv, n_values, page_size, scale, num_pages, num_segments, (float*)nullptr, 0, window, keep_first, cap, head_bias);
   }
   return (int)cudaGetLastError();
 }
@@ -450,17 +460,18 @@ extern "C" int lse_attention_scored_chunk(void) { return CHUNK; }
 // cross != 0: n_values = n_kv (see the top of the file), else 1.  r1/r2 (together) and sink: float32 [n_q] or null.
 // partials != null: every chunk of a row gets a block of its own; it holds tokens * n_q * n_values * max_chunks *
 // (dv + 2) floats, and max_chunks chunks cover the longest context that the block tables can describe.
-// window > 0: a row reads its last `window` keys only; cap > 0: scores capped by cap * tanh(s / cap); head_bias (float32
+// window > 0: a row reads its last `window` keys only, and with keep_first > 0 the request's first keep_first; cap > 0: scores capped by cap * tanh(s / cap); head_bias (float32
 // [n_q] or null): weights sigmoid(s + head_bias_h) without a softmax (no sink then).
 extern "C" int lse_attention_scored_windowed(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype,
                                              int out_f32, const int* block_tables, int bt_stride,
                                              const int* segment_of_token, const int* positions, const float* r1,
                                              const float* r2, const float* sink, int tokens, int n_q, int n_kv, int dk,
                                              int dv, int cross, int page_size, float scale, int num_pages,
-                                             int num_segments, float* partials, int max_chunks, int window, float cap,
-                                             const float* head_bias, cudaStream_t stream) {
+                                             int num_segments, float* partials, int max_chunks, int window,
+                                             int keep_first, float cap, const float* head_bias, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (head_bias && sink) return LSE_ERR_BAD_ARGUMENT;
+  if ((head_bias && sink) || keep_first < 0) return LSE_ERR_BAD_ARGUMENT;
+  if (window <= 0) keep_first = 0;     // every key is read anyway
   if (dk <= 0 || dk > MAX_D || dv <= 0 || dv > MAX_D || n_kv <= 0 || n_q % n_kv || page_size <= 0 || (!r1) != (!r2))
     return LSE_ERR_BAD_ARGUMENT;
   const int n_values = cross ? n_kv : 1;
@@ -470,7 +481,7 @@ extern "C" int lse_attention_scored_windowed(const void* q, const void* k_cache,
   if ((long long)(partials ? max_chunks : 1) * n_values * gchunks > 65535 || n_kv > 65535 || n_q * n_values > 65535)
     return LSE_ERR_TOO_LARGE;
 #define LSE_SCORED_ARGS q, k_cache, v_cache, out, block_tables, bt_stride, segment_of_token, positions, r1, r2, sink, tokens, \
-  n_q, n_kv, dk, dv, n_values, page_size, scale, num_pages, num_segments, partials, max_chunks, window, cap, head_bias, stream
+  n_q, n_kv, dk, dv, n_values, page_size, scale, num_pages, num_segments, partials, max_chunks, window, keep_first, cap, head_bias, stream
   if (dtype == LSE_DTYPE_F32) return launch_scored<float, float>(LSE_SCORED_ARGS);
   if (dtype == LSE_DTYPE_BF16 && out_f32) return launch_scored<__nv_bfloat16, float>(LSE_SCORED_ARGS);
   if (dtype == LSE_DTYPE_BF16) return launch_scored<__nv_bfloat16, __nv_bfloat16>(LSE_SCORED_ARGS);
@@ -486,26 +497,28 @@ extern "C" int lse_attention_scored(const void* q, const void* k_cache, const vo
                                     cudaStream_t stream) {
   return lse_attention_scored_windowed(q, k_cache, v_cache, out, dtype, out_f32, block_tables, bt_stride, segment_of_token,
                                        positions, r1, r2, sink, tokens, n_q, n_kv, dk, dv, cross, page_size, scale,
-                                       num_pages, num_segments, partials, max_chunks, 0, 0.f, nullptr, stream);
+                                       num_pages, num_segments, partials, max_chunks, 0, 0, 0.f, nullptr, stream);
 }
 
 // The second half of a launch with partials, for kernels of other files that leave partials in the same layout
 // ([t][head][value slot][chunk][dv + 2]: sums, maximum, total): out [T, n_q, n_values, dv] in bfloat16 or float32.
-// window, unnormalised: as the launch that left the partials had them (chunks before the window hold nothing).
+// window, keep_first, unnormalised: as the launch that left the partials had them (chunks before the window hold nothing).
 extern "C" int lse_attention_scored_merge_windowed(const float* partials, void* out, int out_dtype,
                                                    const int* segment_of_token, const int* positions, const float* sink,
                                                    int tokens, int n_q, int n_values, int dv, int max_chunks,
-                                                   int num_segments, int window, int unnormalised, cudaStream_t stream) {
+                                                   int num_segments, int window, int keep_first, int unnormalised,
+                                                   cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (dv <= 0 || dv > MAX_D || n_q * n_values > 65535 || max_chunks <= 0) return LSE_ERR_BAD_ARGUMENT;
+  if (dv <= 0 || dv > MAX_D || n_q * n_values > 65535 || max_chunks <= 0 || keep_first < 0) return LSE_ERR_BAD_ARGUMENT;
+  if (window <= 0) keep_first = 0;
   const dim3 grid(tokens, n_q * n_values);
   const int threads = ((dv + 31) / 32) * 32;
   if (out_dtype == LSE_DTYPE_F32)
     lse_launch(attention_scored_merge_kernel<float>, grid, threads, 0, stream, partials, (float*)out, segment_of_token,
-               positions, sink, n_values, dv, max_chunks, num_segments, window, unnormalised);
+               positions, sink, n_values, dv, max_chunks, num_segments, window, keep_first, unnormalised);
   else if (out_dtype == LSE_DTYPE_BF16)
     lse_launch(attention_scored_merge_kernel<__nv_bfloat16>, grid, threads, 0, stream, partials, (__nv_bfloat16*)out,
-               segment_of_token, positions, sink, n_values, dv, max_chunks, num_segments, window, unnormalised);
+               segment_of_token, positions, sink, n_values, dv, max_chunks, num_segments, window, keep_first, unnormalised);
   else
     return LSE_ERR_BAD_ARGUMENT;
   LSE_LAUNCH_CHECK();
@@ -515,7 +528,7 @@ extern "C" int lse_attention_scored_merge(const float* partials, void* out, int 
                                           const int* positions, const float* sink, int tokens, int n_q, int n_values,
                                           int dv, int max_chunks, int num_segments, cudaStream_t stream) {
   return lse_attention_scored_merge_windowed(partials, out, out_dtype, segment_of_token, positions, sink, tokens, n_q,
-                                             n_values, dv, max_chunks, num_segments, 0, 0, stream);
+                                             n_values, dv, max_chunks, num_segments, 0, 0, 0, stream);
 }
 
 // wide [T, n_q, n_values, dv] (n_values = n_kv when cross, else 1) in float32, or in bfloat16 (wide_bf16; only shapes

@@ -11,7 +11,9 @@
 // a small table (a logarithm per table entry instead of one per score).
 //
 // window > 0: a row reads its last `window` keys only; key tiles before the window of the tile's first row are not
-// walked, and keys before it are not fetched (their pages may have been given back).  cap > 0: scores are capped by
+// walked, and keys before it are not fetched (their pages may have been given back).  keep_first > 0 (with a window): the
+// request's first keys are read by every row behind them as well; the walk then takes the tiles that hold them first and
+// goes on with the tiles of the window.  cap > 0: scores are capped by
 // cap * tanh(s / cap).  head_bias: no softmax, a key's weight is sigmoid(s + head_bias_h) and the sums are not divided.
 //
 // With `partials` the keys of a tile of rows are cut into chunks of 256 (counted from key 0) with a block each, which
@@ -42,7 +44,7 @@ attention_scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
                             const int* __restrict__ segment_first_pos, int num_segments, const float* __restrict__ r1,
                             const float* __restrict__ r2, const float* __restrict__ sink, int n_q, int n_kv,
                             int n_values, int page_size, float scale_log2e, int rows_per_tile, int num_pages,
-                            int max_chunks, int window, float cap, const float* __restrict__ head_bias) {
+                            int max_chunks, int window, int keep_first, float cap, const float* __restrict__ head_bias) {
   constexpr int CHK = DK / 8, CHV = DV / 8;
   constexpr int K_BYTES = tile_bytes<DK>(BN), V_BYTES = tile_bytes<DV>(BN);
   extern __shared__ __align__(128) unsigned char smem[];
@@ -71,18 +73,26 @@ attention_scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   const int last_pos = pos0 + nrows - 1;
   const int first_key = window > 0 ? max(0, pos0 + 1 - window) : 0;   // the first key that any row of the tile reads
   int tile_lo = first_key / BN, tile_hi = (last_pos + BN) / BN;         // key tiles [tile_lo, tile_hi)
+  // tiles of kept first keys that lie before tile_lo: [kept_lo, kept_lo + kept_tiles), walked before the others
+  int kept_lo = 0, kept_tiles = min(tile_lo, (keep_first + BN - 1) / BN);
   if (partials) {
-    if (chunk * CHUNK > last_pos || (chunk + 1) * CHUNK <= first_key) return;
-    tile_lo = max(tile_lo, chunk * (CHUNK / BN));
-    tile_hi = min(tile_hi, (chunk + 1) * (CHUNK / BN));
+    if (chunk * CHUNK > last_pos || ((chunk + 1) * CHUNK <= first_key && chunk * CHUNK >= keep_first)) return;
+    const int chunk_lo = chunk * (CHUNK / BN), chunk_hi = (chunk + 1) * (CHUNK / BN);
+    const int kept_hi = min(kept_tiles, chunk_hi);
+    kept_lo = chunk_lo;
+    kept_tiles = max(0, kept_hi - kept_lo);
+    tile_lo = max(tile_lo, chunk_lo);
+    tile_hi = max(tile_lo, min(tile_hi, chunk_hi));
   }
+  const int walk = kept_tiles + tile_hi - tile_lo;
+  if (walk <= 0) return;
   const int* bt = block_tables + (size_t)seg * bt_stride;
   const PageMath pm(page_size);
   const int n_pages = pm.page(last_pos) + 1;
   const bool staged = n_pages <= TABLE_STAGE;
   if (staged)
     for (int i = tid; i < n_pages; i += 128)
-      bt_s[i] = i < pm.page(first_key) ? 0 : LSE_CHECKED(bt[i], 0, num_pages, 0, LSE_CHECK_TABLE_ENTRY);
+      bt_s[i] = i < pm.page(first_key) && i * page_size >= keep_first ? 0 : LSE_CHECKED(bt[i], 0, num_pages, 0, LSE_CHECK_TABLE_ENTRY);
   pdl_wait();
 
   for (int e = tid; e < BM * CHK; e += 128) {
@@ -101,8 +111,9 @@ attention_scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     const uint32_t k_dst = kv_u32 + (uint32_t)stage * (K_BYTES + V_BYTES), v_dst = k_dst + K_BYTES;
     if (page_pieces) {
       const int j0 = kt * BN + warp * 16;
-      const int limit = (j0 <= last_pos && j0 + 15 >= first_key) ? last_pos + 1 - j0 : 0;   // keys of the piece that exist
-      const int skip = first_key - j0;       // keys of the piece before the window: not fetched
+      const int limit = (j0 <= last_pos && (j0 + 15 >= first_key || j0 < keep_first)) ? last_pos + 1 - j0 : 0;   // keys of the piece that exist
+      const int skip = first_key - j0;       // keys of the piece before the window: not fetched,
+      const int kept = keep_first - j0;      // unless they are kept first keys
       size_t k_base = 0, v_base = 0;
       if (limit > 0) {
         const size_t page = (size_t)bt_s[pm.page(j0)];
@@ -112,13 +123,13 @@ attention_scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
 #pragma unroll
       for (int i = 0; i < CHK / 2; ++i) {
         const int n = lane + 32 * i, row = n / CHK, c = n % CHK;
-        const bool valid = row < limit && row >= skip;
+        const bool valid = row < limit && (row >= skip || row < kept);
         cp_async16(k_dst + padded_off<DK>(warp * 16 + row, c), kc + k_base + (valid ? row * DK + c * 8 : 0), valid);
       }
 #pragma unroll
       for (int i = 0; i < CHV / 2; ++i) {
         const int n = lane + 32 * i, row = n / CHV, c = n % CHV;
-        const bool valid = row < limit && row >= skip;
+        const bool valid = row < limit && (row >= skip || row < kept);
         cp_async16(v_dst + padded_off<DV>(warp * 16 + row, c), vc + v_base + (valid ? row * DV + c * 8 : 0), valid);
       }
       return;
@@ -128,7 +139,7 @@ attention_scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
       const int local = is_key ? idx : idx - BN * CHK;
       const int key = is_key ? local / CHK : local / CHV, c = is_key ? local % CHK : local % CHV;
       const int j = kt * BN + key;
-      const bool valid = j <= last_pos && j >= first_key;
+      const bool valid = j <= last_pos && (j >= first_key || j < keep_first);
       size_t slot = 0;
       if (valid) {
         const int logical = pm.page(j);
@@ -140,7 +151,8 @@ attention_scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     }
   };
   __syncthreads();   // q_s and bt_s are filled
-  load_tile(tile_lo, 0);
+  auto tile_at = [&](int step) { return step < kept_tiles ? kept_lo + step : tile_lo + step - kept_tiles; };
+  load_tile(tile_at(0), 0);
   cp_async_commit();
 
   uint32_t qf[DK / 16][4];
@@ -168,9 +180,9 @@ attention_scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   for (int i = 0; i < DV / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
 
-  for (int kt = tile_lo; kt < tile_hi; ++kt) {
-    const int stage = (kt - tile_lo) & 1;
-    if (kt + 1 < tile_hi) load_tile(kt + 1, stage ^ 1);
+  for (int step = 0; step < walk; ++step) {
+    const int kt = tile_at(step), stage = step & 1;
+    if (step + 1 < walk) load_tile(tile_at(step + 1), stage ^ 1);
     cp_async_commit();
     if (penalised) {
       const int nearest = pos0 - (kt * BN + BN - 1);   // distance from the tile's first row to its last key
@@ -218,7 +230,7 @@ attention_scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
         }
         if (penalised) v -= ((e >> 1) ? pen_b : pen_a)[-key];
         if (diagonal && j > pos) v = -INFINITY;
-        if (windowed && j <= pos - window) v = -INFINITY;
+        if (windowed && j <= pos - window && j >= keep_first) v = -INFINITY;
         s[nb][e] = v;
       }
       mx0 = fmaxf(mx0, fmaxf(s[nb][0], s[nb][1]));
@@ -281,8 +293,8 @@ attention_scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
 
   if (partials) {   // unnormalised sums, the maximum in natural units, the total: for the merge kernel
     constexpr float LN2 = 0.6931471805599453f;
-    const bool write_a = rla < nrows && chunk * CHUNK <= pos_a && (window <= 0 || (chunk + 1) * CHUNK > pos_a + 1 - window);
-    const bool write_b = rlb < nrows && chunk * CHUNK <= pos_b && (window <= 0 || (chunk + 1) * CHUNK > pos_b + 1 - window);
+    const bool write_a = rla < nrows && chunk * CHUNK <= pos_a && (window <= 0 || (chunk + 1) * CHUNK > pos_a + 1 - window || chunk * CHUNK < keep_first);
+    const bool write_b = rlb < nrows && chunk * CHUNK <= pos_b && (window <= 0 || (chunk + 1) * CHUNK > pos_b + 1 - window || chunk * CHUNK < keep_first);
     float* dst_a = partials + ((((size_t)(row_base + rla) * n_q + head_a) * n_values + value_slot) * max_chunks + chunk) * (DV + 2);
     float* dst_b = partials + ((((size_t)(row_base + rlb) * n_q + head_b) * n_values + value_slot) * max_chunks + chunk) * (DV + 2);
 #pragma unroll
@@ -326,8 +338,8 @@ template <int D>
 int launch_scored_mma(const void* q, const void* kc, const void* vc, void* out, int out_is_f32, float* partials,
                       const int* block_tables, int bt_stride, const int* segment_start, const int* segment_first_pos,
                       int num_segments, const float* r1, const float* r2, const float* sink, int tokens, int n_q, int n_kv,
-                      int n_values, int page_size, float scale, int num_pages, int max_chunks, int window, float cap,
-                      const float* head_bias, cudaStream_t stream) {
+                      int n_values, int page_size, float scale, int num_pages, int max_chunks, int window, int keep_first,
+                      float cap, const float* head_bias, cudaStream_t stream) {
   const int group = n_q / n_kv;
   const int rows_per_tile = BM / group;
   const size_t tiles_bytes = (size_t)tile_bytes<D>(BM) + 2 * (size_t)(tile_bytes<D>(BN) + tile_bytes<D>(BN));
@@ -347,7 +359,7 @@ int launch_scored_mma(const void* q, const void* kc, const void* vc, void* out, 
              (const __nv_bfloat16*)vc, out_is_f32 ? (__nv_bfloat16*)nullptr : (__nv_bfloat16*)out,
              out_is_f32 ? (float*)out : (float*)nullptr, partials, block_tables, bt_stride, segment_start, segment_first_pos,
              num_segments, r1, r2, sink, n_q, n_kv, n_values, page_size, scale * LOG2E, rows_per_tile, num_pages, max_chunks,
-             window, cap, head_bias);
+             window, keep_first, cap, head_bias);
   return (int)cudaGetLastError();
 }
 }  // namespace
@@ -367,17 +379,18 @@ extern "C" int lse_attention_scored_mma_windowed(const void* q, const void* k_ca
                                                  const int* segment_start, const int* segment_first_pos, int num_segments,
                                                  const float* r1, const float* r2, const float* sink, int tokens, int n_q,
                                                  int n_kv, int dk, int dv, int cross, int page_size, float scale,
-                                                 int num_pages, float* partials, int max_chunks, int window, float cap,
+                                                 int num_pages, float* partials, int max_chunks, int window, int keep_first, float cap,
                                                  const float* head_bias, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (head_bias && sink) return LSE_ERR_BAD_ARGUMENT;
+  if ((head_bias && sink) || keep_first < 0) return LSE_ERR_BAD_ARGUMENT;
+  if (window <= 0) keep_first = 0;
   if (!lse_attention_scored_mma_supported(dk, dv, n_q, n_kv) || page_size <= 0 || (!r1) != (!r2)) return LSE_ERR_BAD_ARGUMENT;
   if (partials && (max_chunks <= 0 || (long long)max_chunks * CHUNK < (long long)bt_stride * page_size))
     return LSE_ERR_BAD_ARGUMENT;
   const int n_values = cross ? n_kv : 1;
 #define LSE_SCORED_MMA_ARGS q, k_cache, v_cache, out, out_f32, partials, block_tables, bt_stride, segment_start, \
   segment_first_pos, num_segments, r1, r2, sink, tokens, n_q, n_kv, n_values, page_size, scale, num_pages, max_chunks, \
-  window, cap, head_bias, stream
+  window, keep_first, cap, head_bias, stream
   switch (dk) {
     case 32: return launch_scored_mma<32>(LSE_SCORED_MMA_ARGS);
     case 48: return launch_scored_mma<48>(LSE_SCORED_MMA_ARGS);
@@ -396,5 +409,5 @@ extern "C" int lse_attention_scored_mma(const void* q, const void* k_cache, cons
                                         cudaStream_t stream) {
   return lse_attention_scored_mma_windowed(q, k_cache, v_cache, out, out_f32, block_tables, bt_stride, segment_start,
                                            segment_first_pos, num_segments, r1, r2, sink, tokens, n_q, n_kv, dk, dv, cross,
-                                           page_size, scale, num_pages, partials, max_chunks, 0, 0.f, nullptr, stream);
+                                           page_size, scale, num_pages, partials, max_chunks, 0, 0, 0.f, nullptr, stream);
 }

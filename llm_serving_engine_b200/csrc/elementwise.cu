@@ -60,6 +60,33 @@ extern "C" int lse_embedding(const void* table, int table_dtype, const int* ids,
   return lse_embedding_copies(table, table_dtype, ids, out, tokens, hidden, vocab, 1, stream);
 }
 
+// out[t, :] += float(table[ids[t], :]) * scale      (rows with an id outside the table are left alone)
+template <typename T>
+__global__ void embedding_add_kernel(const T* __restrict__ table, const int* __restrict__ ids, float* __restrict__ out,
+                                     int hidden, int vocab, float scale) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  const int id = LSE_CHECKED(ids[t], 0, vocab, -1, LSE_CHECK_TOKEN_ID);
+  if (id < 0 || id >= vocab) return;
+  const T* src = table + (size_t)id * hidden;
+  float* dst = out + (size_t)t * hidden;
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] += to_f32<T>(src[i]) * scale;
+}
+
+extern "C" int lse_embedding_add(const void* table, int table_dtype, const int* ids, float* out, int tokens, int hidden,
+                                 int vocab, float scale, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  const int threads = hidden >= 1024 ? 256 : 128;
+  if (table_dtype == LSE_DTYPE_F32)
+    lse_launch(embedding_add_kernel<float>, tokens, threads, 0, stream, (const float*)table, ids, out, hidden, vocab, scale);
+  else if (table_dtype == LSE_DTYPE_BF16)
+    lse_launch(embedding_add_kernel<__nv_bfloat16>, tokens, threads, 0, stream, (const __nv_bfloat16*)table, ids, out, hidden, vocab, scale);
+  else
+    return LSE_ERR_BAD_ARGUMENT;
+  LSE_LAUNCH_CHECK();
+}
+
 // ------------------------------------------------------------------ add + RMSNorm
 // For output row r (source row s = rows ? rows[r] : r):
 //   x = residual[s] + sum_p float(delta[p][s])   (delta may be null)

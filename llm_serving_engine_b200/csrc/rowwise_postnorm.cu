@@ -287,7 +287,9 @@ __global__ void head_norm_kv_write_kernel(const TI* __restrict__ proj, int n_par
 // The same with a rotation behind the norm: the first rot_dims values of every query and key head are rotated in pairs
 // (value i with value i + rot_dims / 2) by the angle position * freq[i], formed in double precision; cosine and sine are
 // multiplied by rot_factor.  A warp owns a head of a token and passes its normed values through shared memory, so
-// that a lane finds its partner's; heads up to 256 wide.
+// that a lane finds its partner's; heads up to 256 wide.  q_factor (per query head, or null) multiplies the finished
+// queries.  values_are_keys: there are no value columns, a value head is the key head as projected (bias added, neither
+// normed nor rotated).
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(128)
 head_norm_rope_kv_write_kernel(const TI* __restrict__ proj, int n_partials, long long partial_stride, long long ld,
@@ -295,7 +297,8 @@ head_norm_rope_kv_write_kernel(const TI* __restrict__ proj, int n_partials, long
                                const float* __restrict__ k_norm, float eps, const int* __restrict__ slot_mapping,
                                const int* __restrict__ positions, const double* __restrict__ freq, float rot_factor,
                                int rot_dims, TO* __restrict__ q_out, TO* __restrict__ k_cache, TO* __restrict__ v_cache,
-                               int tokens, int n_q, int n_kv, int dk, int dv, int page_size, int num_pages) {
+                               int tokens, int n_q, int n_kv, int dk, int dv, int page_size, int num_pages,
+                               const float* __restrict__ q_factor, int values_are_keys) {
   __shared__ float staged[4][256];
   pdl_launch_dependents();
   pdl_wait();
@@ -320,7 +323,7 @@ head_norm_rope_kv_write_kernel(const TI* __restrict__ proj, int n_partials, long
       dst = k_cache + (((size_t)page * n_kv + h) * page_size + offset) * dk;
     } else {
       const int h = item - n_q - n_kv;
-      column = (n_q + n_kv) * dk + h * dv; width = dv;
+      column = values_are_keys ? (n_q + h) * dk : (n_q + n_kv) * dk + h * dv; width = dv;
       dst = v_cache + (((size_t)page * n_kv + h) * page_size + offset) * dv;
       rotated = false;
     }
@@ -339,6 +342,7 @@ head_norm_rope_kv_write_kernel(const TI* __restrict__ proj, int n_partials, long
   __syncwarp();
   const int half = rot_dims / 2;
   const int position = positions[t];
+  const float factor = q_factor && item < n_q ? q_factor[item] : 1.f;
   for (int i = lane; i < width; i += 32) {
     float x = norm_w ? (mine[i] * inv) * norm_w[i] : mine[i];
     if (rotated && i < rot_dims) {
@@ -350,7 +354,7 @@ head_norm_rope_kv_write_kernel(const TI* __restrict__ proj, int n_partials, long
       const float c = (float)cosine * rot_factor, s = (float)sine * rot_factor;
       x = i < half ? x * c - y * s : x * c + y * s;
     }
-    dst[i] = from_f32<TO>(x);
+    dst[i] = from_f32<TO>(x * factor);
   }
 }
 
@@ -434,17 +438,19 @@ extern "C" int lse_head_norm_kv_write(const void* proj, int in_dtype, int n_part
 }
 
 // As lse_head_norm_kv_write, then the first rot_dims values of every query and key head rotated (freq float64
-// [rot_dims / 2], positions int32 [tokens], cosine and sine times rot_factor).  Heads up to 256 wide.
+// [rot_dims / 2], positions int32 [tokens], cosine and sine times rot_factor), the queries times q_factor (float32 [n_q] or
+// null); values_are_keys (dk = dv): the row of proj is [q | k | anything else].  Heads up to 256 wide.
 extern "C" int lse_head_norm_rope_kv_write(const void* proj, int in_dtype, int n_partials, long long partial_stride,
                                            long long ld, const float* bias, const float* q_norm, const float* k_norm,
                                            float eps, const int* slot_mapping, const int* positions, const double* freq,
                                            float rot_factor, int rot_dims, void* q_out, void* k_cache, void* v_cache,
                                            int out_dtype, int tokens, int n_q, int n_kv, int dk, int dv, int page_size,
-                                           int num_pages, cudaStream_t stream) {
+                                           int num_pages, const float* q_factor, int values_are_keys,
+                                           cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (n_q <= 0 || n_kv <= 0 || dk <= 0 || dv <= 0 || n_partials < 1 || dk > 256 || dv > 256) return LSE_ERR_BAD_ARGUMENT;
   if (rot_dims < 0 || rot_dims % 2 || rot_dims > dk || (rot_dims > 0 && (!freq || !positions))) return LSE_ERR_BAD_ARGUMENT;
-  if (!k_cache || !v_cache || !slot_mapping || page_size <= 0) return LSE_ERR_BAD_ARGUMENT;
+  if (!k_cache || !v_cache || !slot_mapping || page_size <= 0 || (values_are_keys && dk != dv)) return LSE_ERR_BAD_ARGUMENT;
   const long long warps = (long long)tokens * (n_q + 2 * n_kv);
   const int threads = 128;
   const long long blocks = (warps * 32 + threads - 1) / threads;
@@ -452,7 +458,7 @@ extern "C" int lse_head_norm_rope_kv_write(const void* proj, int in_dtype, int n
 #define LSE_HEADROPE_CASE(TI, TO)                                                                                      \
   lse_launch(head_norm_rope_kv_write_kernel<TI, TO>, (unsigned)blocks, threads, 0, stream, (const TI*)proj, n_partials, \
              partial_stride, ld, bias, q_norm, k_norm, eps, slot_mapping, positions, freq, rot_factor, rot_dims,       \
-             (TO*)q_out, (TO*)k_cache, (TO*)v_cache, tokens, n_q, n_kv, dk, dv, page_size, num_pages)
+             (TO*)q_out, (TO*)k_cache, (TO*)v_cache, tokens, n_q, n_kv, dk, dv, page_size, num_pages, q_factor, values_are_keys)
   if (in_dtype == LSE_DTYPE_F32 && out_dtype == LSE_DTYPE_F32) LSE_HEADROPE_CASE(float, float);
   else if (in_dtype == LSE_DTYPE_BF16 && out_dtype == LSE_DTYPE_BF16) LSE_HEADROPE_CASE(__nv_bfloat16, __nv_bfloat16);
   else if (in_dtype == LSE_DTYPE_F32 && out_dtype == LSE_DTYPE_BF16) LSE_HEADROPE_CASE(float, __nv_bfloat16);

@@ -140,10 +140,27 @@ _SIGNATURES = {
     "lse_gated_act_mul_limit": [c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p],
     "lse_head_norm_rope_kv_write": [c_void_p, c_int, c_int, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_float,
                                     c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p, c_void_p, c_int,
-                                    c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+                                    c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p],
+    "lse_conv_norm_supported": [c_int, c_int],
+    "lse_conv_norm": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_float,
+                      c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                      c_int, c_int, c_void_p],
+    "lse_conv_norm_state": [c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "lse_delta_norm_rmsnorm": [c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_float,
+                               c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "lse_residual_settle": [c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+    "lse_token_gate": [c_void_p, c_int, c_int, c_longlong, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_int, c_void_p,
+                       c_int, c_int, c_int, c_int, c_void_p],
+    "lse_embedding_add": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
+    "lse_delta_prepare": [c_void_p, c_int, c_int, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                          c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                          c_int, c_int, c_float, c_int, c_int, c_int, c_void_p],
+    "lse_delta_scan": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_longlong, c_void_p, c_void_p,
+                       c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "lse_attention_scored_windowed": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p,
                                       c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                      c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p],
+                                      c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p,
+                                      c_void_p],
     "lse_gated_linear_attention_scan_shared": [c_void_p, c_int, c_int, c_longlong, c_longlong, c_int, c_int, c_int,
                                                c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                                c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
@@ -161,9 +178,9 @@ _SIGNATURES = {
                               c_int, c_int, c_int, c_int, c_int, c_float, c_void_p],
     "lse_attention_scored_mma_windowed": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                           c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                          c_float, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p],
+                                          c_float, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
     "lse_attention_scored_merge_windowed": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                                            c_int, c_int, c_int, c_int, c_int, c_void_p],
+                                            c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "lse_attention_sigmoid_tc": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
                                  c_longlong, c_int, c_int, c_int, c_int, c_float, c_void_p, c_float, c_void_p, c_void_p,
                                  c_longlong, c_void_p],
@@ -210,7 +227,8 @@ CHECK_READERS = ("lse_check_elementwise", "lse_check_attention_generic", "lse_ch
                  "lse_check_residual_streams", "lse_check_linear_attention", "lse_check_linear_attention_gated",
                  "lse_check_linear_attention_vector", "lse_check_attention_latent",
                  "lse_check_attention_latent_mma", "lse_check_rowwise_postnorm", "lse_check_attention_scored",
-                 "lse_check_attention_scored_mma", "lse_check_mlstm", "lse_check_short_conv", "lse_check_selective_scan")
+                 "lse_check_attention_scored_mma", "lse_check_mlstm", "lse_check_short_conv", "lse_check_selective_scan", "lse_check_conv_norm",
+                 "lse_check_delta_memory")
 CHECK_KINDS = {1: "token id", 2: "cache slot", 3: "block-table entry", 4: "segment number", 5: "row index"}
 
 

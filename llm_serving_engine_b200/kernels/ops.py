@@ -57,6 +57,17 @@ def embedding(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, copies:
     return out
 
 
+def embedding_add(table: torch.Tensor, ids: torch.Tensor, residual: torch.Tensor, scale: float = 1.0) -> torch.Tensor:
+    """residual[t] += float32(table[ids[t]]) * scale; ids int32 [T], residual float32 [T, H]."""
+    _need_cuda(table, ids, residual)
+    vocab, hidden = table.shape
+    assert ids.dtype == torch.int32 and residual.dtype == torch.float32 and table.is_contiguous()
+    assert residual.shape == (ids.shape[0], hidden) and residual.is_contiguous()
+    check(library.load().lse_embedding_add(table.data_ptr(), dtype_code(table.dtype), ids.data_ptr(), residual.data_ptr(),
+                                           ids.shape[0], hidden, vocab, float(scale), _stream()), "embedding_add")
+    return residual
+
+
 def _partials(tensor: torch.Tensor | None, rows: int, width: int):
     """(tensor, number of partial sums, elements between them) of a [rows, width] tensor or a
     float32 stack of partial sums [P, rows, width]."""
@@ -812,12 +823,15 @@ def head_norm_kv_write(proj: torch.Tensor, bias: torch.Tensor | None, q_norm: to
 def head_norm_rope_kv_write(proj: torch.Tensor, bias: torch.Tensor | None, q_norm: torch.Tensor | None,
                             k_norm: torch.Tensor | None, eps: float, slot_mapping: torch.Tensor, positions: torch.Tensor,
                             freq: torch.Tensor, rot_factor: float, q_out: torch.Tensor, k_cache: torch.Tensor,
-                            v_cache: torch.Tensor, n_q: int, n_kv: int, dk: int, dv: int, offset: int = 0) -> None:
+                            v_cache: torch.Tensor, n_q: int, n_kv: int, dk: int, dv: int, offset: int = 0,
+                            q_factor: torch.Tensor | None = None, values_are_keys: bool = False) -> None:
     """As :func:`head_norm_kv_write` (the row [q | k | v] starts at column ``offset`` of ``proj``; ``bias`` counts from
     there), and behind the norm the first ``2 * len(freq)`` values of every query and key head
     are rotated: value i with value i + len(freq), by the angle position * freq[i] (``freq`` float64, the angle formed
-    in double precision); cosine and sine are multiplied by ``rot_factor``.  Heads up to 256 wide."""
-    _need_cuda(proj, bias, q_norm, k_norm, slot_mapping, positions, freq, q_out, k_cache, v_cache)
+    in double precision); cosine and sine are multiplied by ``rot_factor``.  Heads up to 256 wide.  ``q_factor`` (float32
+    [n_q]) multiplies the finished queries; ``values_are_keys`` (dk = dv): the row is [q | k], and a value head is the key
+    head as projected, with its bias, neither normed nor rotated."""
+    _need_cuda(proj, bias, q_norm, k_norm, slot_mapping, positions, freq, q_out, k_cache, v_cache, q_factor)
     proj, code, n_partials, stride, ld = _projection(proj)
     tokens = proj.shape[-2]
     assert q_out.shape == (tokens, n_q, dk) and q_out.is_contiguous()
@@ -828,11 +842,13 @@ def head_norm_rope_kv_write(proj: torch.Tensor, bias: torch.Tensor | None, q_nor
     assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == v_cache.dtype == q_out.dtype
     assert k_cache.shape[1] == n_kv and k_cache.shape[3] == dk and v_cache.shape[3] == dv
     assert slot_mapping.dtype == torch.int32 and slot_mapping.shape[0] >= tokens
+    assert q_factor is None or (q_factor.dtype == torch.float32 and q_factor.shape == (n_q,))
     check(library.load().lse_head_norm_rope_kv_write(
         proj.data_ptr() + int(offset) * proj.element_size(), code, n_partials, stride, ld, _ptr(bias), _ptr(q_norm), _ptr(k_norm), float(eps),
         slot_mapping.data_ptr(), positions.data_ptr(), freq.data_ptr() if freq.numel() else None, float(rot_factor),
         2 * freq.numel(), q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), dtype_code(q_out.dtype), tokens, n_q,
-        n_kv, dk, dv, k_cache.shape[2], k_cache.shape[0], _stream()), "head_norm_rope_kv_write")
+        n_kv, dk, dv, k_cache.shape[2], k_cache.shape[0], _ptr(q_factor), int(values_are_keys), _stream()),
+        "head_norm_rope_kv_write")
 
 
 def attention_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor,
@@ -840,7 +856,8 @@ def attention_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      r1: torch.Tensor | None = None, r2: torch.Tensor | None = None, sink: torch.Tensor | None = None,
                      cross: bool = False, split: bool | None = None, segment_start: torch.Tensor | None = None,
                      segment_first_position: torch.Tensor | None = None, tensor_cores: bool = True,
-                     window: int = 0, cap: float = 0.0, head_bias: torch.Tensor | None = None) -> torch.Tensor:
+                     window: int = 0, cap: float = 0.0, head_bias: torch.Tensor | None = None,
+                     keep_first: int = 0) -> torch.Tensor:
     """Causal attention of every row of the step over its request's pages, with the scores or weights changed:
     s_ij = q_i . k_j * scale - r1_h ln(1 + r2_h (i - j)) (``r1``, ``r2`` float32 [n_q]); exp(sink_h) in the
     denominator (``sink`` float32 [n_q]).  q [T, n_q, dk]; k_cache [pages, n_kv, page, dk]; v_cache [.., dv];
@@ -848,7 +865,8 @@ def attention_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     key/value head.  ``out`` is in the cache's dtype or float32.  ``split`` as for :func:`paged_attention_generic`.
     Given the step's ``segment_start`` (int32 [S + 1]) and ``segment_first_position`` (int32 [S]), bfloat16 shapes that
     the tensor-core kernel takes run there (``tensor_cores=False``: the general kernel, for comparisons).
-    ``window`` > 0: a row reads its last ``window`` keys only (itself included).  ``cap`` > 0: scores become
+    ``window`` > 0: a row reads its last ``window`` keys only (itself included) and, with ``keep_first`` > 0, of those before
+    them the request's first ``keep_first``.  ``cap`` > 0: scores become
     cap * tanh(s / cap).  ``head_bias`` (float32 [n_q]): no softmax; a key's weight is sigmoid(s + head_bias_h) and the
     weights are not normalised over the keys."""
     _need_cuda(q, k_cache, v_cache, out, block_tables, segment_of_token, positions, r1, r2, sink, segment_start,
@@ -880,20 +898,20 @@ def attention_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
             q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), int(out.dtype == torch.float32),
             block_tables.data_ptr(), block_tables.stride(0), segment_start.data_ptr(), segment_first_position.data_ptr(),
             segments, _ptr(r1), _ptr(r2), _ptr(sink), tokens, n_q, n_kv, dk, dv, int(cross), page_size, float(scale),
-            k_cache.shape[0], _ptr(partials), max_chunks, int(window), float(cap), _ptr(head_bias), _stream()),
-            "attention_scored_mma")
+            k_cache.shape[0], _ptr(partials), max_chunks, int(window), int(keep_first), float(cap), _ptr(head_bias),
+            _stream()), "attention_scored_mma")
         if partials is not None:
             check(lib.lse_attention_scored_merge_windowed(
                 partials.data_ptr(), out.data_ptr(), dtype_code(out.dtype), segment_of_token.data_ptr(),
                 positions.data_ptr(), _ptr(sink), tokens, n_q, n_values, dv, max_chunks, block_tables.shape[0],
-                int(window), int(head_bias is not None), _stream()), "attention_scored_merge")
+                int(window), int(keep_first), int(head_bias is not None), _stream()), "attention_scored_merge")
         return out
     check(lib.lse_attention_scored_windowed(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), dtype_code(q.dtype),
         int(out.dtype == torch.float32 and q.dtype != torch.float32), block_tables.data_ptr(), block_tables.stride(0),
         segment_of_token.data_ptr(), positions.data_ptr(), _ptr(r1), _ptr(r2), _ptr(sink), tokens, n_q, n_kv, dk, dv,
         int(cross), page_size, float(scale), k_cache.shape[0], block_tables.shape[0], _ptr(partials), max_chunks,
-        int(window), float(cap), _ptr(head_bias), _stream()), "attention_scored")
+        int(window), int(keep_first), float(cap), _ptr(head_bias), _stream()), "attention_scored")
     return out
 
 
@@ -1461,4 +1479,151 @@ def selective_scan(x: torch.Tensor, dt: torch.Tensor, proj: torch.Tensor, z_off:
         state.data_ptr(), step.segment_start.data_ptr(), step.segment_state_slot.data_ptr(), out.data_ptr(),
         dtype_code(out.dtype), out.stride(0), float(scale), step.segment_state_slot.shape[0], channels, states,
         state.shape[0], chunk_rows, _ptr(chunk_state), _ptr(chunk_dt), max_chunks, _stream()), "selective_scan")
+    return out
+
+
+# ------------------------------------------------------------------ norm and convolution of a sublayer's input, token input
+def delta_norm_rmsnorm(residual: torch.Tensor, delta: torch.Tensor | None, bias: torch.Tensor | None,
+                       delta_norm: tuple[torch.Tensor, float] | None, weight: torch.Tensor, eps: float, out: torch.Tensor,
+                       rows: torch.Tensor | None = None, write_residual: bool = True) -> torch.Tensor:
+    """x = residual + d with d = delta + bias, or delta / rms(delta) * w for ``delta_norm`` = (w float32 [H], eps);
+    out = x / rms(x) * weight, and the residual becomes x (``write_residual``).  Other arguments as :func:`add_rmsnorm`."""
+    _need_cuda(residual, delta, bias, weight, out, rows)
+    tokens, hidden = residual.shape
+    assert residual.dtype == torch.float32 and residual.is_contiguous() and weight.dtype == torch.float32 and weight.shape == (hidden,)
+    assert out.is_contiguous() and out.shape[1] == hidden
+    assert bias is None or (bias.dtype == torch.float32 and bias.shape == (hidden,))
+    delta, n_partials, stride = _partials(delta, tokens, hidden)
+    dw, deps = delta_norm if delta_norm is not None else (None, 0.0)
+    assert dw is None or (dw.dtype == torch.float32 and dw.shape == (hidden,))
+    n_rows = out.shape[0]
+    assert (rows is None and n_rows == tokens) or (rows is not None and rows.dtype == torch.int32 and rows.shape[0] == n_rows)
+    check(library.load().lse_delta_norm_rmsnorm(
+        residual.data_ptr(), _ptr(delta), dtype_code(delta.dtype) if delta is not None else F32, n_partials, stride, _ptr(bias),
+        _ptr(dw), float(deps), weight.data_ptr(), float(eps), out.data_ptr(), dtype_code(out.dtype), _ptr(rows), n_rows, hidden,
+        tokens, int(write_residual), _stream()), "delta_norm_rmsnorm")
+    return out
+
+
+CONV_NORM_BLOCKS_PER_SM = 2
+
+
+def conv_norm(residual: torch.Tensor, delta: torch.Tensor | None, bias: torch.Tensor | None,
+              delta_norm: tuple[torch.Tensor, float] | None, weight: torch.Tensor, eps: float, conv_weight: torch.Tensor,
+              state: torch.Tensor, step, out: torch.Tensor) -> torch.Tensor:
+    """The pending output added as in :func:`delta_norm_rmsnorm`, h = rmsnorm(x) * weight, and
+    out_t = h_t + sum_j conv_weight[:, j] h_(t - taps + 1 + j) over the request's rows of h and, before this step's, its
+    window in ``state`` float32 [slots, taps - 1, H], which moves on.  conv_weight float32 [H, taps].  Returns the new
+    residual (a tensor of its own for the shapes of the fused kernel)."""
+    _need_cuda(residual, delta, bias, weight, conv_weight, state, out)
+    tokens, hidden = residual.shape
+    taps = conv_weight.shape[1]
+    assert residual.dtype == torch.float32 and residual.is_contiguous() and weight.dtype == torch.float32 and weight.shape == (hidden,)
+    assert conv_weight.dtype == torch.float32 and conv_weight.shape == (hidden, taps) and conv_weight.is_contiguous()
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (taps - 1, hidden)
+    assert out.is_contiguous() and out.shape == (tokens, hidden)
+    lib = library.load()
+    if not lib.lse_conv_norm_supported(hidden, taps):     # two launches: norm in float32, then the convolution
+        h = torch.empty((tokens, hidden), dtype=torch.float32, device=residual.device)
+        delta_norm_rmsnorm(residual, delta, bias, delta_norm, weight, eps, h)
+        through = conv_weight.clone()
+        through[:, -1] += 1.0                             # h + conv(h)
+        short_conv_act(h, 0, through, None, state, step, out, "none")
+        if taps > 1:
+            short_conv_state(h, 0, hidden, taps, state, step)
+        return residual
+    assert bias is None or (bias.dtype == torch.float32 and bias.shape == (hidden,))
+    delta, n_partials, stride = _partials(delta, tokens, hidden)
+    dw, deps = delta_norm if delta_norm is not None else (None, 0.0)
+    assert dw is None or (dw.dtype == torch.float32 and dw.shape == (hidden,))
+    segments = step.segment_state_slot.shape[0]
+    single = bool(step.decode_only)
+    rows_per_block = 1 if single else max(1, min(16, -(-tokens // (CONV_NORM_BLOCKS_PER_SM * sm_count()))))
+    fresh = torch.empty_like(residual)
+    check(lib.lse_conv_norm(
+        residual.data_ptr(), fresh.data_ptr(), _ptr(delta), dtype_code(delta.dtype) if delta is not None else F32, n_partials,
+        stride, _ptr(bias), _ptr(dw), float(deps), weight.data_ptr(), float(eps), conv_weight.data_ptr(), state.data_ptr(),
+        step.segment_of_token.data_ptr(), step.segment_start.data_ptr(), step.segment_state_slot.data_ptr(), out.data_ptr(),
+        dtype_code(out.dtype), tokens, rows_per_block, hidden, taps, int(single), state.shape[0], segments, _stream()), "conv_norm")
+    if not single and taps > 1:
+        check(lib.lse_conv_norm_state(fresh.data_ptr(), weight.data_ptr(), float(eps), state.data_ptr(),
+                                      step.segment_start.data_ptr(), step.segment_state_slot.data_ptr(), segments, hidden, taps,
+                                      state.shape[0], _stream()), "conv_norm_state")
+    return fresh
+
+
+def residual_settle(residual: torch.Tensor, delta: torch.Tensor, bias: torch.Tensor | None, copy: torch.Tensor | None) -> None:
+    """residual += delta + bias, in place; ``copy`` ([T, H] in float32 or bfloat16, or None) receives the sum, rounded."""
+    _need_cuda(residual, delta, bias, copy)
+    tokens, hidden = residual.shape
+    assert residual.dtype == torch.float32 and residual.is_contiguous()
+    assert bias is None or (bias.dtype == torch.float32 and bias.shape == (hidden,))
+    assert copy is None or (copy.shape == residual.shape and copy.is_contiguous())
+    delta, n_partials, stride = _partials(delta, tokens, hidden)
+    check(library.load().lse_residual_settle(residual.data_ptr(), delta.data_ptr(), dtype_code(delta.dtype), n_partials, stride,
+                                             _ptr(bias), _ptr(copy), dtype_code(copy.dtype) if copy is not None else F32, tokens,
+                                             hidden, _stream()), "residual_settle")
+
+
+def token_gate(z: torch.Tensor, table: torch.Tensor, offset: int, ids: torch.Tensor, out: torch.Tensor, dim: int) -> torch.Tensor:
+    """out[t, i] = gelu_tanh(z[t, i]) * table[ids[t], offset + i] for i < dim, zero in out's further columns; z: a
+    projection's rows or partial sums; table [vocab, N] and out [T, >= dim] in the compute dtype."""
+    _need_cuda(z, table, ids, out)
+    z, code, n_partials, stride, ld = _projection(z)
+    tokens = out.shape[0]
+    assert table.dtype == out.dtype and table.is_contiguous() and out.is_contiguous() and ids.dtype == torch.int32
+    assert out.shape[1] >= dim and z.shape[-1] >= dim and offset + dim <= table.shape[1]
+    check(library.load().lse_token_gate(z.data_ptr(), code, n_partials, stride, ld, table.data_ptr(), table.shape[1], int(offset),
+                                        ids.data_ptr(), table.shape[0], out.data_ptr(), dtype_code(out.dtype), tokens, int(dim),
+                                        out.shape[1], _stream()), "token_gate")
+    return out
+
+
+# ------------------------------------------------------------------ delta memory
+def delta_prepare(proj: torch.Tensor, conv_weight: torch.Tensor, state: torch.Tensor, step, low: torch.Tensor, groups: int,
+                  heads: int, dim: int, vdim: int, rank: int, q_scale: float):
+    """Columns of ``proj``: [q (groups * dim) | k (groups * dim) | v (heads * vdim) | beta (heads) | low (rank)].  q, k and v
+    pass a short convolution per channel (``conv_weight`` float32 [channels, taps], windows in ``state`` float32 [slots,
+    taps - 1, channels], moved on) and SiLU; every head of q and k is divided by sqrt(sum x^2 + 1e-6), q times ``q_scale``;
+    ``low`` [T, >= rank] receives the low-rank columns in the compute dtype, zeros behind them.  Returns float32 (q
+    [T, groups * dim], k, v [T, heads * vdim], beta [T, heads] = sigmoid)."""
+    _need_cuda(proj, conv_weight, state, low)
+    proj, code, n_partials, stride, ld = _projection(proj)
+    tokens = low.shape[0]
+    channels, taps = conv_weight.shape
+    assert channels == 2 * groups * dim + heads * vdim and conv_weight.dtype == torch.float32 and conv_weight.is_contiguous()
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (taps - 1, channels)
+    assert proj.shape[-1] >= channels + heads + rank and proj.shape[-2] == tokens and low.is_contiguous()
+    new = lambda width: torch.empty((tokens, width), dtype=torch.float32, device=low.device)
+    q, k, v, beta = new(groups * dim), new(groups * dim), new(heads * vdim), new(heads)
+    single = bool(step.decode_only)
+    check(library.load().lse_delta_prepare(
+        proj.data_ptr(), code, n_partials, stride, ld, conv_weight.data_ptr(), state.data_ptr(), step.segment_of_token.data_ptr(),
+        step.segment_start.data_ptr(), step.segment_state_slot.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(),
+        low.data_ptr(), dtype_code(low.dtype), low.shape[1], tokens, groups, heads, dim, vdim, rank, taps, float(q_scale),
+        int(single), state.shape[0], step.segment_state_slot.shape[0], _stream()), "delta_prepare")
+    if not single and taps > 1:
+        short_conv_state(proj, 0, channels, taps, state, step)
+    return q, k, v, beta
+
+
+def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Tensor, z: torch.Tensor, dt_bias: torch.Tensor,
+               a_log: torch.Tensor, state: torch.Tensor, segment_start: torch.Tensor, segment_slot: torch.Tensor,
+               out: torch.Tensor, heads: int, groups: int, dim: int, vdim: int) -> torch.Tensor:
+    """S <- diag(keep) S;  u = beta (v - S^T k);  S <- S + k u^T;  out = S^T q, over the rows of every request in order, from
+    and into ``state`` float32 [slots, heads, dim, vdim]; keep = exp(-exp(a_log_h) softplus(z + dt_bias)) per head and key
+    channel, z float32 columns 0 .. heads * dim of a projection (rows or partial sums).  Other arguments as
+    :func:`delta_prepare` returns them; out float32 [T, heads * vdim]."""
+    _need_cuda(q, k, v, beta, z, dt_bias, a_log, state, segment_start, segment_slot, out)
+    z, code, z_partials, z_stride, z_ld = _projection(z)
+    tokens = out.shape[0]
+    assert code == F32 and z.shape[-1] >= heads * dim and dt_bias.shape == (heads * dim,) and a_log.shape == (heads,)
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (heads, dim, vdim)
+    assert out.dtype == torch.float32 and out.is_contiguous() and out.shape == (tokens, heads * vdim)
+    segments = segment_slot.shape[0]
+    assert segment_start.dtype == segment_slot.dtype == torch.int32 and segment_start.shape[0] == segments + 1
+    check(library.load().lse_delta_scan(
+        q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(), z.data_ptr(), z_partials, z_stride, z_ld, dt_bias.data_ptr(),
+        a_log.data_ptr(), state.data_ptr(), segment_start.data_ptr(), segment_slot.data_ptr(), out.data_ptr(), segments, heads,
+        groups, dim, vdim, state.shape[0], 0, _stream()), "delta_scan")
     return out

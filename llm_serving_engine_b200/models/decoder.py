@@ -7,7 +7,7 @@ import torch
 
 from ..config.model_config import LayerSpec, ModelSpec, PartSpec
 from ..kernels import ops
-from ..parts.base import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, BuildContext, ResidualStream)
+from ..parts.base import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, BuildContext, ResidualStream, cache_needs)
 from ..parts.linear import linear
 from ..weights.tensor_spec import TensorSpec
 
@@ -58,6 +58,8 @@ def expected_tensors(spec: ModelSpec) -> dict[str, TensorSpec]:
                 out[prefix + local] = tensor
         for local, tensor in _block_tensors(layer, spec.hidden_size).items():
             out[layer.prefix + local] = tensor
+    for name, shape in spec.shared_tensors.items():
+        out[name] = TensorSpec(tuple(shape))
     if spec.position_table_name:
         out[spec.position_table_name] = TensorSpec((spec.max_position_embeddings, spec.hidden_size))
     norm_cls = NORMS.get(spec.final_norm.kind)
@@ -73,7 +75,8 @@ def cache_requirements(spec: ModelSpec) -> list:
 
     The list runs along ``order``, not along ``layers``: a layer that is named twice
     runs twice with the same weights, and each run has a cache of its own.  An entry
-    is ``PagedKV``, ``RequestState`` or ``None`` (from the mixer), or an int: the
+    is ``PagedKV``, ``RequestState`` or ``None`` (from the mixer), a tuple of such needs (the
+    mixer's, then what the layer's arrangement keeps itself), or an int: the
     position in ``order`` whose cache this run reads (``LayerSpec.cache_from`` names a
     layer; its first run is meant, and it must come earlier in the order).
     """
@@ -88,7 +91,10 @@ def cache_requirements(spec: ModelSpec) -> list:
                 raise ConfigError(f"layer {index} reads the cache of layer {layer.cache_from}, which has not run before it")
             out.append(first_run[layer.cache_from])
         else:
-            out.append(MIXERS.get(layer.mixer.kind).cache_requirement(layer.mixer.params, spec.hidden_size))
+            need = MIXERS.get(layer.mixer.kind).cache_requirement(layer.mixer.params, spec.hidden_size)
+            declare = getattr(BLOCKS.get(layer.block.kind), "cache_requirement", None)
+            own = cache_needs(declare(layer.block.params, spec.hidden_size)) if declare else ()
+            out.append(cache_needs(need) + own if own else need)
         first_run.setdefault(index, position)
     return out
 
@@ -102,8 +108,9 @@ class DecoderModel:
         self.lm_head = self.embedding if spec.tie_word_embeddings else weights[spec.lm_head_name].contiguous()
         self.position_table = weights[spec.position_table_name].contiguous() if spec.position_table_name else None
         self.blocks = []
+        shared = {name: weights[name].contiguous() for name in spec.shared_tensors}
         for index, layer in enumerate(spec.layers):
-            ctx = BuildContext(dtype, self.device, spec.hidden_size, index, spec.max_position_embeddings)
+            ctx = BuildContext(dtype, self.device, spec.hidden_size, index, spec.max_position_embeddings, shared)
             built = []
             for entry in _layer_parts(layer):
                 if entry is None:
@@ -150,12 +157,14 @@ class DecoderModel:
         total = self.lm_head.numel() * self.lm_head.element_size()
         for index in self.spec.order:
             block = self.blocks[index]
-            for part in (block.mixer, block.feed_forward, block.mixer_norm, block.feed_forward_norm):
+            for part in (block.mixer, block.feed_forward, block.mixer_norm, block.feed_forward_norm,
+                         getattr(block, "token_input", None)):
                 if part is None:
                     continue
                 held: dict[int, int] = {}     # a part may keep views of a matrix beside it: every storage counts once
                 for value in vars(part).values():
-                    if isinstance(value, torch.Tensor) and value.dim() >= 1 and value.is_floating_point():
+                    if (isinstance(value, torch.Tensor) and value.dim() >= 1 and value.is_floating_point()
+                            and not any(value is table for table in part.ctx.shared.values())):   # rows are gathered from these
                         key = value.untyped_storage().data_ptr()
                         held[key] = max(held.get(key, 0), value.numel() * value.element_size())
                 total += sum(held.values())
@@ -179,7 +188,11 @@ class DecoderModel:
             # every copy starts as the embedding
             ops.embedding(self.embedding, step.token_ids, residual, copies, scale=self.spec.embedding_scale)
             stream = ResidualStream(residual, copies=copies)
+        if self.spec.embedding_again and copies != 1:
+            raise ops.KernelError("the embedding is added again to one copy of the residual only")
         for position, index in enumerate(self.spec.order):   # caches run along the order
+            if position in self.spec.embedding_again:
+                ops.embedding_add(self.embedding, step.token_ids, stream.residual, self.spec.embedding_scale)
             self.blocks[index].forward(stream, step, caches[position])
             if self.layer_hook is not None:
                 self.layer_hook(position, stream)

@@ -16,8 +16,10 @@ configuration), ``weights`` (its own tensors, by their local names) and a
                        fixed-size state per request, or nothing, or a tuple of
                        several such needs: pages and a state, two states)
 * ``FeedForward``:     ``forward(x) -> y``, row-local
+* ``TokenInput``:      ``forward(x, step) -> y``, row-local, from the rows and the step's token ids
 * ``Block``:           the arrangement of the four in a layer:
-                       ``forward(stream, step, cache)``
+                       ``forward(stream, step, cache)``; its own ``cache_requirement`` (what the arrangement
+                       keeps per request) follows the mixer's in the layer's
 
 Each class also has ``expected_tensors(params, hidden_size)``: local tensor name
 -> ``TensorSpec``; the loader and the random-weights mode are driven by it.
@@ -39,18 +41,21 @@ class BuildContext:
     hidden_size: int
     layer_index: int
     max_position_embeddings: int
+    shared: dict = field(default_factory=dict)   # tensors that several layers read (``ModelSpec.shared_tensors``), by full name
 
 
 @dataclass(frozen=True)
 class PagedKV:
     """The mixer keeps keys and values of every token in pages.  ``window`` > 0:
     only the last ``window`` keys are read, older pages are given back.
-    ``value_dim`` > 0: a value has this size instead of ``head_dim`` (keys and values then lie in two tensors)."""
+    ``value_dim`` > 0: a value has this size instead of ``head_dim`` (keys and values then lie in two tensors).
+    ``keep_first`` > 0 (with a window): the request's first so many keys are read for ever, their pages stay."""
 
     num_kv_heads: int
     head_dim: int
     window: int = 0
     value_dim: int = 0
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)
@@ -103,6 +108,18 @@ class ResidualStream:
         self.delta_bias = None
         self.delta_row_scale = None   # float32 [T] c: c_t times the branch's input row belongs to the pending output too
         self.delta_norm = None        # a Norm that the pending output passes before it is added (a layer that norms after a branch too)
+
+    def settle(self, dtype: torch.dtype) -> torch.Tensor:
+        """Add the pending output (with its bias) to the residual now, for a branch that reads the residual itself;
+        returns the residual's rows in ``dtype``."""
+        from ..kernels import ops
+
+        if not self.plain or self.delta_norm is not None or self.delta_row_scale is not None:
+            raise ops.KernelError("settle: one copy of the residual, an output that is added as it is")
+        rows = self.residual if dtype == torch.float32 else torch.empty_like(self.residual, dtype=dtype)
+        ops.residual_settle(self.residual, self.delta, self.delta_bias, None if rows is self.residual else rows)
+        self.delta = self.delta_bias = None
+        return rows
 
     @property
     def plain(self) -> bool:
@@ -185,6 +202,16 @@ class FeedForward(Part):
         raise NotImplementedError
 
 
+class TokenInput(Part):
+    """What a layer adds to the residual from the token itself: ``forward(x, step)`` over the rows x of the residual (in the
+    compute dtype) and ``step.token_ids``.  ``norm`` (a Norm, or None): its output passes it before it is added."""
+
+    norm = None
+
+    def forward(self, x: torch.Tensor, step) -> torch.Tensor:
+        raise NotImplementedError
+
+
 class Block:
     graph_safe = False     # as for ``Part``: the arrangement itself launches nothing that depends on the step's contents
 
@@ -198,6 +225,12 @@ class Block:
     def expected_tensors(cls, params: dict[str, Any], hidden_size: int) -> dict[str, TensorSpec]:
         """Tensors of the arrangement itself (scales, mixing weights), by their names after the layer's prefix."""
         return {}
+
+    @classmethod
+    def cache_requirement(cls, params: dict[str, Any], hidden_size: int):
+        """What the arrangement itself keeps between steps, as for ``Mixer.cache_requirement``; ``forward`` finds it in
+        ``cache.parts`` behind the mixer's members."""
+        return None
 
     def parts(self) -> list:
         """Every part this block runs (a mixer's position encoding included)."""
@@ -238,9 +271,11 @@ FEED_FORWARDS = _Registry("feed-forward")
 NORMS = _Registry("norm")
 POSITION_ENCODINGS = _Registry("position encoding")
 BLOCKS = _Registry("block")
+TOKEN_INPUTS = _Registry("token input")
 
 register_mixer = MIXERS.register
 register_feed_forward = FEED_FORWARDS.register
 register_norm = NORMS.register
 register_position_encoding = POSITION_ENCODINGS.register
 register_block = BLOCKS.register
+register_token_input = TOKEN_INPUTS.register

@@ -4,7 +4,7 @@ from __future__ import annotations
 import torch
 
 from ..weights.tensor_spec import TensorSpec
-from .base import NORMS, Block, ResidualStream, register_block
+from .base import MIXERS, NORMS, TOKEN_INPUTS, Block, RequestState, ResidualStream, cache_for, cache_needs, register_block
 from .linear import stack_sums
 
 
@@ -156,3 +156,70 @@ class ParallelResidualBlock(Block):
             stream.delta = mixed
         else:
             stream.delta = stack_sums(mixed, self.feed_forward.forward(x))
+
+
+@register_block("convolved_residual")
+class ConvolvedResidualBlock(Block):
+    """Pre-norm residual layer whose sublayers read h + conv(h), h the normed rows and conv a short causal convolution per
+    channel over the request's tokens, and which may add an input of the token's own behind the feed-forward:
+        h = norm1(x);  x <- x + mixer(h + conv1(h));   h = norm2(x);  x <- x + feed_forward(h + conv2(h));
+        x <- x + norm(token_input(x)).
+
+    params: ``taps`` (of both convolutions), ``conv_names`` ({"mixer": ..., "feed_forward": ...}: names of their weights
+    [hidden, taps] after the layer's prefix), ``mixer`` (the mixer's {"kind", "params"}: its cache needs come before the
+    arrangement's own), ``token_input`` (None, or {"kind", "params", "prefix"}: a registered ``TokenInput``),
+    ``feed_forward`` (false: the layer has none).  Kept per request, in float32: the last taps - 1 rows of h of each
+    sublayer.  Sum, norm and convolution are one launch (``RMSNorm.forward_convolved``); the token input's output stays
+    pending with its norm, which the next norm's launch applies."""
+
+    graph_safe = True
+
+    def __init__(self, params, mixer_norm, mixer, feed_forward_norm, feed_forward, weights=None, ctx=None) -> None:
+        super().__init__(params, mixer_norm, mixer, feed_forward_norm, feed_forward)
+        names = params["conv_names"]
+        self.mixer_conv = weights[names["mixer"]].to(torch.float32).contiguous()
+        self.feed_forward_conv = (weights[names["feed_forward"]].to(torch.float32).contiguous()
+                                  if feed_forward is not None else None)
+        self.token_input = None
+        spec = params.get("token_input")
+        if spec is not None:
+            local = {name[len(spec["prefix"]):]: tensor for name, tensor in weights.items() if name.startswith(spec["prefix"])}
+            self.token_input = TOKEN_INPUTS.get(spec["kind"])(spec["params"], local, ctx)
+        self.mixer_needs = self._mixer_needs(params, ctx.hidden_size)
+
+    @staticmethod
+    def _mixer_needs(params, hidden_size: int) -> int:
+        spec = params["mixer"]
+        return len(cache_needs(MIXERS.get(spec["kind"]).cache_requirement(spec["params"], hidden_size)))
+
+    @classmethod
+    def expected_tensors(cls, params, hidden_size):
+        taps, names = int(params["taps"]), params["conv_names"]
+        roles = ("mixer", "feed_forward") if params.get("feed_forward", True) else ("mixer",)
+        out = {names[role]: TensorSpec((hidden_size, taps), "filter") for role in roles}
+        spec = params.get("token_input")
+        if spec is not None:
+            declared = TOKEN_INPUTS.get(spec["kind"]).expected_tensors(spec["params"], hidden_size)
+            out.update({spec["prefix"] + local: tensor for local, tensor in declared.items()})
+        return out
+
+    @classmethod
+    def cache_requirement(cls, params, hidden_size):
+        window = RequestState((int(params["taps"]) - 1, hidden_size), "float32")
+        return (window, window) if params.get("feed_forward", True) else (window,)
+
+    def parts(self) -> list:
+        return super().parts() + ([self.token_input] if self.token_input is not None else [])
+
+    def forward(self, stream: ResidualStream, step, cache) -> None:
+        windows = [part.state for part in cache.parts[self.mixer_needs:]]
+        x = self.mixer_norm.forward_convolved(stream, self.mixer_conv, windows[0], step)
+        stream.delta = self.mixer.forward(x, step, cache_for(cache, self.mixer_needs))
+        stream.delta_bias = self.mixer.output_bias
+        if self.feed_forward is not None:
+            x = self.feed_forward_norm.forward_convolved(stream, self.feed_forward_conv, windows[1], step)
+            stream.delta = self.feed_forward.forward(x)
+        if self.token_input is not None:
+            x = stream.settle(self.token_input.ctx.dtype)
+            stream.delta = self.token_input.forward(x, step)
+            stream.delta_norm = self.token_input.norm

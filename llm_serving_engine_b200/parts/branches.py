@@ -201,7 +201,7 @@ class SelectiveStateSpace(BranchMixer):
 
 
 _HEAD_NORM_NAMES = {"q": "q", "k": "k", "v": "v", "out": "o", "q_norm": "q.norm", "k_norm": "k.norm",
-                    "bias_suffix": ".b", "head_bias": "pb"}
+                    "bias_suffix": ".b", "head_bias": "pb", "head_factor": "temp"}
 
 
 @register_mixer("head_norm_rotary_attention")
@@ -212,10 +212,14 @@ class HeadNormRotaryAttention(BranchMixer):
     paired with i + dims / 2; see ``rotary_frequencies`` for ``scaling``), ``window`` (> 0: a row reads its last
     ``window`` keys, itself included; older pages are given back), ``softcap`` (> 0: scores become cap * tanh(s / cap)),
     ``weights`` ("softmax", the default, or "sigmoid": a key's weight is sigmoid(score + b_h) with a learned number per
-    head, not normalised over the keys), ``tensor_names``.
+    head, not normalised over the keys), ``head_norm`` (default true), ``output_bias`` (the output projection has one; it is
+    left to the norm that adds the output), ``head_factor`` (head h's scores are multiplied by a learned number before the
+    cap: its queries are), ``values`` ("own", the default, or "keys": no value projection, a value is its key as projected,
+    before norm and rotation), ``keep_first`` (with a window: the request's first so many keys are read as well, their pages
+    stay), ``unit_sink`` (one is added to the softmax's denominator), ``tensor_names``.
 
-    Every head of q and of k is RMS-normed over its ``dim`` values with one weight vector for all heads, before the
-    rotation.  One kernel sums the projection, adds the biases, norms, rotates and writes the pages; the attention is
+    With ``head_norm`` every head of q and of k is RMS-normed over its ``dim`` values with one weight vector for all heads,
+    before the rotation.  One kernel sums the projection, adds the biases, norms, rotates and writes the pages; the attention is
     the engine's paged attention for changed scores (window, cap and sigmoid weights are arguments of its kernels)."""
 
     graph_safe = True
@@ -235,14 +239,34 @@ class HeadNormRotaryAttention(BranchMixer):
         freq, self.rot_factor = rotary_frequencies(rot) if int(rot["dims"]) else (torch.zeros(0, dtype=torch.float64), 1.0)
         self.freq = freq.to(torch.float64).contiguous().to(ctx.device)
         names = {**_HEAD_NORM_NAMES, **p.get("tensor_names", {})}
-        roles = ("q", "k", "v")
+        self.tied = self._values_kind(p) == "keys"
+        if self.tied and self.dk != self.dv:
+            raise ops.KernelError(f"attention: keys of {self.dk} as values of {self.dv}")
+        self.keep_first = int(p.get("keep_first", 0)) if self.window > 0 else 0
+        if p.get("unit_sink", False) and self.sigmoid:
+            raise ops.KernelError("attention: a sink belongs to the softmax")
+        roles = ("q", "k") if self.tied else ("q", "k", "v")
         self.in_weight = torch.cat([weights[names[role]] for role in roles], dim=0).contiguous()
         self.in_bias = (torch.cat([weights[names[role] + names["bias_suffix"]].to(torch.float32) for role in roles]).contiguous()
                         if p.get("bias", False) else None)
-        self.q_norm = weights[names["q_norm"]].to(torch.float32).contiguous()
-        self.k_norm = weights[names["k_norm"]].to(torch.float32).contiguous()
-        self.head_bias = weights[names["head_bias"]].to(torch.float32).contiguous() if self.sigmoid else None
+        def vector(role, used):
+            return weights[names[role]].to(torch.float32).contiguous() if used else None
+
+        normed = bool(p.get("head_norm", True))
+        self.q_norm, self.k_norm = vector("q_norm", normed), vector("k_norm", normed)
+        self.head_bias = vector("head_bias", self.sigmoid)
+        self.head_factor = vector("head_factor", bool(p.get("head_factor", False)))
+        self.sink = torch.zeros(self.n_q, dtype=torch.float32, device=ctx.device) if p.get("unit_sink", False) else None
+        self.output_bias = (weights[names["out"] + names["bias_suffix"]].to(torch.float32).contiguous()
+                            if p.get("output_bias", False) else None)
         self.out_weight = weights[names["out"]].contiguous()
+
+    @staticmethod
+    def _values_kind(params) -> str:
+        kind = params.get("values", "own")
+        if kind not in ("own", "keys"):
+            raise ops.KernelError(f"attention: values {kind!r} must be own or keys")
+        return kind
 
     @staticmethod
     def _weights_kind(params) -> str:
@@ -256,11 +280,20 @@ class HeadNormRotaryAttention(BranchMixer):
         p = params
         n_q, n_kv, dk, dv = int(p["heads"]), int(p["kv_heads"]), int(p["dim"]), int(p["vdim"])
         names = {**_HEAD_NORM_NAMES, **p.get("tensor_names", {})}
-        out = {names["q"]: TensorSpec((n_q * dk, hidden_size)), names["k"]: TensorSpec((n_kv * dk, hidden_size)),
-               names["v"]: TensorSpec((n_kv * dv, hidden_size)), names["out"]: TensorSpec((hidden_size, n_q * dv)),
-               names["q_norm"]: TensorSpec((dk,), "norm"), names["k_norm"]: TensorSpec((dk,), "norm")}
+        out = {names["q"]: TensorSpec((n_q * dk, hidden_size)), names["k"]: TensorSpec((n_kv * dk, hidden_size))}
+        roles = ("q", "k")
+        if cls._values_kind(p) == "own":
+            out[names["v"]] = TensorSpec((n_kv * dv, hidden_size))
+            roles += ("v",)
+        out[names["out"]] = TensorSpec((hidden_size, n_q * dv))
+        if p.get("head_norm", True):
+            out[names["q_norm"]], out[names["k_norm"]] = TensorSpec((dk,), "norm"), TensorSpec((dk,), "norm")
+        if p.get("head_factor", False):
+            out[names["head_factor"]] = TensorSpec((n_q,), "norm")
+        if p.get("output_bias", False):
+            out[names["out"] + names["bias_suffix"]] = TensorSpec((hidden_size,), "bias")
         if p.get("bias", False):
-            for role in ("q", "k", "v"):
+            for role in roles:
                 out[names[role] + names["bias_suffix"]] = TensorSpec((out[names[role]].shape[0],), "bias")
         if cls._weights_kind(p) == "sigmoid":
             out[names["head_bias"]] = TensorSpec((n_q,), "bias")
@@ -269,7 +302,9 @@ class HeadNormRotaryAttention(BranchMixer):
     @classmethod
     def cache_requirement(cls, params, hidden_size):
         dk, dv = int(params["dim"]), int(params["vdim"])
-        return PagedKV(int(params["kv_heads"]), dk, int(params.get("window", 0)), 0 if dv == dk else dv)
+        window = int(params.get("window", 0))
+        return PagedKV(int(params["kv_heads"]), dk, window, 0 if dv == dk else dv,
+                       int(params.get("keep_first", 0)) if window > 0 else 0)
 
     def _on_tcgen05(self, segment_counts, page_size=None) -> bool:
         """Long prompt portions of the sigmoid-weighted form without a window run on the tcgen05 kernel."""
@@ -288,8 +323,11 @@ class HeadNormRotaryAttention(BranchMixer):
         q = torch.empty((tokens, self.n_q, self.dk), dtype=out.dtype, device=out.device)
         ops.head_norm_rope_kv_write(proj, self.in_bias, self.q_norm, self.k_norm, self.eps, pages.slot_mapping,
                                     step.positions, self.freq, self.rot_factor, q, pages.keys, pages.values, self.n_q,
-                                    self.n_kv, self.dk, self.dv, offset=offset)
-        attended = torch.empty((tokens, self.n_q, self.dv), dtype=out.dtype, device=out.device)
+                                    self.n_kv, self.dk, self.dv, offset=offset, q_factor=self.head_factor,
+                                    values_are_keys=self.tied)
+        straight = scale == 1.0 and out.is_contiguous()      # the attention's own output is the branch's
+        attended = (out.view(tokens, self.n_q, self.dv) if straight
+                    else torch.empty((tokens, self.n_q, self.dv), dtype=out.dtype, device=out.device))
         if (not step.decode_only and step.segments
                 and self._on_tcgen05([segment.count for segment in step.segments], pages.keys.shape[2])):
             ops.attention_sigmoid_tc(q, pages.keys, pages.values, attended, pages.block_tables, step.segment_start,
@@ -298,8 +336,9 @@ class HeadNormRotaryAttention(BranchMixer):
             ops.attention_scored(q, pages.keys, pages.values, attended, pages.block_tables, step.segment_of_token,
                                  step.positions, self.scale, segment_start=step.segment_start,
                                  segment_first_position=step.segment_first_position, window=self.window, cap=self.softcap,
-                                 head_bias=self.head_bias)
-        ops.head_gate_scale(attended, None, out, scale, step.segment_of_token)
+                                 head_bias=self.head_bias, sink=self.sink, keep_first=self.keep_first)
+        if not straight:
+            ops.head_gate_scale(attended, None, out, scale, step.segment_of_token)
 
 
 _SSD_NAMES = {"in": "in", "conv": "conv", "conv_bias": "conv.b", "dt_bias": "dt_bias", "a_log": "A_log", "skip": "D",
@@ -403,6 +442,8 @@ class ParallelMixers(Mixer):
             prefix = branch["prefix"]
             local = {name[len(prefix):]: tensor for name, tensor in weights.items() if name.startswith(prefix)}
             self.branches.append(cls(branch["params"], local, ctx))
+            if self.branches[-1].output_bias is not None:
+                raise ops.KernelError(f"parallel mixers: {branch['kind']!r} with an output bias")
             self.scales.append(float(branch.get("scale", 1.0)))
             self.needs.append(len(cache_needs(cls.cache_requirement(branch["params"], ctx.hidden_size))))
         if not all(branch.graph_safe for branch in self.branches):

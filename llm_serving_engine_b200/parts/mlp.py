@@ -57,3 +57,29 @@ class SwiGLU(FeedForward):
 
 
 register_feed_forward("gated_mlp", SwiGLU)   # the same part under the name that does not say which activation
+
+
+@register_feed_forward("squared_relu_mlp")
+class SquaredReluMLP(FeedForward):
+    """params: ``intermediate_size``, ``tensor_names`` (of the up and down matrices after the part's prefix).
+    y = down(relu(up(x))^2), no gate, no biases; the activation kernel is the ungated experts' (one expert, no weight)."""
+
+    graph_safe = True
+
+    def __init__(self, params, weights, ctx) -> None:
+        super().__init__(params, weights, ctx)
+        self.inter = int(params["intermediate_size"])
+        names = {**_DEFAULT_NAMES, **params.get("tensor_names", {})}
+        self.up_weight, self.down_weight = weights[names["up"]].contiguous(), weights[names["down"]].contiguous()
+
+    @classmethod
+    def expected_tensors(cls, params, hidden_size):
+        inter = int(params["intermediate_size"])
+        names = {**_DEFAULT_NAMES, **params.get("tensor_names", {})}
+        return {names["up"]: TensorSpec((inter, hidden_size)), names["down"]: TensorSpec((hidden_size, inter))}
+
+    def forward(self, x):
+        up = linear_partials(x, self.up_weight)
+        act = torch.empty((x.shape[0], self.inter), dtype=x.dtype, device=x.device)
+        ops.moe_gated_act(up, None, None, act, 1, self.inter, 0, 0.0, 0.0, activation="squared_relu")
+        return linear_partials(act, self.down_weight)

@@ -16,7 +16,8 @@ class RMSNorm(Norm):
     y = (x * rsqrt(mean(x^2) + eps)) * weight, where x is the float32 residual after the pending branch output has
     been added to it.  When the stream keeps several copies of the residual, or scales what a branch adds
     (``ResidualStream``), the same kernel launch mixes the copies, adds the scaled output and reads x as the
-    weighted sum of the copies."""
+    weighted sum of the copies.  A bias that came with the pending output (``stream.delta_bias``) and a norm of this kind
+    that it passes first (``stream.delta_norm``) are applied in the same launch too."""
 
     graph_safe = True
 
@@ -36,7 +37,10 @@ class RMSNorm(Norm):
         hidden = self.weight.shape[0]
         n_rows = stream.residual.shape[0] if rows is None else rows.shape[0]
         out = torch.empty((n_rows, hidden), dtype=self.ctx.dtype, device=stream.residual.device)
-        if stream.plain:
+        if stream.delta_norm is not None or stream.delta_bias is not None:
+            ops.delta_norm_rmsnorm(stream.residual, stream.delta, stream.delta_bias, self._pending_norm(stream), self.weight,
+                                   self.eps, out, rows=rows, write_residual=rows is None)
+        elif stream.plain:
             ops.add_rmsnorm(stream.residual, stream.delta, self.weight, self.eps, out, rows=rows,
                             write_residual=rows is None)
         else:
@@ -44,7 +48,23 @@ class RMSNorm(Norm):
                                        stream.delta_mult, stream.mix, stream.write, stream.read, self.weight,
                                        self.eps, out, rows=rows, write_back=rows is None)
         if rows is None:
-            stream.delta = None
+            stream.delta = stream.delta_bias = stream.delta_norm = None
+        return out
+
+    def _pending_norm(self, stream: ResidualStream):
+        """(weight, eps) of the norm that the pending output passes, or None."""
+        after = stream.delta_norm
+        if not stream.plain or (after is not None and not isinstance(after, RMSNorm)):
+            raise ops.KernelError("rmsnorm: one copy of the residual, a norm of the same kind on a branch's output")
+        return None if after is None or stream.delta is None else (after.weight, after.eps)
+
+    def forward_convolved(self, stream: ResidualStream, conv_weight: torch.Tensor, window: torch.Tensor, step) -> torch.Tensor:
+        """``forward`` over all rows, h, and then h + conv(h): a short causal convolution of h per channel along every
+        request's rows (``conv_weight`` float32 [H, taps]; ``window``: the requests' last taps - 1 rows of h)."""
+        out = torch.empty(stream.residual.shape, dtype=self.ctx.dtype, device=stream.residual.device)
+        stream.residual = ops.conv_norm(stream.residual, stream.delta, stream.delta_bias, self._pending_norm(stream),
+                                        self.weight, self.eps, conv_weight, window, step, out)
+        stream.delta = stream.delta_bias = stream.delta_norm = None
         return out
 
 
