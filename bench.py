@@ -583,7 +583,18 @@ SEBUDRA_SIZES = {
     "w2048": dict(width=2048, heads=16, ff=8192),
     "w4096": dict(width=4096, heads=32, ff=16384),
 }
-DESIGN_SIZES = {"givelix": GIVELIX_SIZES, "fororax": FORORAX_SIZES, "tufevik": TUFEVIK_SIZES, "sebudra": SEBUDRA_SIZES}
+# Kofipel at layer sizes that resemble real models of the kind: four layers, the first two run twice (six layer runs: delta
+# memory, attention, delta memory, attention, delta memory, delta memory); attention heads of 128 in groups of eight over a
+# window of 512 keys and the first sixteen, half of a head rotated; delta memories with heads of 128 key channels and 128
+# values, two heads a key head, four taps, both low-rank maps of rank 64; ungated squared-relu feed-forwards of half as much
+# again as the gated dense one's size, so that a token's feed-forward work is equal; a token input of 64 numbers.  The
+# closest existing model is Sebudra (a windowed attention, a matrix memory with channel decays, squared-relu experts).
+KOFIPEL_SIZES = {
+    "w2048": dict(width=2048, heads=16, ff=8192),
+    "w4096": dict(width=4096, heads=32, ff=16384),
+}
+DESIGN_SIZES = {"givelix": GIVELIX_SIZES, "fororax": FORORAX_SIZES, "tufevik": TUFEVIK_SIZES, "sebudra": SEBUDRA_SIZES,
+                "kofipel": KOFIPEL_SIZES}
 
 
 def fororax_config(width: int, heads: int, ff: int, vocab: int = 32768, context: int = 4096) -> dict:
@@ -630,6 +641,18 @@ def sebudra_config(width: int, heads: int, ff: int, vocab: int = 32768, context:
               {"type": "attention", "mixer": attention, "mlp": dense}, {"type": "gla", "mixer": memory, "mlp": mixture}]
     return {"architecture": "Sebudra", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": 1e-6},
             "embedding": {"scale": 1.0}, "max_position_embeddings": context}
+
+
+def kofipel_config(width: int, heads: int, ff: int, vocab: int = 32768, context: int = 4096) -> dict:
+    mlp = {"kind": "dense", "ff": ff * 3 // 2}
+    memory = {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4, "decay_rank": 64, "gate_rank": 64}
+    attention = {"heads": heads, "kv_heads": max(2, heads // 8), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 40.0,
+                 "mask": {"size": 512, "keep_first": 16}, "rot": {"base": 500000.0, "dims": 64}}
+    layers = [{"type": "channel_delta", "mixer": memory, "mlp": mlp}, {"type": "attention", "mixer": attention, "mlp": mlp},
+              {"type": "channel_delta", "mixer": memory, "mlp": mlp}, {"type": "channel_delta", "mixer": memory, "mlp": mlp}]
+    return {"architecture": "Kofipel", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": 1e-6},
+            "canon": {"taps": 4}, "token_side": {"dim": 64}, "loop": {"start": 0, "stop": 2, "times": 2},
+            "max_position_embeddings": context}
 
 
 def kernel_times(run, repeats: int = 3) -> dict:
@@ -681,11 +704,12 @@ def run_design(args) -> dict:
     fma_tflops = 2 * 128 * torch.cuda.get_device_properties(0).multi_processor_count * 1.965e9 / 1e12   # float32 FMA pipe
     design = args.design
     make_config = {"givelix": givelix_config, "fororax": fororax_config, "tufevik": tufevik_config,
-                   "sebudra": sebudra_config}[design]
+                   "sebudra": sebudra_config, "kofipel": kofipel_config}[design]
     rooflines = {"givelix": design_rooflines, "fororax": fororax_rooflines, "tufevik": tufevik_rooflines,
-                 "sebudra": sebudra_rooflines}[design]
+                 "sebudra": sebudra_rooflines, "kofipel": kofipel_rooflines}[design]
     # designs that are set beside another model than Qwen2 as well: (label, config maker)
-    beside = {"sebudra": [("tufevik_equal_size", tufevik_config)]}.get(design, [])
+    beside = {"sebudra": [("tufevik_equal_size", tufevik_config)],
+              "kofipel": [("sebudra_equal_size", sebudra_config)]}.get(design, [])
     batch, out = args.batch, {"design": design, "peaks": dict(peak, fp32_fma_tflops=round(fma_tflops, 1)), "sizes": {}}
     names = [args.design_size] if args.design_size else list(DESIGN_SIZES[design])
     with ClockSampler() as clocks:
@@ -1019,6 +1043,79 @@ def sebudra_rooflines(shape: dict, entry: dict, batch: int, peak: dict, fma_tflo
     return out
 
 
+
+def kofipel_rooflines(shape: dict, entry: dict, batch: int, peak: dict, fma_tflops: float) -> dict:
+    """As :func:`design_rooflines`, for Kofipel beside Sebudra (the closest existing model) at equal size: every kind of
+    kernel that is not a plain product, each against the slower of the bytes it must move and the operations it must do
+    (scans and row-wise kernels against the float32 FMA pipe, attention against the measured bfloat16 tensor throughput).
+    The delta memory's work is counted row by row: decay, read, write and read-out of the state, 3.5 multiply-adds an
+    element; Sebudra's scans as its own table counts them (two passes of update and read-out)."""
+    heads, width, tokens = shape["heads"], shape["width"], PROMPT
+    kv_heads = max(2, heads // 8)
+    config = kofipel_config(**shape)
+    memory, attention = config["layers"][0]["mixer"], config["layers"][1]["mixer"]
+    groups, dim, vdim = memory["kv_heads"], memory["dim"], memory["vdim"]
+    channels = 2 * groups * dim + heads * vdim
+    low, ff, side = memory["decay_rank"] + memory["gate_rank"], config["layers"][0]["mlp"]["ff"], config["token_side"]["dim"]
+    window = attention["mask"]["size"] + attention["mask"]["keep_first"]
+    bandwidth, tensor, fma = peak["hbm_gbs"] * 1e9, peak["bf16_tflops"] * 1e12, fma_tflops * 1e12
+
+    def frac(kernels: dict, keys, launches_of_work: float, bytes_each: float, flops_each: float, pipe: float, without=()):
+        keys = (keys,) if isinstance(keys, str) else keys
+        found = [(name, value) for name, value in kernels.items()
+                 if any(key in name for key in keys) and not any(key in name for key in without)]
+        if not found:
+            return None
+        us = sum(value["us"] for _, value in found)
+        count = sum(value["launches"] for _, value in found)
+        bound = max(bytes_each / bandwidth, flops_each / pipe) * launches_of_work
+        return {"us": round(us, 1), "launches": count, "bound_us": round(bound * 1e6, 2), "frac": round(bound * 1e6 / us, 4)}
+
+    k = entry["kofipel"]
+    memories, attentions, runs = 4, 2, 6
+    state = heads * dim * vdim
+    pairs = tokens * window - window * (window - 1) / 2
+    qk_row = (heads + 2 * kv_heads) * 128
+    out = {"prefill": {}, "decode": {}}
+    p = k["prefill_kernels"]
+    scan_bytes = tokens * 4 * (2 * groups * dim + heads * (vdim + dim + 1) + heads * vdim)
+    out["prefill"]["kofipel delta memory scans"] = frac(p, ("delta_scan", "delta_chunk"), memories, scan_bytes, tokens * state * 7, fma)
+    out["prefill"]["kofipel convolutions, unit vectors, write strengths"] = frac(
+        p, ("delta_prepare", "short_conv"), memories, tokens * (channels + heads + low) * (2 + 4), 0, fma)
+    out["prefill"]["kofipel gated norms in parts"] = frac(p, "gated_group_rmsnorm", memories, tokens * heads * vdim * (4 + 4 + 2), 0, fma)
+    out["prefill"]["kofipel attention (2 windowed layers that keep the first keys)"] = frac(
+        p, ("attention_scored",), attentions, tokens * qk_row * 2 * 2, 4 * pairs * heads * 128, tensor)
+    out["prefill"]["kofipel rotation + page write"] = frac(p, "head_norm_rope", attentions, tokens * qk_row * (2 + 2), 0, fma)
+    out["prefill"]["kofipel sum, norm, convolution of a sublayer's input"] = frac(
+        p, "conv_norm", 2 * runs, tokens * width * (4 * 2 + 2 + 2), 0, fma)
+    out["prefill"]["kofipel squared relu"] = frac(p, "moe_gated_act", runs, tokens * ff * 4, 0, fma)
+    out["prefill"]["kofipel token input (sum + copy, gate)"] = frac(
+        p, ("residual_settle", "token_gate"), runs, tokens * width * (4 * 2 + 2 + 2) + tokens * side * 6, 0, fma)
+    d = k["decode_kernels"]
+    out["decode"]["kofipel delta memory scans"] = frac(d, ("delta_scan", "delta_chunk"), memories, batch * state * 4 * 2, batch * state * 7, fma)
+    out["decode"]["kofipel convolutions, unit vectors, gated norms"] = frac(
+        d, ("delta_prepare", "gated_group_rmsnorm"), memories, batch * (channels * 4 * 8 + heads * vdim * 10), 0, fma)
+    out["decode"]["kofipel attention (2 windowed layers, chunks + merge)"] = frac(
+        d, ("attention_scored",), attentions, batch * window * 2 * kv_heads * 128 * 2, 4 * batch * window * heads * 128, tensor)
+    out["decode"]["kofipel rotation + page write"] = frac(d, "head_norm_rope", attentions, batch * qk_row * 4 * 5, 0, fma)
+    out["decode"]["kofipel sum, norm, convolution of a sublayer's input"] = frac(
+        d, "conv_norm", 2 * runs, batch * width * (4 * 2 + 4 * 4 + 2 + 3 * 4 * 2) + width * 5 * 4, 0, fma)
+    out["decode"]["kofipel squared relu"] = frac(d, "moe_gated_act", runs, batch * ff * (4 + 2), 0, fma)
+    out["decode"]["kofipel token input (sum + copy, gate)"] = frac(
+        d, ("residual_settle", "token_gate"), runs, batch * width * (4 * 2 + 4 * 4 + 2), 0, fma)
+    # Sebudra's own table, with its closest model left out
+    other = sebudra_rooflines(shape, {"sebudra": entry["sebudra_equal_size"],
+                                      "tufevik_equal_size": {"prefill_kernels": {}, "decode_kernels": {}}}, batch, peak, fma_tflops)
+    for step in ("prefill", "decode"):
+        out[step] = {key: value for key, value in out[step].items() if value is not None}
+        out[step].update({key: value for key, value in other[step].items() if value is not None})
+    # the windowed layers alone, the like of this design's attention: the tensor-core kernel of a prompt
+    s = entry["sebudra_equal_size"]
+    out["prefill"]["sebudra windowed attention alone (2 layers)"] = frac(
+        s["prefill_kernels"], "attention_scored", 2, tokens * qk_row * 2 * 2, 4 * (tokens * 512 - 512 * 511 / 2) * heads * 128, tensor)
+    return out
+
+
 def bench_config(config: dict, layers: int, batch: int) -> dict:
     """The ``config`` of the bench line: every size, flat; the same dict in both arms."""
     return {
@@ -1339,7 +1436,7 @@ def main() -> int:
                         help="with --only: the true float32 path instead of the serving precision")
     parser.add_argument("--quick", action="store_true", help="the headline, its points and the end-to-end number only "
                                                              "(no other model sizes, no float32 point, no kernel table)")
-    parser.add_argument("--design", choices=("givelix", "fororax", "tufevik", "sebudra"), default=None,
+    parser.add_argument("--design", choices=("givelix", "fororax", "tufevik", "sebudra", "kofipel"), default=None,
                         help="instead of the default workload: the named design at layer sizes of real models beside the "
                              "Qwen2 model of equal size (prefill and decode throughput, kernel times, rooflines)")
     parser.add_argument("--design-size", choices=tuple(sorted({name for sizes in DESIGN_SIZES.values() for name in sizes})),

@@ -7,7 +7,8 @@
 //       convolution per channel and SiLU; each head of q and k becomes a unit vector (x / sqrt(sum x^2 + 1e-6)), q times
 //       q_scale; beta = sigmoid of its column; the low-rank columns (inputs of the decays' and the gate's second product)
 //       are rounded into the compute dtype.
-//   lse_delta_scan:    the recurrence row by row over every request's rows, from and into its state slot; the keep
+//   lse_delta_scan:    the recurrence row by row over every request's rows, from and into its state slot (few rows, single
+//       decoded tokens; delta_memory_chunks.cu has the form for many rows of a request); the keep
 //       factors exp(-exp(a_log) softplus(z + dt_bias)) are worked out from the decays' product while a tile is staged.
 #include "common.cuh"
 

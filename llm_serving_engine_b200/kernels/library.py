@@ -157,6 +157,11 @@ _SIGNATURES = {
                           c_int, c_int, c_float, c_int, c_int, c_int, c_void_p],
     "lse_delta_scan": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_longlong, c_void_p, c_void_p,
                        c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "lse_delta_chunk_rows": [],
+    "lse_delta_chunk_floats": [c_int, c_int],
+    "lse_delta_chunk_scan": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_longlong, c_void_p, c_void_p,
+                             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                             c_int, c_void_p],
     "lse_attention_scored_windowed": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p,
                                       c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                       c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p,
@@ -228,7 +233,7 @@ CHECK_READERS = ("lse_check_elementwise", "lse_check_attention_generic", "lse_ch
                  "lse_check_linear_attention_vector", "lse_check_attention_latent",
                  "lse_check_attention_latent_mma", "lse_check_rowwise_postnorm", "lse_check_attention_scored",
                  "lse_check_attention_scored_mma", "lse_check_mlstm", "lse_check_short_conv", "lse_check_selective_scan", "lse_check_conv_norm",
-                 "lse_check_delta_memory")
+                 "lse_check_delta_memory", "lse_check_delta_memory_chunks")
 CHECK_KINDS = {1: "token id", 2: "cache slot", 3: "block-table entry", 4: "segment number", 5: "row index"}
 
 

@@ -1607,13 +1607,18 @@ def delta_prepare(proj: torch.Tensor, conv_weight: torch.Tensor, state: torch.Te
     return q, k, v, beta
 
 
+DELTA_CHUNKED_ABOVE = 16      # rows of a request in a step beyond which its rows are worked on in chunks
+
+
 def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Tensor, z: torch.Tensor, dt_bias: torch.Tensor,
                a_log: torch.Tensor, state: torch.Tensor, segment_start: torch.Tensor, segment_slot: torch.Tensor,
-               out: torch.Tensor, heads: int, groups: int, dim: int, vdim: int) -> torch.Tensor:
+               out: torch.Tensor, heads: int, groups: int, dim: int, vdim: int, chunked_above: int | None = None) -> torch.Tensor:
     """S <- diag(keep) S;  u = beta (v - S^T k);  S <- S + k u^T;  out = S^T q, over the rows of every request in order, from
     and into ``state`` float32 [slots, heads, dim, vdim]; keep = exp(-exp(a_log_h) softplus(z + dt_bias)) per head and key
     channel, z float32 columns 0 .. heads * dim of a projection (rows or partial sums).  Other arguments as
-    :func:`delta_prepare` returns them; out float32 [T, heads * vdim]."""
+    :func:`delta_prepare` returns them; out float32 [T, heads * vdim].  Requests of more than ``chunked_above`` rows (default
+    ``DELTA_CHUNKED_ABOVE``; a number beyond the step's rows: none) take the chunked form, the others go row by row; the two
+    differ by rounding only."""
     _need_cuda(q, k, v, beta, z, dt_bias, a_log, state, segment_start, segment_slot, out)
     z, code, z_partials, z_stride, z_ld = _projection(z)
     tokens = out.shape[0]
@@ -1622,8 +1627,19 @@ def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Te
     assert out.dtype == torch.float32 and out.is_contiguous() and out.shape == (tokens, heads * vdim)
     segments = segment_slot.shape[0]
     assert segment_start.dtype == segment_slot.dtype == torch.int32 and segment_start.shape[0] == segments + 1
-    check(library.load().lse_delta_scan(
-        q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(), z.data_ptr(), z_partials, z_stride, z_ld, dt_bias.data_ptr(),
-        a_log.data_ptr(), state.data_ptr(), segment_start.data_ptr(), segment_slot.data_ptr(), out.data_ptr(), segments, heads,
-        groups, dim, vdim, state.shape[0], 0, _stream()), "delta_scan")
+    lib = library.load()
+    above = DELTA_CHUNKED_ABOVE if chunked_above is None else int(chunked_above)
+    chunked = tokens > above      # by the number of rows alone: a captured step is replayed with other portions
+    inputs = (q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(), z.data_ptr(), z_partials, z_stride, z_ld,
+              dt_bias.data_ptr(), a_log.data_ptr(), state.data_ptr(), segment_start.data_ptr(), segment_slot.data_ptr(),
+              out.data_ptr())
+    if chunked:
+        rows = int(lib.lse_delta_chunk_rows())
+        max_chunks = tokens // rows + min(segments, tokens // (above + 1))    # a request in chunks has more than `above` rows
+        buffer = torch.empty(max_chunks * heads * int(lib.lse_delta_chunk_floats(dim, vdim)), dtype=torch.float32, device=out.device)
+        check(lib.lse_delta_chunk_scan(*inputs, buffer.data_ptr(), max_chunks, segments, heads, groups, dim, vdim, state.shape[0],
+                                       above, _stream()), "delta_chunk_scan")
+    if above > 0 or not chunked:
+        check(lib.lse_delta_scan(*inputs, segments, heads, groups, dim, vdim, state.shape[0], above if chunked else 0, _stream()),
+              "delta_scan")
     return out
