@@ -9,11 +9,9 @@
 // taps - 1 rows of h are kept, in float32, in its state slot ([slots, taps - 1, hidden], oldest first), so that a step
 // can start anywhere.
 //
-//   lse_conv_norm:         the whole of it for 1 to 4 taps and widths that are multiples of four.  x goes to a residual
-//       tensor of its own (residual_out): a block works its rows' predecessors out again from residual and delta,
-//       so those must stay as they were.  A block walks a few rows with the last taps - 1 rows of h in registers.
-//   lse_conv_norm_state:   moves the windows on after a step with portions (a block per request works the last
-//       rows of h out from residual_out).  Steps of single tokens move them on inside lse_conv_norm.
+//   lse_conv_norm:         the whole of it for 1 to 4 taps and widths that are multiples of four up to 8,192.  When every
+//       request brings one token: one launch, a block per row, which moves its window on.  Else three: the sum with
+//       the rows' factors 1 / rms, the norm with the convolution (x is read once more, from L2), the windows.
 //   lse_delta_norm_rmsnorm: x and h without a convolution, any width, with gathered rows (a model's last norm) and as the
 //       first half of convolutions that lse_conv_norm was not built for.
 //   lse_residual_settle:   residual += d in place, and the sum rounded into the compute dtype.
@@ -23,8 +21,6 @@
 LSE_CHECK_DEFINE(lse_check_conv_norm)
 
 namespace {
-constexpr int CN_GROUP = 4;       // rows whose sums of squares are reduced together
-
 template <typename T> __device__ __forceinline__ void cn_load4(const T* p, float (&v)[4]);
 template <> __device__ __forceinline__ void cn_load4<float>(const float* p, float (&v)[4]) {
   const float4 a = *reinterpret_cast<const float4*>(p);
@@ -47,187 +43,261 @@ template <> __device__ __forceinline__ void cn_store4<__nv_bfloat16>(__nv_bfloat
   *reinterpret_cast<uint2*>(p) = raw;
 }
 
-// N sums over the block at once (lanes by butterfly, then warps in index order); scratch holds N * 32 floats.
-template <int N>
-__device__ __forceinline__ void block_sums(float (&v)[N], float* scratch) {
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
+// d and the sum: x (this thread's pieces threadIdx.x, threadIdx.x + blockDim.x, ... of four channels of one row) becomes
+// residual + d; returns the sum of squares over the row.  Every load is issued before any is used.
+template <typename TD, int C>
+__device__ __forceinline__ float cn_sum_row(const float* __restrict__ res, const TD* __restrict__ del, int n_partials,
+                                            long long partial_stride, const float* __restrict__ bias,
+                                            const float* __restrict__ delta_weight, float delta_eps, int hidden,
+                                            float* scratch, float (&x)[C][4]) {
+  const int pieces = hidden / 4;
+  float r[C][4], dw[C][4], sq = 0.f;
 #pragma unroll
-  for (int n = 0; n < N; ++n) v[n] = warp_sum(v[n]);
-  __syncthreads();
-  if (lane == 0) {
+  for (int c = 0; c < C; ++c) {
+    const int piece = threadIdx.x + c * blockDim.x;
 #pragma unroll
-    for (int n = 0; n < N; ++n) scratch[n * 32 + warp] = v[n];
+    for (int e = 0; e < 4; ++e) x[c][e] = r[c][e] = dw[c][e] = 0.f;
+    if (piece < pieces) {
+      cn_load4<float>(res + piece * 4, r[c]);
+      if (delta_weight) cn_load4<float>(delta_weight + piece * 4, dw[c]);
+      if (del) {
+        const TD* src = del + piece * 4;
+        int p = 0;
+        for (; p + 8 <= n_partials; p += 8) {     // eight loads in flight, added in index order
+          float a[8][4];
+#pragma unroll
+          for (int k = 0; k < 8; ++k) cn_load4<TD>(src + (size_t)(p + k) * partial_stride, a[k]);
+#pragma unroll
+          for (int k = 0; k < 8; ++k)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) x[c][e] += a[k][e];
+        }
+        for (; p + 2 <= n_partials; p += 2) {
+          float a[2][4];
+#pragma unroll
+          for (int k = 0; k < 2; ++k) cn_load4<TD>(src + (size_t)(p + k) * partial_stride, a[k]);
+#pragma unroll
+          for (int k = 0; k < 2; ++k)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) x[c][e] += a[k][e];
+        }
+        for (; p < n_partials; ++p) {
+          float a[4];
+          cn_load4<TD>(src + (size_t)p * partial_stride, a);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) x[c][e] += a[e];
+        }
+        if (bias) {
+          float b[4];
+          cn_load4<float>(bias + piece * 4, b);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) x[c][e] += b[e];
+        }
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) sq = fmaf(x[c][e], x[c][e], sq);
   }
-  __syncthreads();
+  if (delta_weight && del) {                      // the pending output passes a norm of its own
+    const float inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)hidden + delta_eps);
 #pragma unroll
-  for (int n = 0; n < N; ++n) {
-    float total = 0.f;
-    for (int w = 0; w < nwarps; ++w) total += scratch[n * 32 + w];
-    v[n] = total;
+    for (int c = 0; c < C; ++c)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[c][e] = (x[c][e] * inv) * dw[c][e];
   }
+  sq = 0.f;
+#pragma unroll
+  for (int c = 0; c < C; ++c)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      x[c][e] += r[c][e];
+      sq = fmaf(x[c][e], x[c][e], sq);
+    }
+  return block_sum(sq, scratch);
 }
 
-// A thread owns pieces threadIdx.x, threadIdx.x + blockDim.x, ... (C of them) of four neighbouring channels.
+// Every request brings one row: a block per row, which finds its predecessors in the window and moves it on.
 template <typename TD, typename TO, int TAPS, int C>
 __global__ void __launch_bounds__(512)
-conv_norm_kernel(const float* __restrict__ residual, float* __restrict__ residual_out, const TD* __restrict__ delta,
-                 int n_partials, long long partial_stride, const float* __restrict__ bias,
-                 const float* __restrict__ delta_weight, float delta_eps, const float* __restrict__ weight, float eps,
-                 const float* __restrict__ conv_weight, float* __restrict__ state,
-                 const int* __restrict__ segment_of_token, const int* __restrict__ segment_start,
-                 const int* __restrict__ segment_slot, TO* __restrict__ out, int tokens, int rows_per_block, int hidden,
-                 int move_windows, int num_slots, int num_segments) {
+conv_norm_single_kernel(float* __restrict__ residual, const TD* __restrict__ delta, int n_partials, long long partial_stride,
+                        const float* __restrict__ bias, const float* __restrict__ delta_weight, float delta_eps,
+                        const float* __restrict__ weight, float eps, const float* __restrict__ conv_weight,
+                        float* __restrict__ state, const int* __restrict__ segment_of_token,
+                        const int* __restrict__ segment_slot, TO* __restrict__ out, int hidden, int num_slots,
+                        int num_segments) {
   constexpr int BACK = TAPS - 1, HELD = BACK > 0 ? BACK : 1;
-  __shared__ float scratch[CN_GROUP * 32];
+  __shared__ float scratch[32];
   pdl_launch_dependents();
   const int pieces = hidden / 4;
-  float nw[C][4], cw[TAPS][C][4];
+  float nw[C][4], cw[C][4][TAPS];
 #pragma unroll
   for (int c = 0; c < C; ++c) {      // the weights do not depend on earlier kernels
     const int piece = threadIdx.x + c * blockDim.x;
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      nw[c][e] = piece < pieces ? weight[piece * 4 + e] : 0.f;
+      nw[c][e] = 0.f;
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) cw[j][c][e] = piece < pieces ? conv_weight[(size_t)(piece * 4 + e) * TAPS + j] : 0.f;
+      for (int j = 0; j < TAPS; ++j) cw[c][e][j] = 0.f;
+    }
+    if (piece < pieces) {
+      cn_load4<float>(weight + piece * 4, nw[c]);
+      float* flat = &cw[c][0][0];    // four channels' taps lie one after the other
+#pragma unroll
+      for (int k = 0; k < TAPS; ++k) {
+        float a[4];
+        cn_load4<float>(conv_weight + (size_t)piece * 4 * TAPS + 4 * k, a);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) flat[4 * k + e] = a[e];
+      }
     }
   }
   pdl_wait();
-  const int first = blockIdx.x * rows_per_block, end = min(tokens, first + rows_per_block);
-  int start = first;
-  if (BACK > 0) {                    // the rows before the block's own that belong to the same request
-    const int seg = segment_of_token[first];
-    if (seg >= 0) start = max(segment_start[LSE_CHECKED(seg, 0, num_segments, 0, LSE_CHECK_SEGMENT)], first - BACK);
-  }
-  float before[HELD][C][4];          // before[i]: h of the row BACK - i rows back
+  const int row = blockIdx.x;
+  int seg = segment_of_token[row];
+  if (seg < 0) return;
+  seg = LSE_CHECKED(seg, 0, num_segments, 0, LSE_CHECK_SEGMENT);
+  float* window = BACK > 0 ? state + (size_t)LSE_CHECKED(segment_slot[seg], 0, num_slots, 0, LSE_CHECK_ROW) * BACK * hidden : nullptr;
+  float before[HELD][C][4];
 #pragma unroll
-  for (int i = 0; i < HELD; ++i)
+  for (int i = 0; i < BACK; ++i)
 #pragma unroll
-    for (int c = 0; c < C; ++c)
+    for (int c = 0; c < C; ++c) {
+      const int piece = threadIdx.x + c * blockDim.x;
 #pragma unroll
       for (int e = 0; e < 4; ++e) before[i][c][e] = 0.f;
-  int held = -1;                     // the request that `before` belongs to
-  for (int base = start; base < end; base += CN_GROUP) {
-    float x[CN_GROUP][C][4], sums[CN_GROUP];
-#pragma unroll
-    for (int g = 0; g < CN_GROUP; ++g) {
-      sums[g] = 0.f;
-#pragma unroll
-      for (int c = 0; c < C; ++c) {
-        const int piece = threadIdx.x + c * blockDim.x;
-#pragma unroll
-        for (int e = 0; e < 4; ++e) x[g][c][e] = 0.f;
-        if (base + g < end && piece < pieces && delta) {
-          const TD* src = delta + (size_t)(base + g) * hidden + piece * 4;
-          int p = 0;
-          for (; p + 4 <= n_partials; p += 4) {     // four loads in flight, added in index order
-            float a[4][4];
-#pragma unroll
-            for (int k = 0; k < 4; ++k) cn_load4<TD>(src + (size_t)(p + k) * partial_stride, a[k]);
-#pragma unroll
-            for (int k = 0; k < 4; ++k)
-#pragma unroll
-              for (int e = 0; e < 4; ++e) x[g][c][e] += a[k][e];
-          }
-          for (; p < n_partials; ++p) {
-            float a[4];
-            cn_load4<TD>(src + (size_t)p * partial_stride, a);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) x[g][c][e] += a[e];
-          }
-          if (bias) {
-#pragma unroll
-            for (int e = 0; e < 4; ++e) x[g][c][e] += bias[piece * 4 + e];
-          }
-        }
-#pragma unroll
-        for (int e = 0; e < 4; ++e) sums[g] = fmaf(x[g][c][e], x[g][c][e], sums[g]);
-      }
+      if (piece < pieces) cn_load4<float>(window + (size_t)i * hidden + piece * 4, before[i][c]);
     }
-    if (delta_weight) {              // the pending output passes a norm of its own
-      block_sums<CN_GROUP>(sums, scratch);
+  float* res = residual + (size_t)row * hidden;
+  float x[C][4];
+  const float sq = cn_sum_row<TD, C>(res, delta ? delta + (size_t)row * hidden : nullptr, n_partials, partial_stride, bias,
+                                     delta_weight, delta_eps, hidden, scratch, x);
+  const float inv = 1.0f / sqrtf(sq / (float)hidden + eps);
 #pragma unroll
-      for (int c = 0; c < C; ++c) {
-        const int piece = threadIdx.x + c * blockDim.x;
-        float dw[4] = {0.f, 0.f, 0.f, 0.f};
-        if (piece < pieces) cn_load4<float>(delta_weight + piece * 4, dw);
+  for (int c = 0; c < C; ++c) {
+    const int piece = threadIdx.x + c * blockDim.x;
+    if (piece < pieces) {
+      float h[4], y[4];
 #pragma unroll
-        for (int g = 0; g < CN_GROUP; ++g) {
-          const float inv = 1.0f / sqrtf(sums[g] / (float)hidden + delta_eps);
+      for (int e = 0; e < 4; ++e) {
+        h[e] = (x[c][e] * inv) * nw[c][e];
+        float sum = 0.f;
 #pragma unroll
-          for (int e = 0; e < 4; ++e) x[g][c][e] = (x[g][c][e] * inv) * dw[e];
-        }
+        for (int j = 0; j < BACK; ++j) sum = fmaf(cw[c][e][j], before[j][c][e], sum);
+        y[e] = h[e] + fmaf(cw[c][e][TAPS - 1], h[e], sum);
       }
+      cn_store4<TO>(out + (size_t)row * hidden + piece * 4, y);
+      cn_store4<float>(res + piece * 4, x[c]);
+#pragma unroll
+      for (int i = 0; i + 1 < BACK; ++i) cn_store4<float>(window + (size_t)i * hidden + piece * 4, before[i + 1][c]);
+      if (BACK > 0) cn_store4<float>(window + (size_t)(BACK - 1) * hidden + piece * 4, h);
+    }
+  }
+}
+
+// Many rows, first half: x in place, and every row's factor 1 / sqrt(mean(x^2) + eps).  A block per row.
+template <typename TD, int C>
+__global__ void __launch_bounds__(256)
+conv_norm_rows_kernel(float* __restrict__ residual, const TD* __restrict__ delta, int n_partials, long long partial_stride,
+                      const float* __restrict__ bias, const float* __restrict__ delta_weight, float delta_eps, float eps,
+                      float* __restrict__ factor, int hidden) {
+  __shared__ float scratch[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x, pieces = hidden / 4;
+  float* res = residual + (size_t)row * hidden;
+  float x[C][4];
+  const float sq = cn_sum_row<TD, C>(res, delta ? delta + (size_t)row * hidden : nullptr, n_partials, partial_stride, bias,
+                                     delta_weight, delta_eps, hidden, scratch, x);
+  if (delta) {
+#pragma unroll
+    for (int c = 0; c < C; ++c) {
+      const int piece = threadIdx.x + c * blockDim.x;
+      if (piece < pieces) cn_store4<float>(res + piece * 4, x[c]);
+    }
+  }
+  if (threadIdx.x == 0) factor[row] = 1.0f / sqrtf(sq / (float)hidden + eps);
+}
+
+// Second half: h = x * factor * weight and h + conv(h).  A thread owns four channels and walks CN_ROWS rows with the last
+// taps - 1 rows of h in registers; the rows of x are fetched CN_AHEAD at a time.  grid (row tiles, channel tiles)
+constexpr int CN_ROWS = 16, CN_AHEAD = 4;
+template <typename TO, int TAPS>
+__global__ void __launch_bounds__(128)
+conv_norm_apply_kernel(const float* __restrict__ x, const float* __restrict__ factor, const float* __restrict__ weight,
+                       const float* __restrict__ conv_weight, const float* __restrict__ state,
+                       const int* __restrict__ segment_of_token, const int* __restrict__ segment_start,
+                       const int* __restrict__ segment_slot, TO* __restrict__ out, int tokens, int hidden, int num_slots,
+                       int num_segments) {
+  constexpr int BACK = TAPS - 1, HELD = BACK > 0 ? BACK : 1;
+  pdl_launch_dependents();
+  const int piece = blockIdx.y * blockDim.x + threadIdx.x;
+  if (piece * 4 >= hidden) return;
+  float nw[4], cw[4][TAPS];
+  cn_load4<float>(weight + piece * 4, nw);
+  float* flat = &cw[0][0];
+#pragma unroll
+  for (int k = 0; k < TAPS; ++k) {
+    float a[4];
+    cn_load4<float>(conv_weight + (size_t)piece * 4 * TAPS + 4 * k, a);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) flat[4 * k + e] = a[e];
+  }
+  pdl_wait();
+  const int first = blockIdx.x * CN_ROWS, end = min(tokens, first + CN_ROWS);
+  auto normed = [&](int row, float (&h)[4]) {
+    float v[4];
+    cn_load4<float>(x + (size_t)row * hidden + piece * 4, v);
+    const float f = factor[row];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) h[e] = (v[e] * f) * nw[e];
+  };
+  float before[HELD][4];
+  int held = -1;
+  for (int base = first; base < end; base += CN_AHEAD) {
+    float h[CN_AHEAD][4];
+    int segs[CN_AHEAD];
+#pragma unroll
+    for (int g = 0; g < CN_AHEAD; ++g) {
+      const int row = min(base + g, end - 1);
+      segs[g] = segment_of_token[row];
+      normed(row, h[g]);
     }
 #pragma unroll
-    for (int g = 0; g < CN_GROUP; ++g) {
-      sums[g] = 0.f;
-#pragma unroll
-      for (int c = 0; c < C; ++c) {
-        const int piece = threadIdx.x + c * blockDim.x;
-        if (base + g < end && piece < pieces) {
-          float r[4];
-          cn_load4<float>(residual + (size_t)(base + g) * hidden + piece * 4, r);
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            x[g][c][e] += r[e];
-            sums[g] = fmaf(x[g][c][e], x[g][c][e], sums[g]);
-          }
-        }
-      }
-    }
-    block_sums<CN_GROUP>(sums, scratch);
-#pragma unroll
-    for (int g = 0; g < CN_GROUP; ++g) {
+    for (int g = 0; g < CN_AHEAD; ++g) {
       const int row = base + g;
       if (row < end) {
-        int seg = segment_of_token[row];
+        int seg = segs[g];
         if (seg < 0) {
           held = -1;
         } else {
           seg = LSE_CHECKED(seg, 0, num_segments, 0, LSE_CHECK_SEGMENT);
-          float* window = BACK > 0 ? state + (size_t)LSE_CHECKED(segment_slot[seg], 0, num_slots, 0, LSE_CHECK_ROW) * BACK * hidden : nullptr;
-          if (BACK > 0 && seg != held) {
-            if (row == segment_start[seg]) {    // else the block's first, predecessor, rows fill it
+          if (BACK > 0 && seg != held) {        // the first row of a request in this tile
+            const float* window = state + (size_t)LSE_CHECKED(segment_slot[seg], 0, num_slots, 0, LSE_CHECK_ROW) * BACK * hidden;
+            const int l = row - segment_start[seg];
 #pragma unroll
-              for (int i = 0; i < BACK; ++i)
-#pragma unroll
-                for (int c = 0; c < C; ++c) {
-                  const int piece = threadIdx.x + c * blockDim.x;
-                  if (piece < pieces) cn_load4<float>(window + (size_t)i * hidden + piece * 4, before[i][c]);
-                }
+            for (int i = 0; i < BACK; ++i) {
+              const int back = BACK - i;
+              if (l - back >= 0) normed(row - back, before[i]);
+              else cn_load4<float>(window + (size_t)(BACK + l - back) * hidden + piece * 4, before[i]);
             }
             held = seg;
           }
-          const float inv = 1.0f / sqrtf(sums[g] / (float)hidden + eps);
+          float y[4];
 #pragma unroll
-          for (int c = 0; c < C; ++c) {
-            const int piece = threadIdx.x + c * blockDim.x;
-            float h[4], y[4];
+          for (int e = 0; e < 4; ++e) {
+            float sum = 0.f;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              h[e] = (x[g][c][e] * inv) * nw[c][e];
-              float sum = 0.f;
+            for (int j = 0; j < BACK; ++j) sum = fmaf(cw[e][j], before[j][e], sum);
+            y[e] = h[g][e] + fmaf(cw[e][TAPS - 1], h[g][e], sum);
+          }
+          cn_store4<TO>(out + (size_t)row * hidden + piece * 4, y);
+          if (BACK > 0) {
 #pragma unroll
-              for (int j = 0; j < BACK; ++j) sum = fmaf(cw[j][c][e], before[j][c][e], sum);
-              y[e] = h[e] + fmaf(cw[TAPS - 1][c][e], h[e], sum);
-            }
-            if (BACK > 0) {
+            for (int i = 0; i + 1 < BACK; ++i)
 #pragma unroll
-              for (int i = 0; i + 1 < BACK; ++i)
+              for (int e = 0; e < 4; ++e) before[i][e] = before[i + 1][e];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) before[i][c][e] = before[i + 1][c][e];
-#pragma unroll
-              for (int e = 0; e < 4; ++e) before[HELD - 1][c][e] = h[e];
-            }
-            if (row >= first && piece < pieces) {
-              cn_store4<float>(residual_out + (size_t)row * hidden + piece * 4, x[g][c]);
-              cn_store4<TO>(out + (size_t)row * hidden + piece * 4, y);
-              if (BACK > 0 && move_windows) {
-#pragma unroll
-                for (int i = 0; i < BACK; ++i) cn_store4<float>(window + (size_t)i * hidden + piece * 4, before[i][c]);
-              }
-            }
+            for (int e = 0; e < 4; ++e) before[HELD - 1][e] = h[g][e];
           }
         }
       }
@@ -235,31 +305,34 @@ conv_norm_kernel(const float* __restrict__ residual, float* __restrict__ residua
   }
 }
 
-// The windows after a step: entry i holds h at the request's row count - (taps - 1) + i of this step, or moves up from
-// behind (in ascending order an entry only reads entries behind it).  A block per request; x: residual_out.
-__global__ void __launch_bounds__(256)
-conv_norm_state_kernel(const float* __restrict__ x, const float* __restrict__ weight, float eps, float* __restrict__ state,
-                       const int* __restrict__ segment_start, const int* __restrict__ segment_slot, int hidden, int taps,
-                       int num_slots) {
-  __shared__ float scratch[32];
+// The windows after a step of many rows: entry i holds h at the request's row count - (taps - 1) + i of this step, or moves up
+// from behind (in ascending order an entry only reads entries behind it).  grid (requests, channel tiles)
+__global__ void __launch_bounds__(128)
+conv_norm_state_kernel(const float* __restrict__ x, const float* __restrict__ factor, const float* __restrict__ weight,
+                       float* __restrict__ state, const int* __restrict__ segment_start,
+                       const int* __restrict__ segment_slot, int hidden, int taps, int num_slots) {
   pdl_launch_dependents();
   pdl_wait();
   const int seg = blockIdx.x;
   const int row0 = segment_start[seg], count = segment_start[seg + 1] - row0;
-  if (count <= 0) return;
-  float* window = state + (size_t)LSE_CHECKED(segment_slot[seg], 0, num_slots, 0, LSE_CHECK_ROW) * (taps - 1) * hidden;
+  const int piece = blockIdx.y * blockDim.x + threadIdx.x;
+  if (count <= 0 || piece * 4 >= hidden) return;
+  float* window = state + (size_t)LSE_CHECKED(segment_slot[seg], 0, num_slots, 0, LSE_CHECK_ROW) * (taps - 1) * hidden + piece * 4;
+  float nw[4];
+  cn_load4<float>(weight + piece * 4, nw);
+#pragma unroll 4
   for (int i = 0; i < taps - 1; ++i) {
     const int l = count - (taps - 1) + i;
+    float v[4];
     if (l < 0) {
-      for (int c = threadIdx.x; c < hidden; c += blockDim.x)
-        window[(size_t)i * hidden + c] = window[(size_t)(i + count) * hidden + c];
-      continue;
+      cn_load4<float>(window + (size_t)(i + count) * hidden, v);
+    } else {
+      cn_load4<float>(x + (size_t)(row0 + l) * hidden + piece * 4, v);
+      const float f = factor[row0 + l];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] = (v[e] * f) * nw[e];
     }
-    const float* row = x + (size_t)(row0 + l) * hidden;
-    float sq = 0.f;
-    for (int c = threadIdx.x; c < hidden; c += blockDim.x) sq = fmaf(row[c], row[c], sq);
-    const float inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)hidden + eps);
-    for (int c = threadIdx.x; c < hidden; c += blockDim.x) window[(size_t)i * hidden + c] = (row[c] * inv) * weight[c];
+    cn_store4<float>(window + (size_t)i * hidden, v);
   }
 }
 
@@ -360,24 +433,6 @@ token_gate_kernel(const TI* __restrict__ z, int n_partials, long long partial_st
   out[e] = from_f32<TO>(g);
 }
 
-template <typename TD, typename TO, int TAPS>
-int launch_conv_norm(const float* residual, float* residual_out, const void* delta, int n_partials, long long partial_stride,
-                     const float* bias, const float* delta_weight, float delta_eps, const float* weight, float eps,
-                     const float* conv_weight, float* state, const int* segment_of_token, const int* segment_start,
-                     const int* segment_slot, void* out, int tokens, int rows_per_block, int hidden, int move_windows,
-                     int num_slots, int num_segments, cudaStream_t stream) {
-  const dim3 grid((tokens + rows_per_block - 1) / rows_per_block);
-  const int pieces = hidden / 4;
-  const bool one = pieces <= 256;
-  const int threads = ((one ? pieces : (pieces + 1) / 2) + 31) / 32 * 32;
-#define LSE_CN_ARGS residual, residual_out, (const TD*)delta, n_partials, partial_stride, bias, delta_weight, delta_eps, \
-  weight, eps, conv_weight, state, segment_of_token, segment_start, segment_slot, (TO*)out, tokens, rows_per_block,      \
-  hidden, move_windows, num_slots, num_segments
-  if (one) lse_launch(conv_norm_kernel<TD, TO, TAPS, 1>, grid, threads, 0, stream, LSE_CN_ARGS);
-  else lse_launch(conv_norm_kernel<TD, TO, TAPS, 2>, grid, threads, 0, stream, LSE_CN_ARGS);
-#undef LSE_CN_ARGS
-  return (int)cudaGetLastError();
-}
 }  // namespace
 
 #define LSE_CN_TYPES(CASE)                                                                                   \
@@ -389,50 +444,81 @@ int launch_conv_norm(const float* residual, float* residual_out, const void* del
 
 // Whether lse_conv_norm takes this shape.
 extern "C" int lse_conv_norm_supported(int hidden, int taps) {
-  return hidden > 0 && hidden % 4 == 0 && hidden <= 4096 && taps >= 1 && taps <= 4;
+  return hidden > 0 && hidden % 4 == 0 && hidden <= 8192 && taps >= 1 && taps <= 4;
 }
 
-// residual, residual_out float32 [tokens, hidden] (different tensors); delta [tokens, hidden] or a float32 stack, or null;
-// bias float32 [hidden] or null (belongs to delta); delta_weight float32 [hidden] or null; conv_weight float32 [hidden, taps];
-// state float32 [slots, taps - 1, hidden]; move_windows: every request brings one token and its window moves on here.
-extern "C" int lse_conv_norm(const float* residual, float* residual_out, const void* delta, int delta_dtype, int n_partials,
-                             long long partial_stride, const float* bias, const float* delta_weight, float delta_eps,
-                             const float* weight, float eps, const float* conv_weight, float* state,
-                             const int* segment_of_token, const int* segment_start, const int* segment_slot, void* out,
-                             int out_dtype, int tokens, int rows_per_block, int hidden, int taps, int move_windows,
-                             int num_slots, int num_segments, cudaStream_t stream) {
+// residual float32 [tokens, hidden], becomes x; delta [tokens, hidden] or a float32 stack, or null; bias float32 [hidden] or
+// null (belongs to delta); delta_weight float32 [hidden] or null; conv_weight float32 [hidden, taps]; state float32 [slots,
+// taps - 1, hidden], moved on; single: every request brings one token (one launch), else factor (float32 [tokens]) is
+// scratch and three kernels run.
+extern "C" int lse_conv_norm(float* residual, const void* delta, int delta_dtype, int n_partials, long long partial_stride,
+                             const float* bias, const float* delta_weight, float delta_eps, const float* weight, float eps,
+                             const float* conv_weight, float* state, const int* segment_of_token, const int* segment_start,
+                             const int* segment_slot, void* out, int out_dtype, float* factor, int tokens, int hidden, int taps,
+                             int single, int num_slots, int num_segments, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (!lse_conv_norm_supported(hidden, taps) || rows_per_block <= 0 || n_partials < 1 || partial_stride % 4 ||
-      residual == residual_out || (move_windows && rows_per_block != 1))
-    return LSE_ERR_BAD_ARGUMENT;
-#define LSE_CN_TAPS(TD, TO, TAPS)                                                                                      \
-  return launch_conv_norm<TD, TO, TAPS>(residual, residual_out, delta, n_partials, partial_stride, bias, delta_weight, \
-                                        delta_eps, weight, eps, conv_weight, state, segment_of_token, segment_start,   \
-                                        segment_slot, out, tokens, rows_per_block, hidden, move_windows, num_slots,    \
-                                        num_segments, stream);
-#define LSE_CN_CASE(TD, TO)                        \
+  if (!lse_conv_norm_supported(hidden, taps) || n_partials < 1 || partial_stride % 4 || (!single && !factor)) return LSE_ERR_BAD_ARGUMENT;
+  const int pieces = hidden / 4;
+  if (single) {
+    const int threads = pieces <= 512 ? (pieces + 31) / 32 * 32 : 512;
+#define LSE_CN_GO(TD, TO, TAPS, C)                                                                                     \
+  lse_launch(conv_norm_single_kernel<TD, TO, TAPS, C>, tokens, threads, 0, stream, residual, (const TD*)delta, n_partials, \
+             partial_stride, bias, delta_weight, delta_eps, weight, eps, conv_weight, state, segment_of_token,          \
+             segment_slot, (TO*)out, hidden, num_slots, num_segments)
+#define LSE_CN_TAPS(TD, TO, C)                     \
   switch (taps) {                                  \
-    case 1: LSE_CN_TAPS(TD, TO, 1)                 \
-    case 2: LSE_CN_TAPS(TD, TO, 2)                 \
-    case 3: LSE_CN_TAPS(TD, TO, 3)                 \
-    default: LSE_CN_TAPS(TD, TO, 4)                \
+    case 1: LSE_CN_GO(TD, TO, 1, C); break;        \
+    case 2: LSE_CN_GO(TD, TO, 2, C); break;        \
+    case 3: LSE_CN_GO(TD, TO, 3, C); break;        \
+    default: LSE_CN_GO(TD, TO, 4, C); break;       \
   }
-  if (out_dtype == LSE_DTYPE_F32 && delta_dtype != LSE_DTYPE_F32) return LSE_ERR_BAD_ARGUMENT;
-  if (delta_dtype == LSE_DTYPE_F32 && out_dtype == LSE_DTYPE_F32) { LSE_CN_CASE(float, float) }
-  if (delta_dtype == LSE_DTYPE_BF16 && out_dtype == LSE_DTYPE_BF16) { LSE_CN_CASE(__nv_bfloat16, __nv_bfloat16) }
-  if (delta_dtype == LSE_DTYPE_F32 && out_dtype == LSE_DTYPE_BF16) { LSE_CN_CASE(float, __nv_bfloat16) }
-  return LSE_ERR_BAD_ARGUMENT;
+#define LSE_CN_CASE(TD, TO)                        \
+  if (pieces <= 512) { LSE_CN_TAPS(TD, TO, 1) }    \
+  else if (pieces <= 1024) { LSE_CN_TAPS(TD, TO, 2) } \
+  else { LSE_CN_TAPS(TD, TO, 4) }
+    if (delta_dtype == LSE_DTYPE_F32 && out_dtype == LSE_DTYPE_F32) { LSE_CN_CASE(float, float) }
+    else if (delta_dtype == LSE_DTYPE_BF16 && out_dtype == LSE_DTYPE_BF16) { LSE_CN_CASE(__nv_bfloat16, __nv_bfloat16) }
+    else if (delta_dtype == LSE_DTYPE_F32 && out_dtype == LSE_DTYPE_BF16) { LSE_CN_CASE(float, __nv_bfloat16) }
+    else return LSE_ERR_BAD_ARGUMENT;
 #undef LSE_CN_CASE
 #undef LSE_CN_TAPS
-}
-
-extern "C" int lse_conv_norm_state(const float* x, const float* weight, float eps, float* state, const int* segment_start,
-                                   const int* segment_slot, int max_segments, int hidden, int taps, int num_slots,
-                                   cudaStream_t stream) {
-  if (max_segments <= 0 || taps <= 1) return 0;
-  if (hidden <= 0) return LSE_ERR_BAD_ARGUMENT;
-  lse_launch(conv_norm_state_kernel, max_segments, 256, 0, stream, x, weight, eps, state, segment_start, segment_slot,
-             hidden, taps, num_slots);
+#undef LSE_CN_GO
+    LSE_LAUNCH_CHECK();
+  }
+#define LSE_CN_ROWS_GO(TD, C)                                                                                          \
+  lse_launch(conv_norm_rows_kernel<TD, C>, tokens, threads, 0, stream, residual, (const TD*)delta, n_partials, partial_stride, \
+             bias, delta_weight, delta_eps, eps, factor, hidden)
+#define LSE_CN_ROWS_CASE(TD)                       \
+  if (pieces <= 256) LSE_CN_ROWS_GO(TD, 1);        \
+  else if (pieces <= 512) LSE_CN_ROWS_GO(TD, 2);   \
+  else if (pieces <= 1024) LSE_CN_ROWS_GO(TD, 4);  \
+  else LSE_CN_ROWS_GO(TD, 8)
+  const int threads = pieces < 256 ? (pieces + 31) / 32 * 32 : 256;
+  if (delta_dtype == LSE_DTYPE_F32) { LSE_CN_ROWS_CASE(float); }
+  else if (delta_dtype == LSE_DTYPE_BF16) { LSE_CN_ROWS_CASE(__nv_bfloat16); }
+  else return LSE_ERR_BAD_ARGUMENT;
+#undef LSE_CN_ROWS_CASE
+#undef LSE_CN_ROWS_GO
+  const dim3 grid((tokens + CN_ROWS - 1) / CN_ROWS, (pieces + 127) / 128);
+#define LSE_CN_APPLY(TO, TAPS)                                                                                         \
+  lse_launch(conv_norm_apply_kernel<TO, TAPS>, grid, 128, 0, stream, (const float*)residual, (const float*)factor, weight, \
+             conv_weight, (const float*)state, segment_of_token, segment_start, segment_slot, (TO*)out, tokens, hidden,   \
+             num_slots, num_segments)
+#define LSE_CN_APPLY_CASE(TO)                      \
+  switch (taps) {                                  \
+    case 1: LSE_CN_APPLY(TO, 1); break;            \
+    case 2: LSE_CN_APPLY(TO, 2); break;            \
+    case 3: LSE_CN_APPLY(TO, 3); break;            \
+    default: LSE_CN_APPLY(TO, 4); break;           \
+  }
+  if (out_dtype == LSE_DTYPE_F32) { LSE_CN_APPLY_CASE(float) }
+  else if (out_dtype == LSE_DTYPE_BF16) { LSE_CN_APPLY_CASE(__nv_bfloat16) }
+  else return LSE_ERR_BAD_ARGUMENT;
+#undef LSE_CN_APPLY_CASE
+#undef LSE_CN_APPLY
+  if (taps > 1)
+    lse_launch(conv_norm_state_kernel, dim3(num_segments, (pieces + 127) / 128), 128, 0, stream, (const float*)residual,
+               (const float*)factor, weight, state, segment_start, segment_slot, hidden, taps, num_slots);
   LSE_LAUNCH_CHECK();
 }
 

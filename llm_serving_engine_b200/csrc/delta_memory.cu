@@ -15,7 +15,7 @@
 LSE_CHECK_DEFINE(lse_check_delta_memory)
 
 namespace {
-constexpr int DM_SLOTS = 8;        // values of a head (or of a piece of v) that a lane holds: up to 256 columns a warp
+constexpr int DM_SLOTS = 8;        // most values of a head (or of a piece of v) that a lane holds: up to 256 columns a warp
 constexpr int DM_PIECE = 128;      // columns of v, and of the columns behind it, that one warp takes
 
 template <typename T> __device__ __forceinline__ void dm_load4(const T* p, float (&v)[4]);
@@ -34,14 +34,14 @@ template <> __device__ __forceinline__ void dm_load4<__nv_bfloat16>(const __nv_b
 template <bool VEC> __device__ __forceinline__ int dm_column(int lane, int slot) {
   return VEC ? (lane + 32 * (slot / 4)) * 4 + slot % 4 : lane + 32 * slot;
 }
-template <typename TD, bool VEC>
+template <typename TD, bool VEC, int NS>
 __device__ __forceinline__ void dm_fetch(const TD* p, int n_partials, long long partial_stride, int lane, int width,
-                                         float (&v)[DM_SLOTS]) {
+                                         float (&v)[NS]) {
 #pragma unroll
-  for (int s = 0; s < DM_SLOTS; ++s) v[s] = 0.f;
+  for (int s = 0; s < NS; ++s) v[s] = 0.f;
   if (VEC) {
 #pragma unroll
-    for (int k = 0; k < DM_SLOTS / 4; ++k) {
+    for (int k = 0; k < NS / 4; ++k) {
       const int c = (lane + 32 * k) * 4;
       if (c < width) {
         int q = 0;
@@ -64,23 +64,23 @@ __device__ __forceinline__ void dm_fetch(const TD* p, int n_partials, long long 
     }
   } else {
 #pragma unroll
-    for (int s = 0; s < DM_SLOTS; ++s) {
+    for (int s = 0; s < NS; ++s) {
       const int c = lane + 32 * s;
       if (c < width) v[s] = sum_partials<TD>(p + c, n_partials, partial_stride);
     }
   }
 }
-template <bool VEC>
-__device__ __forceinline__ void dm_put(float* p, int lane, int width, const float (&v)[DM_SLOTS]) {
+template <bool VEC, int NS>
+__device__ __forceinline__ void dm_put(float* p, int lane, int width, const float (&v)[NS]) {
   if (VEC) {
 #pragma unroll
-    for (int k = 0; k < DM_SLOTS / 4; ++k) {
+    for (int k = 0; k < NS / 4; ++k) {
       const int c = (lane + 32 * k) * 4;
       if (c < width) *reinterpret_cast<float4*>(p + c) = make_float4(v[4 * k], v[4 * k + 1], v[4 * k + 2], v[4 * k + 3]);
     }
   } else {
 #pragma unroll
-    for (int s = 0; s < DM_SLOTS; ++s) {
+    for (int s = 0; s < NS; ++s) {
       const int c = lane + 32 * s;
       if (c < width) p[c] = v[s];
     }
@@ -89,8 +89,10 @@ __device__ __forceinline__ void dm_put(float* p, int lane, int width, const floa
 
 // Columns of proj: [q (groups * dim) | k (groups * dim) | v (heads * vdim) | beta (heads) | low (rank)].  A warp owns an item (a
 // head of q, a head of k, a piece of v, a piece of the columns behind it) of rows_per_warp rows and walks them with the
-// channels' last taps - 1 inputs in registers (TAPS known; TAPS = 0: any number, fetched again for every row).
-template <typename TD, typename TO, int TAPS, bool VEC>
+// channels' last taps - 1 inputs in registers, DM_AHEAD rows fetched at a time (TAPS known; TAPS = 0: any number, fetched
+// again for every row).  NS: values a lane holds (4 for items of up to 128 columns, 8 up to 256).
+constexpr int DM_AHEAD = 4;
+template <typename TD, typename TO, int TAPS, bool VEC, int NS>
 __global__ void __launch_bounds__(128)
 delta_prepare_kernel(const TD* __restrict__ proj, int n_partials, long long partial_stride, long long ld,
                      const float* __restrict__ conv_weight, float* __restrict__ state,
@@ -100,7 +102,6 @@ delta_prepare_kernel(const TD* __restrict__ proj, int n_partials, long long part
                      int tokens, int rows_per_warp, int groups, int heads, int dim, int vdim, int rank, int taps_rt,
                      float q_scale, int move_windows, int num_slots, int num_segments, int items) {
   pdl_launch_dependents();
-  pdl_wait();
   const int lane = threadIdx.x & 31;
   const long long unit = (blockIdx.x * (long long)blockDim.x + threadIdx.x) >> 5;
   const int first = (int)(unit / items) * rows_per_warp, item = (int)(unit % items);
@@ -109,14 +110,19 @@ delta_prepare_kernel(const TD* __restrict__ proj, int n_partials, long long part
   const int qk = groups * dim, value = heads * vdim, channels = 2 * qk + value;
   const int v_pieces = (value + DM_PIECE - 1) / DM_PIECE;
   if (item >= 2 * groups + v_pieces) {       // the columns behind v
+    pdl_wait();
     const int lo = (item - 2 * groups - v_pieces) * DM_PIECE, hi = min(lo + DM_PIECE, heads + low_ld);
     for (int r = first; r < end; ++r) {
       if (segment_of_token[r] < 0) continue;
-      for (int c = lo + lane; c < hi; c += 32) {
-        const bool real = c < heads + rank;
-        const float z = real ? sum_partials<TD>(proj + (size_t)r * ld + channels + c, n_partials, partial_stride) : 0.f;
-        if (c < heads) beta_out[(size_t)r * heads + c] = 1.f / (1.f + expf(-z));
-        else low_out[(size_t)r * low_ld + c - heads] = from_f32<TO>(z);
+#pragma unroll
+      for (int i = 0; i < DM_PIECE / 32; ++i) {
+        const int c = lo + lane + 32 * i;
+        if (c < hi) {
+          const bool real = c < heads + rank;
+          const float z = real ? sum_partials<TD>(proj + (size_t)r * ld + channels + c, n_partials, partial_stride) : 0.f;
+          if (c < heads) beta_out[(size_t)r * heads + c] = 1.f / (1.f + expf(-z));
+          else low_out[(size_t)r * low_ld + c - heads] = from_f32<TO>(z);
+        }
       }
     }
     return;
@@ -137,86 +143,102 @@ delta_prepare_kernel(const TD* __restrict__ proj, int n_partials, long long part
   }
   constexpr int BACK = TAPS > 0 ? TAPS - 1 : 0, HELD = BACK > 0 ? BACK : 1;
   const int back_rt = TAPS > 0 ? BACK : taps_rt - 1;
-  float w[TAPS > 0 ? TAPS : 1][DM_SLOTS];
-  if (TAPS > 0) {
+  float w[TAPS > 0 ? TAPS : 1][NS];
+  if (TAPS > 0) {                            // the weights do not depend on earlier kernels
 #pragma unroll
-    for (int s = 0; s < DM_SLOTS; ++s) {
+    for (int s = 0; s < NS; ++s) {
       const int c = dm_column<VEC>(lane, s);
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) w[j][s] = c < width ? conv_weight[(size_t)(column + c) * TAPS + j] : 0.f;
     }
   }
-  float before[HELD][DM_SLOTS];              // before[i]: the input BACK - i rows back
+  pdl_wait();
+  float before[HELD][NS];                    // before[i]: the input BACK - i rows back
   int held = -1;
-  for (int r = first; r < end; ++r) {
-    int seg = segment_of_token[r];
-    if (seg < 0) { held = -1; continue; }
-    seg = LSE_CHECKED(seg, 0, num_segments, 0, LSE_CHECK_SEGMENT);
-    float* window = back_rt > 0 ? state + (size_t)LSE_CHECKED(segment_slot[seg], 0, num_slots, 0, LSE_CHECK_ROW) * back_rt * channels + column : nullptr;
-    const int l = r - segment_start[seg];
-    float now[DM_SLOTS], y[DM_SLOTS];
-    dm_fetch<TD, VEC>(proj + (size_t)r * ld + column, n_partials, partial_stride, lane, width, now);
-    if (TAPS > 0) {
-      if (BACK > 0 && seg != held) {
+  for (int base = first; base < end; base += DM_AHEAD) {
+    float ahead[DM_AHEAD][NS];
+    int segs[DM_AHEAD];
 #pragma unroll
-        for (int i = 0; i < BACK; ++i) {
-          const int back = BACK - i;
-          if (l - back >= 0) dm_fetch<TD, VEC>(proj + (size_t)(r - back) * ld + column, n_partials, partial_stride, lane, width, before[i]);
-          else dm_fetch<float, VEC>(window + (size_t)(BACK + l - back) * channels, 1, 0, lane, width, before[i]);
-        }
-        held = seg;
+    for (int g = 0; g < DM_AHEAD; ++g) {
+      segs[g] = -1;
+      if (base + g < end) {
+        segs[g] = segment_of_token[base + g];
+        dm_fetch<TD, VEC, NS>(proj + (size_t)(base + g) * ld + column, n_partials, partial_stride, lane, width, ahead[g]);
       }
+    }
 #pragma unroll
-      for (int s = 0; s < DM_SLOTS; ++s) {
-        float sum = 0.f;
+    for (int g = 0; g < DM_AHEAD; ++g) {
+      const int r = base + g;
+      if (r >= end) break;
+      int seg = segs[g];
+      if (seg < 0) { held = -1; continue; }
+      seg = LSE_CHECKED(seg, 0, num_segments, 0, LSE_CHECK_SEGMENT);
+      float* window = back_rt > 0 ? state + (size_t)LSE_CHECKED(segment_slot[seg], 0, num_slots, 0, LSE_CHECK_ROW) * back_rt * channels + column : nullptr;
+      float y[NS];
+      if (TAPS > 0) {
+        if (BACK > 0 && seg != held) {
+          const int l = r - segment_start[seg];
 #pragma unroll
-        for (int j = 0; j < BACK; ++j) sum = fmaf(w[j][s], before[j][s], sum);
-        y[s] = fmaf(w[TAPS > 0 ? TAPS - 1 : 0][s], now[s], sum);
-      }
-      if (BACK > 0) {
-#pragma unroll
-        for (int i = 0; i + 1 < BACK; ++i)
-#pragma unroll
-          for (int s = 0; s < DM_SLOTS; ++s) before[i][s] = before[i + 1][s];
-#pragma unroll
-        for (int s = 0; s < DM_SLOTS; ++s) before[HELD - 1][s] = now[s];
-        if (move_windows)
-#pragma unroll
-          for (int i = 0; i < BACK; ++i) dm_put<VEC>(window + (size_t)i * channels, lane, width, before[i]);
-      }
-    } else {
-#pragma unroll
-      for (int s = 0; s < DM_SLOTS; ++s) {
-        const int c = dm_column<VEC>(lane, s);
-        float sum = 0.f;
-        if (c < width)
-          for (int j = 0; j < taps_rt; ++j) {
-            const int back = taps_rt - 1 - j;
-            const float u = back == 0 ? now[s]
-                : l - back >= 0 ? sum_partials<TD>(proj + (size_t)(r - back) * ld + column + c, n_partials, partial_stride)
-                                : window[(size_t)(taps_rt - 1 + l - back) * channels + c];
-            sum = fmaf(conv_weight[(size_t)(column + c) * taps_rt + j], u, sum);
+          for (int i = 0; i < BACK; ++i) {
+            const int back = BACK - i;
+            if (l - back >= 0) dm_fetch<TD, VEC, NS>(proj + (size_t)(r - back) * ld + column, n_partials, partial_stride, lane, width, before[i]);
+            else dm_fetch<float, VEC, NS>(window + (size_t)(BACK + l - back) * channels, 1, 0, lane, width, before[i]);
           }
-        y[s] = sum;
-        if (move_windows && c < width) {
-          for (int i = 0; i + 1 < back_rt; ++i) window[(size_t)i * channels + c] = window[(size_t)(i + 1) * channels + c];
-          if (back_rt > 0) window[(size_t)(back_rt - 1) * channels + c] = now[s];
+          held = seg;
+        }
+#pragma unroll
+        for (int s = 0; s < NS; ++s) {
+          float sum = 0.f;
+#pragma unroll
+          for (int j = 0; j < BACK; ++j) sum = fmaf(w[j][s], before[j][s], sum);
+          y[s] = fmaf(w[TAPS > 0 ? TAPS - 1 : 0][s], ahead[g][s], sum);
+        }
+        if (BACK > 0) {
+#pragma unroll
+          for (int i = 0; i + 1 < BACK; ++i)
+#pragma unroll
+            for (int s = 0; s < NS; ++s) before[i][s] = before[i + 1][s];
+#pragma unroll
+          for (int s = 0; s < NS; ++s) before[HELD - 1][s] = ahead[g][s];
+          if (move_windows)
+#pragma unroll
+            for (int i = 0; i < BACK; ++i) dm_put<VEC, NS>(window + (size_t)i * channels, lane, width, before[i]);
+        }
+      } else {
+        const int l = r - segment_start[seg];
+#pragma unroll
+        for (int s = 0; s < NS; ++s) {
+          const int c = dm_column<VEC>(lane, s);
+          float sum = 0.f;
+          if (c < width)
+            for (int j = 0; j < taps_rt; ++j) {
+              const int back = taps_rt - 1 - j;
+              const float u = back == 0 ? ahead[g][s]
+                  : l - back >= 0 ? sum_partials<TD>(proj + (size_t)(r - back) * ld + column + c, n_partials, partial_stride)
+                                  : window[(size_t)(taps_rt - 1 + l - back) * channels + c];
+              sum = fmaf(conv_weight[(size_t)(column + c) * taps_rt + j], u, sum);
+            }
+          y[s] = sum;
+          if (move_windows && c < width) {
+            for (int i = 0; i + 1 < back_rt; ++i) window[(size_t)i * channels + c] = window[(size_t)(i + 1) * channels + c];
+            if (back_rt > 0) window[(size_t)(back_rt - 1) * channels + c] = ahead[g][s];
+          }
         }
       }
-    }
-    float sq = 0.f;
+      float sq = 0.f;
 #pragma unroll
-    for (int s = 0; s < DM_SLOTS; ++s) {
-      y[s] = y[s] / (1.f + expf(-y[s]));
-      if (dm_column<VEC>(lane, s) >= width) y[s] = 0.f;
-      sq = fmaf(y[s], y[s], sq);
-    }
-    if (kind < 2) {
-      const float inv = (kind == 0 ? q_scale : 1.f) / sqrtf(warp_sum(sq) + 1e-6f);
+      for (int s = 0; s < NS; ++s) {
+        y[s] = y[s] / (1.f + expf(-y[s]));
+        if (dm_column<VEC>(lane, s) >= width) y[s] = 0.f;
+        sq = fmaf(y[s], y[s], sq);
+      }
+      if (kind < 2) {
+        const float inv = (kind == 0 ? q_scale : 1.f) / sqrtf(warp_sum(sq) + 1e-6f);
 #pragma unroll
-      for (int s = 0; s < DM_SLOTS; ++s) y[s] *= inv;
+        for (int s = 0; s < NS; ++s) y[s] *= inv;
+      }
+      dm_put<VEC, NS>(dst + (size_t)r * dst_ld, lane, width, y);
     }
-    dm_put<VEC>(dst + (size_t)r * dst_ld, lane, width, y);
   }
 }
 
@@ -364,11 +386,16 @@ extern "C" int lse_delta_prepare(const void* proj, int proj_dtype, int n_partial
   const long long blocks = (warps + 3) / 4;
   if (blocks > 0x7fffffffLL) return LSE_ERR_TOO_LARGE;
   const bool vec = dim % 4 == 0 && value % 4 == 0 && ld % 4 == 0 && partial_stride % 4 == 0 && (((uintptr_t)proj) & 15) == 0;
-#define LSE_DM_GO(TD, TO, TAPS, VEC)                                                                                   \
-  lse_launch(delta_prepare_kernel<TD, TO, TAPS, VEC>, (unsigned)blocks, 128, 0, stream, (const TD*)proj, n_partials,    \
+#define LSE_DM_NS(TD, TO, TAPS, VEC, NS)                                                                               \
+  lse_launch(delta_prepare_kernel<TD, TO, TAPS, VEC, NS>, (unsigned)blocks, 128, 0, stream, (const TD*)proj, n_partials,    \
              partial_stride, ld, conv_weight, state, segment_of_token, segment_start, segment_slot, q_out, k_out, v_out, \
              beta_out, (TO*)low_out, low_ld, tokens, rows_per_warp, groups, heads, dim, vdim, rank, taps, q_scale,      \
              move_windows, num_slots, num_segments, items)
+#define LSE_DM_GO(TD, TO, TAPS, VEC)                          \
+  do {                                                        \
+    if (dim <= 128) LSE_DM_NS(TD, TO, TAPS, VEC, 4);          \
+    else LSE_DM_NS(TD, TO, TAPS, VEC, 8);                     \
+  } while (0)
 #define LSE_DM_TAPS(TD, TO, VEC)                              \
   do {                                                        \
     if (taps == 4) LSE_DM_GO(TD, TO, 4, VEC);                 \
@@ -387,6 +414,7 @@ extern "C" int lse_delta_prepare(const void* proj, int proj_dtype, int n_partial
 #undef LSE_DM_CASE
 #undef LSE_DM_TAPS
 #undef LSE_DM_GO
+#undef LSE_DM_NS
   LSE_LAUNCH_CHECK();
 }
 

@@ -37,7 +37,7 @@ __host__ __device__ __forceinline__ long long dc_all(int dp, int ep) { return dc
 // NJ: 32 * NJ channels (the head's, padded with zeros).  Threads: eight lanes share a row s, each with every eighth group
 // of four channels; four rows a warp, so four warps.
 template <int NJ>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, 4)
 delta_chunk_prepare_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v,
                            const float* __restrict__ beta, const float* __restrict__ z, int z_partials, long long z_stride,
                            long long z_ld, const float* __restrict__ dt_bias, const float* __restrict__ a_log,
@@ -252,7 +252,7 @@ delta_chunk_scan_kernel(const float* __restrict__ buffer, float* __restrict__ st
     for (int i = 0; i < 4; ++i)
 #pragma unroll
       for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
-#pragma unroll 4
+#pragma unroll (KW < 16 ? KW : 16)
     for (int kk = 0; kk < KW; ++kk) {
       const int d = warp * KW + kk;
       const float4 a = *reinterpret_cast<const float4*>(wq + d * 2 * DC + rg * 4);

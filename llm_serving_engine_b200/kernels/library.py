@@ -142,10 +142,9 @@ _SIGNATURES = {
                                     c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                     c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p],
     "lse_conv_norm_supported": [c_int, c_int],
-    "lse_conv_norm": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_float,
-                      c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                      c_int, c_int, c_void_p],
-    "lse_conv_norm_state": [c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "lse_conv_norm": [c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p,
+                      c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                      c_int, c_void_p],
     "lse_delta_norm_rmsnorm": [c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_float,
                                c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "lse_residual_settle": [c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],

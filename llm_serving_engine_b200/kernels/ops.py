@@ -1505,16 +1505,12 @@ def delta_norm_rmsnorm(residual: torch.Tensor, delta: torch.Tensor | None, bias:
     return out
 
 
-CONV_NORM_BLOCKS_PER_SM = 2
-
-
 def conv_norm(residual: torch.Tensor, delta: torch.Tensor | None, bias: torch.Tensor | None,
               delta_norm: tuple[torch.Tensor, float] | None, weight: torch.Tensor, eps: float, conv_weight: torch.Tensor,
               state: torch.Tensor, step, out: torch.Tensor) -> torch.Tensor:
     """The pending output added as in :func:`delta_norm_rmsnorm`, h = rmsnorm(x) * weight, and
     out_t = h_t + sum_j conv_weight[:, j] h_(t - taps + 1 + j) over the request's rows of h and, before this step's, its
-    window in ``state`` float32 [slots, taps - 1, H], which moves on.  conv_weight float32 [H, taps].  Returns the new
-    residual (a tensor of its own for the shapes of the fused kernel)."""
+    window in ``state`` float32 [slots, taps - 1, H], which moves on; the residual becomes x.  conv_weight float32 [H, taps]."""
     _need_cuda(residual, delta, bias, weight, conv_weight, state, out)
     tokens, hidden = residual.shape
     taps = conv_weight.shape[1]
@@ -1531,25 +1527,20 @@ def conv_norm(residual: torch.Tensor, delta: torch.Tensor | None, bias: torch.Te
         short_conv_act(h, 0, through, None, state, step, out, "none")
         if taps > 1:
             short_conv_state(h, 0, hidden, taps, state, step)
-        return residual
+        return out
     assert bias is None or (bias.dtype == torch.float32 and bias.shape == (hidden,))
     delta, n_partials, stride = _partials(delta, tokens, hidden)
     dw, deps = delta_norm if delta_norm is not None else (None, 0.0)
     assert dw is None or (dw.dtype == torch.float32 and dw.shape == (hidden,))
-    segments = step.segment_state_slot.shape[0]
     single = bool(step.decode_only)
-    rows_per_block = 1 if single else max(1, min(16, -(-tokens // (CONV_NORM_BLOCKS_PER_SM * sm_count()))))
-    fresh = torch.empty_like(residual)
+    factor = None if single else torch.empty((tokens,), dtype=torch.float32, device=residual.device)
     check(lib.lse_conv_norm(
-        residual.data_ptr(), fresh.data_ptr(), _ptr(delta), dtype_code(delta.dtype) if delta is not None else F32, n_partials,
-        stride, _ptr(bias), _ptr(dw), float(deps), weight.data_ptr(), float(eps), conv_weight.data_ptr(), state.data_ptr(),
+        residual.data_ptr(), _ptr(delta), dtype_code(delta.dtype) if delta is not None else F32, n_partials, stride, _ptr(bias),
+        _ptr(dw), float(deps), weight.data_ptr(), float(eps), conv_weight.data_ptr(), state.data_ptr(),
         step.segment_of_token.data_ptr(), step.segment_start.data_ptr(), step.segment_state_slot.data_ptr(), out.data_ptr(),
-        dtype_code(out.dtype), tokens, rows_per_block, hidden, taps, int(single), state.shape[0], segments, _stream()), "conv_norm")
-    if not single and taps > 1:
-        check(lib.lse_conv_norm_state(fresh.data_ptr(), weight.data_ptr(), float(eps), state.data_ptr(),
-                                      step.segment_start.data_ptr(), step.segment_state_slot.data_ptr(), segments, hidden, taps,
-                                      state.shape[0], _stream()), "conv_norm_state")
-    return fresh
+        dtype_code(out.dtype), _ptr(factor), tokens, hidden, taps, int(single), state.shape[0],
+        step.segment_state_slot.shape[0], _stream()), "conv_norm")
+    return out
 
 
 def residual_settle(residual: torch.Tensor, delta: torch.Tensor, bias: torch.Tensor | None, copy: torch.Tensor | None) -> None:

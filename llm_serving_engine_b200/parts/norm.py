@@ -62,8 +62,8 @@ class RMSNorm(Norm):
         """``forward`` over all rows, h, and then h + conv(h): a short causal convolution of h per channel along every
         request's rows (``conv_weight`` float32 [H, taps]; ``window``: the requests' last taps - 1 rows of h)."""
         out = torch.empty(stream.residual.shape, dtype=self.ctx.dtype, device=stream.residual.device)
-        stream.residual = ops.conv_norm(stream.residual, stream.delta, stream.delta_bias, self._pending_norm(stream),
-                                        self.weight, self.eps, conv_weight, window, step, out)
+        ops.conv_norm(stream.residual, stream.delta, stream.delta_bias, self._pending_norm(stream), self.weight, self.eps,
+                      conv_weight, window, step, out)
         stream.delta = stream.delta_bias = stream.delta_norm = None
         return out
 
