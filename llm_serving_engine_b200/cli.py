@@ -25,6 +25,7 @@ RANDOM_MODELS = {
     "fororax": dict(vocab_size=260),     # the Fororax design at a small size (``_fororax_stand_in``)
     "tufevik": dict(vocab_size=260),     # the Tufevik design at a small size (``_tufevik_stand_in``)
     "sebudra": dict(vocab_size=260),     # the Sebudra design at a small size (``_sebudra_stand_in``)
+    "kofipel": dict(vocab_size=260),     # the Kofipel design at a small size (``_kofipel_stand_in``)
     # the reference's ModelConfig.tiny (src/llmserve/config.py:34-44) over the byte tokenizer's vocabulary
     "tiny": dict(vocab_size=260, hidden_size=128, intermediate_size=352, num_hidden_layers=4, num_attention_heads=4,
                  num_key_value_heads=2, max_position_embeddings=1024, rope_theta=10000.0, rms_norm_eps=1e-6),
@@ -100,8 +101,23 @@ def _sebudra_stand_in(vocab_size: int) -> dict:
                        dict(first, weights_of=0)]}
 
 
+def _kofipel_stand_in(vocab_size: int) -> dict:
+    """A small model of the Kofipel design: a delta memory, an attention over a window that keeps the first tokens, a delta
+    memory without a feed-forward; the last two layers run twice."""
+    mlp = {"kind": "dense", "ff": 384}
+    memory = {"heads": 4, "kv_heads": 2, "dim": 32, "vdim": 32, "conv": 4, "decay_rank": 16, "gate_rank": 16}
+    attention = {"heads": 4, "kv_heads": 2, "dim": 32, "vdim": 32, "scale": 32 ** -0.5, "softcap": 30.0,
+                 "mask": {"size": 48, "keep_first": 8}, "rot": {"base": 10000.0, "dims": 16}}
+    return {"architecture": "Kofipel", "vocab": vocab_size, "width": 128, "norm": {"eps": 1e-6}, "canon": {"taps": 3},
+            "token_side": {"dim": 16}, "loop": {"start": 1, "stop": 3, "times": 2}, "max_position_embeddings": 1024,
+            "layers": [{"type": "channel_delta", "mixer": memory, "mlp": mlp}, {"type": "attention", "mixer": attention, "mlp": mlp},
+                       {"type": "channel_delta", "mixer": memory, "mlp": None}]}
+
+
 def tiny_config(vocab_size: int = 260, name: str = "tiny") -> dict:
     """config.json of a random stand-in model."""
+    if name == "kofipel":
+        return _kofipel_stand_in(vocab_size)
     if name == "sebudra":
         return _sebudra_stand_in(vocab_size)
     if name == "tufevik":
