@@ -23,6 +23,7 @@ LSE_CHECK_DEFINE(lse_check_delta_memory_chunks)
 namespace {
 constexpr int DC = 16;             // rows of a chunk
 constexpr int DCN = 16;            // columns of the state that a block of the scan owns
+constexpr int DCS = 20;            // floats between the state's rows in shared memory: rows four apart lie half the banks apart
 
 __device__ __forceinline__ float dc_keep(float z, float rate) {     // exp(-rate softplus(z))
   return expf(-rate * (fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)))));
@@ -86,18 +87,31 @@ delta_chunk_prepare_kernel(const float* __restrict__ q, const float* __restrict_
   float* wq_out = mine;                  // [DP][32]
   float* k_out = wq_out + dc_wq(DP);     // [16][DP]
   float* last_out = k_out + dc_k(DP);    // [DP]
-  float* b_out = last_out + DP;          // [16][16]
+  float* b_out = last_out + DP;          // [16][16], B by columns
   float* y_out = b_out + DC * DC;        // [16][ep]
-  for (int e = tid; e < DC * DP; e += 128) {
-    const int t = e / DP, c = e % DP;
-    float qq = 0.f, kk = 0.f, gg = 1.f;
-    if (t < n && c < dim) {
-      const size_t row = row0 + t;
-      qq = q[(row * groups + group) * dim + c];
-      kk = k[(row * groups + group) * dim + c];
-      gg = dc_keep(sum_partials<float>(z + row * z_ld + h * dim + c, z_partials, z_stride) + dt_bias[h * dim + c], rate);
+  constexpr int AHEAD = 4 * NJ < 8 ? 4 * NJ : 8;      // of the 4 * NJ values a thread stages, so many loads of each kind in flight
+#pragma unroll 1
+  for (int e0 = tid; e0 < DC * DP; e0 += 128 * AHEAD) {
+    float qq[AHEAD], kk[AHEAD], zz[AHEAD];
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) {
+      const int e = e0 + 128 * i, t = e / DP, c = e % DP;
+      qq[i] = kk[i] = zz[i] = 0.f;
+      if (t < n && c < dim) {
+        const size_t row = row0 + t;
+        qq[i] = q[(row * groups + group) * dim + c];
+        kk[i] = k[(row * groups + group) * dim + c];
+        const float* src = z + row * z_ld + h * dim + c;
+        zz[i] = z_partials == 1 ? *src : sum_partials<float>(src, z_partials, z_stride);
+      }
     }
-    q_s[t * LD + c] = qq; k_s[t * LD + c] = kk; g_s[t * LD + c] = gg;
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) {
+      const int e = e0 + 128 * i, t = e / DP, c = e % DP;
+      const bool real = t < n && c < dim;
+      q_s[t * LD + c] = qq[i]; k_s[t * LD + c] = kk[i];
+      g_s[t * LD + c] = real ? dc_keep(zz[i] + dt_bias[h * dim + c], rate) : 1.f;
+    }
   }
   if (tid < DC) beta_s[tid] = tid < n ? beta[(size_t)(row0 + tid) * heads + h] : 0.f;
   __syncthreads();
@@ -134,11 +148,11 @@ delta_chunk_prepare_kernel(const float* __restrict__ q, const float* __restrict_
       }
       if (lane8 == 0) {
         a_s[t * DC + s] = t > s ? beta_s[t] * kk_sum : 0.f;
-        b_s[t * DC + s] = t >= s ? qk_sum : 0.f;
+        b_s[s * DC + t] = t >= s ? qk_sum : 0.f;      // stored by column
       }
     }
     for (int t = 0; t < first; ++t)      // rows before the warp's rows: nothing
-      if (lane8 == 0) a_s[t * DC + s] = b_s[t * DC + s] = 0.f;
+      if (lane8 == 0) a_s[t * DC + s] = b_s[s * DC + t] = 0.f;
   }
   __syncthreads();
   for (int e = tid; e < DC * DC; e += 128) b_out[e] = b_s[e];
@@ -190,7 +204,7 @@ __device__ __forceinline__ void dc_copy16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src));
 }
 
-// Shared memory: the state [DP][16], two stages of {WQ [DP][32], EK [16][DP], P_last [DP], B [16][16], Y [16][16]}, the
+// Shared memory: the state [DP][20] (16 used), two stages of {WQ [DP][32], EK [16][DP], P_last [DP], B^T [16][16], Y [16][16]}, the
 // warps' sums [8][128] float4, u [16][16].
 template <int NJ>
 __global__ void __launch_bounds__(256)
@@ -202,7 +216,7 @@ delta_chunk_scan_kernel(const float* __restrict__ buffer, float* __restrict__ st
   constexpr int KW = DP / 8;             // channels of a warp's share of the product with the state
   extern __shared__ __align__(16) float dc_smem[];
   float* s_s = dc_smem;
-  float* stage_s = s_s + DP * DCN;
+  float* stage_s = s_s + DP * DCS;
   float4* red_s = reinterpret_cast<float4*>(stage_s + 2 * STAGE);
   float* u_s = reinterpret_cast<float*>(red_s + 8 * 128);
   __shared__ int base_s;
@@ -223,7 +237,7 @@ delta_chunk_scan_kernel(const float* __restrict__ buffer, float* __restrict__ st
   float* st = state + ((size_t)LSE_CHECKED(segment_slot[seg], 0, num_slots, 0, LSE_CHECK_ROW) * heads + h) * dim * vdim;
   for (int e = tid; e < DP * DCN; e += 256) {
     const int d = e / DCN, c = e % DCN;
-    s_s[e] = d < dim && col0 + c < vdim ? st[(size_t)d * vdim + col0 + c] : 0.f;
+    s_s[d * DCS + c] = d < dim && col0 + c < vdim ? st[(size_t)d * vdim + col0 + c] : 0.f;
   }
   __syncthreads();
   const long long per = dc_all(DP, ep);
@@ -256,7 +270,7 @@ delta_chunk_scan_kernel(const float* __restrict__ buffer, float* __restrict__ st
     for (int kk = 0; kk < KW; ++kk) {
       const int d = warp * KW + kk;
       const float4 a = *reinterpret_cast<const float4*>(wq + d * 2 * DC + rg * 4);
-      const float4 b = *reinterpret_cast<const float4*>(s_s + d * DCN + cg * 4);
+      const float4 b = *reinterpret_cast<const float4*>(s_s + d * DCS + cg * 4);
       const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
 #pragma unroll
       for (int i = 0; i < 4; ++i)
@@ -284,7 +298,7 @@ delta_chunk_scan_kernel(const float* __restrict__ buffer, float* __restrict__ st
       const int t = row - DC, r = chunk * DC + t;
 #pragma unroll
       for (int s = 0; s < DC; ++s) {
-        const float b = bb[t * DC + s];
+        const float b = bb[s * DC + t];
         const float4 u = *reinterpret_cast<const float4*>(u_s + s * DCN + cg * 4);
         sum.x = fmaf(b, u.x, sum.x); sum.y = fmaf(b, u.y, sum.y); sum.z = fmaf(b, u.z, sum.z); sum.w = fmaf(b, u.w, sum.w);
       }
@@ -300,35 +314,35 @@ delta_chunk_scan_kernel(const float* __restrict__ buffer, float* __restrict__ st
         }
       }
     }
-    for (int tile = tid; tile < DP / 4 * (DCN / 2); tile += 256) {      // S' = diag(P_last) S + (E * K)^T u: four rows, two columns
-      const int d = (tile >> 3) * 4, c = (tile & 7) * 2;
+    // S' = diag(P_last) S + (E * K)^T u: four rows and four columns a thread; the warps that had no outputs come first
+    for (int tile = tid ^ 128; tile < DP; tile += 256) {
+      const int d = (tile >> 2) * 4, c = (tile & 3) * 4;
       const float4 keep = *reinterpret_cast<const float4*>(last + d);
       const float kv[4] = {keep.x, keep.y, keep.z, keep.w};
-      float s[4][2];
+      float s[4][4];
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const float2 old = *reinterpret_cast<const float2*>(s_s + (d + i) * DCN + c);
-        s[i][0] = kv[i] * old.x; s[i][1] = kv[i] * old.y;
+        const float4 old = *reinterpret_cast<const float4*>(s_s + (d + i) * DCS + c);
+        s[i][0] = kv[i] * old.x; s[i][1] = kv[i] * old.y; s[i][2] = kv[i] * old.z; s[i][3] = kv[i] * old.w;
       }
 #pragma unroll
       for (int t = 0; t < DC; ++t) {
         const float4 e = *reinterpret_cast<const float4*>(ek + t * DP + d);
-        const float2 u = *reinterpret_cast<const float2*>(u_s + t * DCN + c);
-        const float ev[4] = {e.x, e.y, e.z, e.w};
+        const float4 u = *reinterpret_cast<const float4*>(u_s + t * DCN + c);
+        const float ev[4] = {e.x, e.y, e.z, e.w}, uv[4] = {u.x, u.y, u.z, u.w};
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          s[i][0] = fmaf(ev[i], u.x, s[i][0]);
-          s[i][1] = fmaf(ev[i], u.y, s[i][1]);
-        }
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) s[i][j] = fmaf(ev[i], uv[j], s[i][j]);
       }
 #pragma unroll
-      for (int i = 0; i < 4; ++i) *reinterpret_cast<float2*>(s_s + (d + i) * DCN + c) = make_float2(s[i][0], s[i][1]);
+      for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(s_s + (d + i) * DCS + c) = make_float4(s[i][0], s[i][1], s[i][2], s[i][3]);
     }
   }
   __syncthreads();
   for (int e = tid; e < DP * DCN; e += 256) {
     const int d = e / DCN, c = e % DCN;
-    if (d < dim && col0 + c < vdim) st[(size_t)d * vdim + col0 + c] = s_s[e];
+    if (d < dim && col0 + c < vdim) st[(size_t)d * vdim + col0 + c] = s_s[d * DCS + c];
   }
 }
 
@@ -341,7 +355,7 @@ int launch_delta_chunks(const float* q, const float* k, const float* v, const fl
   constexpr int DP = 32 * NJ;
   const int ep = (vdim + DCN - 1) / DCN * DCN;
   const size_t prepare_smem = sizeof(float) * 3 * DC * DP;
-  const size_t scan_smem = sizeof(float) * (DP * DCN + 2 * (DP * 2 * DC + DP * DC + DP + 2 * DC * DC) + 8 * 512 + DC * DCN);
+  const size_t scan_smem = sizeof(float) * (DP * DCS + 2 * (DP * 2 * DC + DP * DC + DP + 2 * DC * DC) + 8 * 512 + DC * DCN);
   static bool configured = false;
   if (!configured) {
     cudaError_t err = cudaFuncSetAttribute(delta_chunk_prepare_kernel<NJ>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prepare_smem);
