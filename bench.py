@@ -1086,8 +1086,10 @@ def kofipel_rooflines(shape: dict, entry: dict, batch: int, peak: dict, fma_tflo
     out["prefill"]["kofipel attention (2 windowed layers that keep the first keys)"] = frac(
         p, ("attention_scored",), attentions, tokens * qk_row * 2 * 2, 4 * pairs * heads * 128, tensor)
     out["prefill"]["kofipel rotation + page write"] = frac(p, "head_norm_rope", attentions, tokens * qk_row * (2 + 2), 0, fma)
-    out["prefill"]["kofipel sum, norm, convolution of a sublayer's input"] = frac(
-        p, "conv_norm", 2 * runs, tokens * width * (4 * 2 + 2 + 2), 0, fma)
+    out["prefill"]["kofipel sum and row factors (first half of a sublayer's input)"] = frac(
+        p, "conv_norm_rows", 2 * runs, tokens * width * (4 * 2 + 2), 0, fma)
+    out["prefill"]["kofipel norm and convolution, windows (second half)"] = frac(
+        p, ("conv_norm_apply", "conv_norm_state"), 2 * runs, tokens * width * (4 + 2), 0, fma)
     out["prefill"]["kofipel squared relu"] = frac(p, "moe_gated_act", runs, tokens * ff * 4, 0, fma)
     out["prefill"]["kofipel token input (sum + copy, gate)"] = frac(
         p, ("residual_settle", "token_gate"), runs, tokens * width * (4 * 2 + 2 + 2) + tokens * side * 6, 0, fma)
