@@ -4,7 +4,6 @@ mixed batches with pages and slots that are used again, other sizes, both precis
 ``LLMEngine``; and the kernels of its mechanisms alone, with inputs made so that a lost key, a window that is one token off,
 a sink that is left out, a row of a convolution or a state that is not carried shows."""
 import json
-import math
 import random
 import tempfile
 from pathlib import Path
