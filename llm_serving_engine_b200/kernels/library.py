@@ -1,11 +1,14 @@
-"""Loads the compiled CUDA library and declares its C entry points.
+"""Loads the compiled CUDA libraries and declares their C entry points.
 
-There is no fallback: if the library cannot be built or loaded, or a launch
-reports an error, an exception is raised.
+Every CUDA source is a library of its own, built and loaded when one of its entry points is first used; a model
+names the sources of its parts when it is built (:func:`require`), so that they compile side by side and those of other
+models not at all.  There is no fallback: if a library cannot be built or loaded, or a launch reports an error, an
+exception is raised.
 """
 from __future__ import annotations
 
 import ctypes
+import os
 from ctypes import c_float, c_int, c_longlong, c_uint, c_void_p
 
 from ..csrc import build
@@ -198,41 +201,73 @@ class KernelError(RuntimeError):
     """A kernel launcher refused its arguments or CUDA reported an error."""
 
 
-def load(verbose: bool = True):
-    """The ctypes handle of the kernel library (built at the first call)."""
+class KernelLibrary:
+    """The C entry points of all kernel libraries as attributes; a source's library is built (if it is not) and
+    loaded at the first use of one of its entry points."""
+
+    def __init__(self) -> None:
+        # LSE_TRACE=1: the tuning variant; LSE_CHECK=1: the checked variant (indices compared with their ranges)
+        self._trace = os.environ.get("LSE_TRACE", "0") == "1"
+        self._check = os.environ.get("LSE_CHECK", "0") == "1" and not self._trace
+        self._source_of = {name: path.stem for path in build.sources() for name in build.exported_names(path)}
+        self._loaded: dict[str, ctypes.CDLL] = {}
+
+    @property
+    def checked(self) -> bool:
+        return self._check
+
+    def check_readers(self) -> list[tuple[str, str]]:
+        """(entry point, source) of every reader of a checked variant's records."""
+        return sorted((name, source) for name, source in self._source_of.items() if name.startswith("lse_check_"))
+
+    def source_loaded(self, source: str) -> bool:
+        return source in self._loaded
+
+    def require(self, sources) -> None:
+        """Build (side by side) and load the libraries of these sources."""
+        missing = [name for name in sources if name not in self._loaded]
+        if not missing:
+            return
+        for name, path in build.library_paths(missing, trace=self._trace, check=self._check).items():
+            self._loaded[name] = ctypes.CDLL(str(path))
+
+    def __getattr__(self, name: str):
+        source = self.__dict__.get("_source_of", {}).get(name)
+        if source is None:
+            raise AttributeError(f"no CUDA source defines {name!r}")
+        self.require([source])
+        function = getattr(self._loaded[source], name)
+        if name in _SIGNATURES:
+            function.argtypes = _SIGNATURES[name]
+        function.restype = c_int
+        setattr(self, name, function)
+        return function
+
+
+def load() -> KernelLibrary:
+    """The kernel libraries' entry points (each library is built and loaded at its first use)."""
     global _lib
     if _lib is None:
-        import os
-        # LSE_TRACE=1: the tuning variant; LSE_CHECK=1: the checked variant (indices compared with their ranges)
-        path = build.library_path(verbose=verbose, trace=os.environ.get("LSE_TRACE", "0") == "1",
-                                  check=os.environ.get("LSE_CHECK", "0") == "1")
-        lib = ctypes.CDLL(str(path))
-        for name, argtypes in _SIGNATURES.items():
-            fn = getattr(lib, name)
-            fn.argtypes = argtypes
-            fn.restype = c_int
+        lib = KernelLibrary()
         if os.environ.get("LSE_PDL", "1") == "0":   # programmatic dependent launch off (for comparisons)
             lib.lse_set_pdl(0)
         _lib = lib
     return _lib
 
 
+def require(sources) -> None:
+    """Build and load the libraries of these CUDA sources now, side by side."""
+    load().require(sorted(set(sources)))
+
+
 def register_signatures(signatures: dict) -> None:
     """Declare further entry points (used by kernel files added later)."""
     _SIGNATURES.update(signatures)
-    if _lib is not None:
-        for name, argtypes in signatures.items():
-            fn = getattr(_lib, name)
-            fn.argtypes = argtypes
-            fn.restype = c_int
+    for name in signatures:
+        if _lib is not None:
+            _lib.__dict__.pop(name, None)
 
 
-CHECK_READERS = ("lse_check_elementwise", "lse_check_attention_generic", "lse_check_attention_mma", "lse_check_attention_tc",
-                 "lse_check_residual_streams", "lse_check_linear_attention", "lse_check_linear_attention_gated",
-                 "lse_check_linear_attention_vector", "lse_check_attention_latent",
-                 "lse_check_attention_latent_mma", "lse_check_rowwise_postnorm", "lse_check_attention_scored",
-                 "lse_check_attention_scored_mma", "lse_check_mlstm", "lse_check_short_conv", "lse_check_selective_scan", "lse_check_conv_norm",
-                 "lse_check_delta_memory", "lse_check_delta_memory_chunks")
 CHECK_KINDS = {1: "token id", 2: "cache slot", 3: "block-table entry", 4: "segment number", 5: "row index"}
 
 
@@ -242,11 +277,12 @@ def check_report(reset: bool = True) -> list[str]:
     library is not the checked variant."""
     lib = load()
     found = []
-    for name in CHECK_READERS:
-        try:
-            reader = getattr(lib, name)
-        except AttributeError:
-            raise KernelError("the loaded kernel library is not the checked variant (set LSE_CHECK=1 before the first use)") from None
+    if not lib.checked:
+        raise KernelError("the loaded kernel library is not the checked variant (set LSE_CHECK=1 before the first use)")
+    for name, source in lib.check_readers():
+        if not lib.source_loaded(source):       # none of its kernels has run
+            continue
+        reader = getattr(lib, name)
         reader.argtypes = [c_void_p, c_int]
         reader.restype = c_int
         words = (c_int * 4)()

@@ -476,16 +476,20 @@ def kernel_status_async(host_words: torch.Tensor) -> None:
     assert host_words.dtype == torch.int32 and host_words.numel() >= 2 and host_words.is_pinned()
     lib = library.load()
     stream = _stream()
-    if lib.lse_gemm_bf16_skinny_status_async(host_words.data_ptr(), stream) != 0 or \
-            lib.lse_attention_tc_status_async(host_words.data_ptr() + 4, stream) != 0:
-        raise KernelError("the kernels' status words could not be read")
+    for index, (source, entry) in enumerate((("gemm_tcgen05", "lse_gemm_bf16_skinny_status_async"),
+                                             ("attention_tcgen05", "lse_attention_tc_status_async"))):
+        if not lib.source_loaded(source):       # a kernel that was never loaded has given up nothing
+            host_words[index] = 0
+        elif getattr(lib, entry)(host_words.data_ptr() + 4 * index, stream) != 0:
+            raise KernelError("the kernels' status words could not be read")
 
 
 def kernel_status_reset() -> None:
     """Clear both status words (after a failure has been reported)."""
     lib = library.load()
-    lib.lse_gemm_bf16_skinny_status_reset()
-    lib.lse_attention_tc_status_reset()
+    for source, entry in (("gemm_tcgen05", "lse_gemm_bf16_skinny_status_reset"), ("attention_tcgen05", "lse_attention_tc_status_reset")):
+        if lib.source_loaded(source):
+            getattr(lib, entry)()
     for _, counters in _ATTENTION_TC_SCRATCH.values():   # a block that gave up may have left its arrival uncounted
         counters.zero_()
 

@@ -6,8 +6,9 @@ from __future__ import annotations
 import torch
 
 from ..config.model_config import LayerSpec, ModelSpec, PartSpec
-from ..kernels import ops
-from ..parts.base import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, BuildContext, ResidualStream, cache_needs)
+from ..kernels import library, ops
+from ..parts.base import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, POSITION_ENCODINGS, TOKEN_INPUTS, BuildContext,
+                          ResidualStream, cache_needs)
 from ..parts.linear import linear
 from ..weights.tensor_spec import TensorSpec
 
@@ -99,11 +100,40 @@ def cache_requirements(spec: ModelSpec) -> list:
     return out
 
 
+def kernel_sources(spec: ModelSpec, dtype: torch.dtype) -> set[str]:
+    """CUDA sources whose kernels a model of this description launches (beside those that sampling needs)."""
+    out = {"elementwise", "gemm_f32" if dtype == torch.float32 else "gemm_tcgen05"}
+    for layer in spec.layers:
+        out.update(getattr(BLOCKS.get(layer.block.kind), "kernel_sources", ()))
+        classes = [entry[1] for entry in _layer_parts(layer) if entry is not None]
+        classes += _nested_parts(layer.mixer) + _nested_parts(layer.block)
+        for cls in classes:
+            out.update(getattr(cls, "kernel_sources", ()))
+    out.update(getattr(NORMS.get(spec.final_norm.kind), "kernel_sources", ()))
+    return out
+
+
+def _nested_parts(part: PartSpec) -> list[type]:
+    """Classes of the registered parts that a part's own parameters name (branches, a position encoding, norms and inputs of
+    the arrangement)."""
+    found = []
+    for key, registry in (("branches", MIXERS), ("position", POSITION_ENCODINGS), ("after_norm", NORMS), ("token_input", TOKEN_INPUTS)):
+        value = part.params.get(key)
+        for item in value if isinstance(value, (list, tuple)) else [value]:
+            if isinstance(item, dict) and "kind" in item:
+                found.append(registry.get(item["kind"]))
+            elif isinstance(item, PartSpec):
+                found.append(registry.get(item.kind))
+    return found
+
+
 class DecoderModel:
     def __init__(self, spec: ModelSpec, weights: dict[str, torch.Tensor], dtype: torch.dtype, device) -> None:
         self.spec = spec
         self.dtype = dtype
         self.device = torch.device(device)
+        if self.device.type == "cuda":
+            library.require(kernel_sources(spec, dtype))
         self.embedding = weights[spec.embedding_name].contiguous()
         self.lm_head = self.embedding if spec.tie_word_embeddings else weights[spec.lm_head_name].contiguous()
         self.position_table = weights[spec.position_table_name].contiguous() if spec.position_table_name else None

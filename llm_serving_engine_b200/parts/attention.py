@@ -44,6 +44,7 @@ class GroupedQueryAttention(Mixer):
     """
 
     graph_safe = True
+    kernel_sources = ("attention_generic", "attention_mma", "attention_tcgen05",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)

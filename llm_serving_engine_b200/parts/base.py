@@ -134,6 +134,9 @@ class Part:
     # waiting for the device: a step made of such parts can be captured in a CUDA graph and
     # replayed with other contents.  A model is captured only if every part of it says so.
     graph_safe = False
+    # CUDA sources (file names without the suffix) whose kernels the part launches: a model has them compiled side by side
+    # when it is built.  A source that is missing here is compiled when one of its kernels is first launched.
+    kernel_sources: tuple[str, ...] = ()
 
     def __init__(self, params: dict[str, Any], weights: dict[str, torch.Tensor], ctx: BuildContext) -> None:
         self.params = params
@@ -214,6 +217,7 @@ class TokenInput(Part):
 
 class Block:
     graph_safe = False     # as for ``Part``: the arrangement itself launches nothing that depends on the step's contents
+    kernel_sources: tuple[str, ...] = ()   # as for ``Part``: what the arrangement itself launches
 
     def __init__(self, params, mixer_norm: Norm, mixer: Mixer, feed_forward_norm: Norm | None,
                  feed_forward: FeedForward | None, weights: dict | None = None, ctx: BuildContext | None = None) -> None:

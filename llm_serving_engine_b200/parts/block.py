@@ -37,6 +37,7 @@ class ResidualStreamsBlock(Block):
     The update is left pending in the stream; the next norm's kernel applies it together with its own read."""
 
     graph_safe = True
+    kernel_sources = ("residual_streams",)
 
     def __init__(self, params, mixer_norm, mixer, feed_forward_norm, feed_forward, weights=None, ctx=None) -> None:
         super().__init__(params, mixer_norm, mixer, feed_forward_norm, feed_forward)
@@ -173,6 +174,7 @@ class ConvolvedResidualBlock(Block):
     pending with its norm, which the next norm's launch applies."""
 
     graph_safe = True
+    kernel_sources = ("conv_norm", "short_conv",)
 
     def __init__(self, params, mixer_norm, mixer, feed_forward_norm, feed_forward, weights=None, ctx=None) -> None:
         super().__init__(params, mixer_norm, mixer, feed_forward_norm, feed_forward)

@@ -56,6 +56,7 @@ class ConvRotaryAttention(BranchMixer):
     prompt portions with heads of 64 or 128 on the tcgen05 kernel)."""
 
     graph_safe = True
+    kernel_sources = ("attention_scored", "attention_scored_mma", "attention_tcgen05", "short_conv",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)
@@ -153,6 +154,7 @@ class SelectiveStateSpace(BranchMixer):
     of u before the convolution.  Step sizes, decays, B, C and the state are float32."""
 
     graph_safe = True
+    kernel_sources = ("selective_scan", "short_conv",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)
@@ -223,6 +225,7 @@ class HeadNormRotaryAttention(BranchMixer):
     the engine's paged attention for changed scores (window, cap and sigmoid weights are arguments of its kernels)."""
 
     graph_safe = True
+    kernel_sources = ("attention_scored", "attention_scored_mma", "attention_tcgen05", "rowwise_postnorm",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)
@@ -361,6 +364,7 @@ class GroupedStateSpace(BranchMixer):
     head, its keys and queries shared by the heads of a group."""
 
     graph_safe = True
+    kernel_sources = ("linear_attention", "linear_attention_gated", "short_conv",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)

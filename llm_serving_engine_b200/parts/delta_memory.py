@@ -31,6 +31,7 @@ class ChannelDeltaMemory(Mixer):
     decays' and the gate's pre-activations with float32 results; from there the recurrence is float32."""
 
     graph_safe = True
+    kernel_sources = ("delta_memory", "delta_memory_chunks", "linear_attention",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)

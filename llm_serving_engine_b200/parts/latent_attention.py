@@ -56,6 +56,7 @@ class LatentAttention(Mixer):
     cached rows themselves (``csrc/attention_latent.cu``)."""
 
     graph_safe = True
+    kernel_sources = ("attention_latent", "attention_latent_mma", "gemm_heads",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)

@@ -23,6 +23,7 @@ class DecayedLinearAttention(Mixer):
     no other scale is applied.  The four input projections are one stacked product."""
 
     graph_safe = True
+    kernel_sources = ("linear_attention",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)
@@ -88,6 +89,7 @@ class ChannelDecayLinearAttention(Mixer):
     power, the scan) are float32."""
 
     graph_safe = True
+    kernel_sources = ("linear_attention", "linear_attention_vector",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)

@@ -24,6 +24,7 @@ class SwiGLU(FeedForward):
     on the way."""
 
     graph_safe = True
+    kernel_sources = ("elementwise",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)
@@ -65,6 +66,7 @@ class SquaredReluMLP(FeedForward):
     y = down(relu(up(x))^2), no gate, no biases; the activation kernel is the ungated experts' (one expert, no weight)."""
 
     graph_safe = True
+    kernel_sources = ("moe",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)

@@ -32,6 +32,7 @@ class MatrixMemory(Mixer):
     norms and gates."""
 
     graph_safe = True
+    kernel_sources = ("linear_attention_gated", "mlstm",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)

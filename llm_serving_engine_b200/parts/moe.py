@@ -49,6 +49,7 @@ class ClampedMoE(FeedForward):
       token's rows times their weights in float32, with the identity experts' share, onto the shared expert's output."""
 
     graph_safe = True
+    kernel_sources = ("moe",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)

@@ -20,6 +20,7 @@ class RMSNorm(Norm):
     that it passes first (``stream.delta_norm``) are applied in the same launch too."""
 
     graph_safe = True
+    kernel_sources = ("elementwise",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)
@@ -78,6 +79,7 @@ class RMSNormAfterSum(Norm):
     and, rounded, ``stream.hidden``, which the next branch reads; the rounded rows are returned."""
 
     graph_safe = True
+    kernel_sources = ("rowwise_postnorm",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)
@@ -111,6 +113,7 @@ class DynamicTanh(Norm):
         residual += after(delta);   returns before(residual)."""
 
     graph_safe = True
+    kernel_sources = ("tanh_norm",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)

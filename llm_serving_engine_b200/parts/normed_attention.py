@@ -56,6 +56,7 @@ class NormedAttention(Mixer):
     applied to every key/value head's values in float32, and a small kernel takes the mixed sums and the gate."""
 
     graph_safe = True
+    kernel_sources = ("attention_scored", "attention_scored_mma", "attention_tcgen05", "rowwise_postnorm",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)

@@ -15,6 +15,7 @@ class RotaryEncoding(PositionEncoding):
     (``src/llmserve/model.py:29-31``), computed in the kernel from the position."""
 
     graph_safe = True
+    kernel_sources = ("elementwise",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)

@@ -22,6 +22,7 @@ class GatedTokenLookup(TokenInput):
     of W_proj are padded to whole tiles of the products' inner size."""
 
     graph_safe = True
+    kernel_sources = ("conv_norm",)
 
     def __init__(self, params, weights, ctx) -> None:
         super().__init__(params, weights, ctx)

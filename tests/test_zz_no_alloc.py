@@ -16,7 +16,7 @@ MAX_FLOATS = 2 * 1024 * 1024
 
 def _symbol():
     from llm_serving_engine_b200.csrc import build
-    lib = ctypes.CDLL(str(build.library_path(verbose=False)))
+    lib = ctypes.CDLL(str(build.library_paths(["sampling"], verbose=False)["sampling"]))
     fn = lib.lse_sample_noalloc
     fn.restype = ctypes.c_int
     fn.argtypes = [ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int, ctypes.c_int, ctypes.c_void_p, ctypes.c_void_p,
