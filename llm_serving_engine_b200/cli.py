@@ -26,6 +26,7 @@ RANDOM_MODELS = {
     "tufevik": dict(vocab_size=260),     # the Tufevik design at a small size (``_tufevik_stand_in``)
     "sebudra": dict(vocab_size=260),     # the Sebudra design at a small size (``_sebudra_stand_in``)
     "kofipel": dict(vocab_size=260),     # the Kofipel design at a small size (``_kofipel_stand_in``)
+    "daferax": dict(vocab_size=260),     # the Daferax design at a small size (``_daferax_stand_in``)
     # the reference's ModelConfig.tiny (src/llmserve/config.py:34-44) over the byte tokenizer's vocabulary
     "tiny": dict(vocab_size=260, hidden_size=128, intermediate_size=352, num_hidden_layers=4, num_attention_heads=4,
                  num_key_value_heads=2, max_position_embeddings=1024, rope_theta=10000.0, rms_norm_eps=1e-6),
@@ -114,8 +115,24 @@ def _kofipel_stand_in(vocab_size: int) -> dict:
                        {"type": "channel_delta", "mixer": memory, "mlp": None}]}
 
 
+def _daferax_stand_in(vocab_size: int) -> dict:
+    """A small model of the Daferax design: two attentions whose values mix around a windowed latent attention, mixtures of
+    experts chosen within the best groups, the last layer without one."""
+    mlp = {"kind": "moe", "router": {"experts": 6, "top": 2, "scale": 2.0, "groups": {"count": 3, "keep": 2}},
+           "expert": {"ff": 64}, "shared": {"ff": 160}}
+    attention = {"heads": 4, "kv_heads": 2, "dim": 32, "vdim": 32, "scale": 32 ** -0.5, "v_mix": True,
+                 "rot": {"base": 10000.0, "dims": 32}}
+    latent = {"heads": 4, "dim": 24, "rot_dim": 8, "vdim": 24, "kv_rank": 40, "scale": 32 ** -0.5, "mask": {"size": 48},
+              "rot": {"base": 10000.0, "dims": 8, "scaling": {"factor": 4.0, "original": 256, "fast": 16.0, "slow": 1.0}}}
+    return {"architecture": "Daferax", "vocab": vocab_size, "width": 128, "norm": {"eps": 1e-6}, "max_position_embeddings": 1024,
+            "layers": [{"type": "attention", "mixer": attention, "mlp": mlp}, {"type": "latent_attention", "mixer": latent, "mlp": mlp},
+                       {"type": "attention", "mixer": attention, "mlp": None}]}
+
+
 def tiny_config(vocab_size: int = 260, name: str = "tiny") -> dict:
     """config.json of a random stand-in model."""
+    if name == "daferax":
+        return _daferax_stand_in(vocab_size)
     if name == "kofipel":
         return _kofipel_stand_in(vocab_size)
     if name == "sebudra":

@@ -9,21 +9,23 @@
 // afterwards.  So the attention itself is a multi-query attention with one shared "head" of keys of width DK whose
 // first DV columns are also the values.
 //
-// Three kernels:
+// Four kernels:
 //   * latent_prepare: per row of the step, from the fused down-projection: RMS norm of the query latent (if any),
 //     RMS norm of the key/value latent and rotation of the shared key part, both written into the cache row of the
 //     token; the per-head output gates sigmoid(g) (if any).
 //   * latent_query: sums the query projection's partial sums, copies the unrotated part of every head out and writes
 //     the rotated part behind the place where the folded part will go.
+//   * latent_front: the two above in one launch for layers without a query latent, whose one stacked projection holds queries,
+//     latent and gates: a block per token and head, one for the token's cached row, some for its gates.
 //   * latent_attention: the attention proper, any sizes, float32 arithmetic, storage float32 or bfloat16, keys in
 //     tiles of 32 and chunks of 256 counted from key 0 (a chunk per block with few rows, merged in order by a second
 //     kernel: the same bits either way), with an optional sink per head: a term exp(sink_h) in the softmax's
 //     denominator that has no key and no value.
 //
 // Rotation: the pair (2i, 2i+1), i < rot_dims / 2, by the angle position * freq[i]; cos and sin times `rot_factor`
-// (frequency scaling schemes are folded into freq and rot_factor by the host).  The angle is formed and brought into [-pi, pi] in
-// double precision, its sine and cosine taken in float32: a float32 product of a position in the thousands and a frequency near one is already off by 1e-4.
+// (frequency scaling schemes are folded into freq and rot_factor by the host; rotary.cuh has the precision of the angle).
 #include "common.cuh"
+#include "rotary.cuh"
 
 LSE_CHECK_DEFINE(lse_check_attention_latent)
 
@@ -33,15 +35,6 @@ __device__ __forceinline__ float lat_load(const TD* p, int n_partials, long long
   float v = 0.f;
   for (int i = 0; i < n_partials; ++i) v += to_f32<TD>(p[(size_t)i * partial_stride]);
   return v;
-}
-
-__device__ __forceinline__ void lat_sincos(int position, double freq, float factor, float& sn, float& cs) {
-  double angle = (double)position * freq;
-  angle -= 6.283185307179586 * rint(angle * 0.15915494309189535);    // into [-pi, pi], still in double
-  float s, c;
-  sincosf((float)angle, &s, &c);
-  sn = s * factor;
-  cs = c * factor;
 }
 
 constexpr int PREP_THREADS = 128;
@@ -112,7 +105,7 @@ latent_prepare_kernel(const TI* __restrict__ proj, int n_partials, long long par
       const float b = value(src + 2 * i + 1);
       if (2 * i + 1 < rot_dims) {
         float sn, cs;
-        lat_sincos(position, freq[i], rot_factor, sn, cs);
+        rotary_sincos(position, freq[i], rot_factor, sn, cs);
         dst[rank + 2 * i] = from_f32<TO>(a * cs - b * sn);
         dst[rank + 2 * i + 1] = from_f32<TO>(b * cs + a * sn);
       } else {
@@ -147,7 +140,7 @@ latent_query_kernel(const TI* __restrict__ proj, int n_partials, long long parti
     const float b = lat_load(src + 2 * i + 1, n_partials, partial_stride);
     if (2 * i + 1 < rot_dims) {
       float sn, cs;
-      lat_sincos(position, freq[i], rot_factor, sn, cs);
+      rotary_sincos(position, freq[i], rot_factor, sn, cs);
       dst[2 * i] = from_f32<TO>(a * cs - b * sn);
       dst[2 * i + 1] = from_f32<TO>(b * cs + a * sn);
     } else {
@@ -155,6 +148,61 @@ latent_query_kernel(const TI* __restrict__ proj, int n_partials, long long parti
       dst[2 * i + 1] = from_f32<TO>(b);
     }
   }
+}
+
+// Layers without a query latent: the row of `proj` is [queries (heads * (dim + rot)) | latent (rank) | shared key part (rot) |
+// gate columns], at q_off, kv_off, g_off.  grid (tokens, heads + 1 + blocks of gates).
+constexpr int GATES_A_BLOCK = 512;
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(PREP_THREADS)
+latent_front_kernel(const TI* __restrict__ proj, int n_partials, long long partial_stride, long long ld, int q_off, int heads,
+                    int dim, int rot, int rot_dims, const double* __restrict__ freq, float rot_factor, int kv_off, int rank,
+                    const float* __restrict__ kv_norm, float eps, const int* __restrict__ positions,
+                    const int* __restrict__ slot_mapping, TO* __restrict__ q_plain, TO* __restrict__ q_wide, int wide,
+                    TO* __restrict__ cache, int g_off, int gates, float* __restrict__ gate, int num_slots) {
+  extern __shared__ float row_s[];    // the cached row's sums (rank + rot floats)
+  __shared__ float scratch[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, part = blockIdx.y;
+  const int slot = LSE_CHECKED(slot_mapping[t], -1, num_slots, -1, LSE_CHECK_CACHE_SLOT);
+  if (slot < 0) return;      // a padding row
+  const TI* row = proj + (size_t)t * ld;
+  if (part > heads) {
+    const int begin = (part - heads - 1) * GATES_A_BLOCK, end = min(gates, begin + GATES_A_BLOCK);
+    for (int i = begin + threadIdx.x; i < end; i += PREP_THREADS)
+      gate[(size_t)t * gates + i] = 1.f / (1.f + expf(-sum_partials<TI>(row + g_off + i, n_partials, partial_stride)));
+    return;
+  }
+  const int position = positions[t];
+  const bool query = part < heads;
+  const TI* src = row + (query ? q_off + part * (dim + rot) + dim : kv_off + rank);     // the rotated part
+  TO* dst = query ? q_wide + ((size_t)t * heads + part) * wide + rank : cache + (size_t)slot * (rank + rot) + rank;
+  for (int i = threadIdx.x; i < (rot + 1) / 2; i += PREP_THREADS) {
+    const float a = sum_partials<TI>(src + 2 * i, n_partials, partial_stride);
+    if (2 * i + 1 >= rot) { dst[2 * i] = from_f32<TO>(a); continue; }
+    const float b = sum_partials<TI>(src + 2 * i + 1, n_partials, partial_stride);
+    float sn = 0.f, cs = 1.f;
+    if (2 * i + 1 < rot_dims) rotary_sincos(position, freq[i], rot_factor, sn, cs);
+    dst[2 * i] = from_f32<TO>(a * cs - b * sn);
+    dst[2 * i + 1] = from_f32<TO>(b * cs + a * sn);
+  }
+  if (query) {
+    src -= dim;
+    TO* plain = q_plain + ((size_t)t * heads + part) * dim;
+    for (int i = threadIdx.x; i < dim; i += PREP_THREADS) plain[i] = from_f32<TO>(sum_partials<TI>(src + i, n_partials, partial_stride));
+    return;
+  }
+  src -= rank;
+  dst -= rank;
+  float sq = 0.f;
+  for (int i = threadIdx.x; i < rank; i += PREP_THREADS) {
+    const float v = sum_partials<TI>(src + i, n_partials, partial_stride);
+    row_s[i] = v;
+    sq = fmaf(v, v, sq);
+  }
+  const float inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)rank + eps);
+  for (int i = threadIdx.x; i < rank; i += PREP_THREADS) dst[i] = from_f32<TO>((row_s[i] * inv) * kv_norm[i]);
 }
 
 // ------------------------------------------------------------------ the attention
@@ -203,8 +251,8 @@ latent_attention_kernel(const T* __restrict__ q, const T* __restrict__ cache, T*
   const int kv_begin = window > 0 ? max(0, ctx - window) : 0;
   int chunk_lo = kv_begin / CHUNK, chunk_hi = pos / CHUNK;
   if (SPLIT) {
-    const int mine = blockIdx.z / gchunks;
-    if (mine < chunk_lo || mine > chunk_hi) return;
+    const int mine = chunk_lo + blockIdx.z / gchunks;
+    if (mine > chunk_hi) return;
     chunk_lo = chunk_hi = mine;
   }
   const int* bt = block_tables + (size_t)seg * bt_stride;
@@ -305,7 +353,7 @@ latent_attention_kernel(const T* __restrict__ q, const T* __restrict__ cache, T*
 #pragma unroll
       for (int g = 0; g < GC; ++g) {
         if (g < gcount) {
-          float* dst = partials + (((size_t)t * n_q + g0 + g) * max_chunks + chunk) * (DV + 2);
+          float* dst = partials + (((size_t)t * n_q + g0 + g) * max_chunks + chunk - kv_begin / CHUNK) * (DV + 2);
 #pragma unroll
           for (int i = 0; i < DPT; ++i) {
             const int d = tid + i * THREADS;
@@ -356,7 +404,7 @@ latent_attention_merge_kernel(const float* __restrict__ partials, T* __restrict_
   for (int d = threadIdx.x; d < DV; d += blockDim.x) {
     float total = 0.f, M = -INFINITY, L = 0.f;
     for (int chunk = kv_begin / CHUNK; chunk <= pos / CHUNK; ++chunk) {
-      const float* part = src + (size_t)chunk * (DV + 2);
+      const float* part = src + (size_t)(chunk - kv_begin / CHUNK) * (DV + 2);
       float wa, wb;
       merge_chunk(M, L, part[DV], part[DV + 1], wa, wb);
       total = fmaf(part[d], wb, total * wa);
@@ -416,6 +464,31 @@ extern "C" int lse_latent_query(const void* proj, int in_dtype, int n_partials, 
   LSE_LAUNCH_CHECK();
 }
 
+// latent_prepare and latent_query in one launch (no query latent); gate float32 [tokens, gates] or null.
+extern "C" int lse_latent_front(const void* proj, int in_dtype, int n_partials, long long partial_stride, long long ld, int q_off,
+                                int heads, int dim, int rot, int rot_dims, const double* freq, float rot_factor, int kv_off,
+                                int rank, const float* kv_norm, float eps, const int* positions, const int* slot_mapping,
+                                void* q_plain, void* q_wide, int wide, void* cache, int out_dtype, int g_off, int gates,
+                                float* gate, int tokens, int num_slots, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (rot_dims > rot || (rot_dims & 1) || heads <= 0 || rank <= 0 || dim < 0 || wide < rank + rot || n_partials < 1 || !kv_norm) return LSE_ERR_BAD_ARGUMENT;
+  const long long parts = (long long)heads + 1 + (gate ? (gates + GATES_A_BLOCK - 1) / GATES_A_BLOCK : 0);
+  const size_t smem = (size_t)rank * sizeof(float);
+  if (parts > 65535 || smem > 40 * 1024) return LSE_ERR_TOO_LARGE;
+  const dim3 grid(tokens, (unsigned)parts);
+#define LSE_LF_CASE(TI, TO)                                                                                              \
+  lse_launch(latent_front_kernel<TI, TO>, grid, PREP_THREADS, smem, stream, (const TI*)proj, n_partials, partial_stride, ld, \
+             q_off, heads, dim, rot, rot_dims, freq, rot_factor, kv_off, rank, kv_norm, eps, positions, slot_mapping,    \
+             (TO*)q_plain, (TO*)q_wide, wide, (TO*)cache, g_off, gates, gate, num_slots);
+  const bool i32 = in_dtype == LSE_DTYPE_F32, o32 = out_dtype == LSE_DTYPE_F32;
+  if (i32 && o32) LSE_LF_CASE(float, float)
+  else if (i32 && !o32) LSE_LF_CASE(float, __nv_bfloat16)
+  else if (!i32 && !o32) LSE_LF_CASE(__nv_bfloat16, __nv_bfloat16)
+  else return LSE_ERR_BAD_ARGUMENT;
+#undef LSE_LF_CASE
+  LSE_LAUNCH_CHECK();
+}
+
 extern "C" int lse_latent_attention_chunk(void) { return CHUNK; }
 
 // The merge alone: adds up the chunks that a split kernel (this file's, or the tensor-core one) left in `partials`.
@@ -437,7 +510,7 @@ extern "C" int lse_latent_attention_merge(const float* partials, void* out, int 
 }
 
 // partials != null: a block per chunk of a row, merged by a second kernel (few rows); partials holds
-// tokens * n_q * max_chunks * (DV + 2) floats.
+// tokens * n_q * max_chunks * (DV + 2) floats, a row's chunks counted from the first that its window touches.
 extern "C" int lse_latent_attention(const void* q, const void* cache, void* out, int dtype, const int* block_tables,
                                     int bt_stride, const int* segment_of_token, const int* positions,
                                     const float* sink, int tokens, int n_q, int DK, int DV, int page_size, float scale,
@@ -451,7 +524,7 @@ extern "C" int lse_latent_attention(const void* q, const void* cache, void* out,
   const int gchunks = (n_q + GC - 1) / GC;
   const bool split = partials != nullptr;
   if (split && (max_chunks <= 0 || (long long)gchunks * max_chunks > 65535 ||
-                (long long)max_chunks * CHUNK < (long long)bt_stride * page_size))
+                ((long long)max_chunks * CHUNK < (long long)bt_stride * page_size && (window <= 0 || max_chunks < (window - 1) / CHUNK + 2))))
     return LSE_ERR_BAD_ARGUMENT;
   dim3 grid(tokens, 1, split ? gchunks * max_chunks : gchunks);
   const dim3 merge_grid(tokens, n_q);

@@ -11,7 +11,8 @@
 //            the product, V the first DV columns of the very rows that were the keys
 // With few rows (decoding) every chunk of 256 keys has a block of its own (blockIdx.z) that leaves O, m and l of
 // its chunk in the layout of attention_latent.cu's split kernel, whose merge kernel adds the chunks up and lets
-// the sink join the denominator.  With many rows a block walks all its keys and finishes the row itself.
+// the sink join the denominator.  window > 0: a row reads its last `window` keys only; a row's chunks are then numbered from
+// the one that holds the first key of its window, and the grid has as many as a tile's window can touch.  With many rows a block walks all its keys and finishes the row itself.
 #include "common.cuh"
 
 LSE_CHECK_DEFINE(lse_check_attention_latent_mma)
@@ -68,7 +69,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
                             const int* __restrict__ segment_start, const int* __restrict__ segment_first_position,
                             const float* __restrict__ sink, int num_segments, int n_q, int DK, int DV, int page_size,
                             float scale, int num_pages, float* __restrict__ partials, int max_chunks,
-                            int tokens_per_tile, int heads_per_block) {
+                            int tokens_per_tile, int heads_per_block, int window) {
   extern __shared__ __align__(16) unsigned char smem[];
   __shared__ int tile_slot[3];
   pdl_launch_dependents();
@@ -95,11 +96,13 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   const int ctx = first_pos + tile_tokens;                        // keys that the tile's last token sees
   const int h0 = blockIdx.y * heads_per_block;
   const int heads_here = min(heads_per_block, n_q - h0);
-  int key_lo = 0, key_hi = ctx;
+  // window > 0: the first key that any row of the tile reads; keys before it are not fetched (their pages may be given back)
+  int key_lo = window > 0 ? max(0, first_pos + 1 - window) : 0, key_hi = ctx;
+  const int chunk = key_lo / CHUNK + blockIdx.z;                  // split: the tile's chunks from its first one on
   if (split) {
-    key_lo = blockIdx.z * CHUNK;
-    key_hi = min(ctx, key_lo + CHUNK);
-    if (key_lo >= ctx) return;
+    key_lo = max(key_lo, chunk * CHUNK);
+    key_hi = min(ctx, (chunk + 1) * CHUNK);
+    if (chunk * CHUNK >= ctx) return;
   }
   const int* bt = block_tables + (size_t)seg * bt_stride;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -118,12 +121,12 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     const __nv_bfloat16* src = valid ? q + ((size_t)(first_row + tok) * n_q + h0 + hh) * DK + c * 8 : q;
     cp_async16(smem_u32(q_s + (size_t)r * dks + c * 8), src, valid);
   }
-  auto load_keys = [&](int base, int buffer) {    // keys base .. base + KEYS - 1 (zeros beyond key_hi)
+  auto load_keys = [&](int base, int buffer) {    // keys base .. base + KEYS - 1 (zeros outside [key_lo, key_hi))
     __syncthreads();                              // off_s of the tile before has been used
     if (tid < KEYS) {
       const int j = base + tid;
       long long off = -1;
-      if (j < key_hi) {
+      if (j >= key_lo && j < key_hi) {
         const int page = LSE_CHECKED(bt[j / page_size], 0, num_pages, 0, LSE_CHECK_TABLE_ENTRY);
         off = ((long long)page * page_size + (j % page_size)) * DK;
       }
@@ -178,7 +181,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
         for (int i = 0; i < 4; ++i) {
           const int r = mi * 16 + (lane >> 2) + (i >> 1) * 8, c = warp * 8 + (lane & 3) * 2 + (i & 1);
           const int j = base + c;
-          s_s[r * SS + c] = (j <= pos_s[r] && j >= key_lo && j < key_hi) ? s[mi][i] * scale : -INFINITY;
+          s_s[r * SS + c] = (j <= pos_s[r] && j >= key_lo && j < key_hi && (window <= 0 || j > pos_s[r] - window)) ? s[mi][i] * scale : -INFINITY;
         }
     }
     __syncthreads();
@@ -257,8 +260,10 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
       const int tok = r / heads_per_block, head = h0 + r % heads_per_block;
       const size_t row = (size_t)(first_row + tok) * n_q + head;
       if (split) {
-        if (pos_s[r] < key_lo) continue;     // the row sees no key of this chunk; the merge does not read it
-        float* dst = partials + (row * max_chunks + blockIdx.z) * (DV + 2);
+        const int row_first = window > 0 ? max(0, pos_s[r] + 1 - window) : 0;
+        // the row sees no key of this chunk: the merge does not read it
+        if (pos_s[r] < key_lo || (chunk + 1) * CHUNK <= row_first) continue;
+        float* dst = partials + (row * max_chunks + chunk - row_first / CHUNK) * (DV + 2);   // a row's chunks from its own first one
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt) {
           const int c = col_base + nt * 8 + (lane & 3) * 2;
@@ -299,15 +304,16 @@ extern "C" int lse_latent_attention_mma_supported(int DK, int DV) {
 extern "C" int lse_latent_attention_mma(const void* q, const void* cache, void* out, const int* block_tables,
                                         int bt_stride, const int* segment_start, const int* segment_first_position,
                                         const float* sink, int tokens, int num_segments, int n_q, int DK, int DV,
-                                        int page_size, float scale, int num_pages, float* partials, int max_chunks,
-                                        cudaStream_t stream) {
+                                        int page_size, float scale, int window, int num_pages, float* partials,
+                                        int max_chunks, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (!lse_latent_attention_mma_supported(DK, DV) || n_q <= 0 || page_size <= 0 || num_segments <= 0) return LSE_ERR_BAD_ARGUMENT;
   const int heads_per_block = min(n_q, ROWS);
   const int tokens_per_tile = max(1, ROWS / heads_per_block);
   const int tiles = min(tokens, tokens / tokens_per_tile + num_segments);       // an upper bound
   const bool split = partials != nullptr;
-  if (split && (max_chunks <= 0 || max_chunks > 65535 || (long long)max_chunks * CHUNK < (long long)bt_stride * page_size))
+  if (split && (max_chunks <= 0 || max_chunks > 65535 ||
+                ((long long)max_chunks * CHUNK < (long long)bt_stride * page_size && (window <= 0 || max_chunks < (window + ROWS - 2) / CHUNK + 2))))
     return LSE_ERR_BAD_ARGUMENT;
   dim3 grid(tiles, (n_q + heads_per_block - 1) / heads_per_block, split ? max_chunks : 1);
   const size_t smem = Layout(DK).total;
@@ -324,7 +330,7 @@ extern "C" int lse_latent_attention_mma(const void* q, const void* cache, void* 
     lse_launch(latent_attention_mma_kernel<NT>, grid, THREADS, smem, stream, (const __nv_bfloat16*)q,              \
                (const __nv_bfloat16*)cache, (__nv_bfloat16*)out, block_tables, bt_stride, segment_start,           \
                segment_first_position, sink, num_segments, n_q, DK, DV, page_size, scale, num_pages, partials,     \
-               max_chunks, tokens_per_tile, heads_per_block);                                                      \
+               max_chunks, tokens_per_tile, heads_per_block, window);                                                      \
   }
   if (per_warp <= 1) LSE_LMMA_CASE(1)
   else if (per_warp <= 2) LSE_LMMA_CASE(2)

@@ -69,7 +69,7 @@ attention_scored_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
                         const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink,
                         int n_q, int n_kv, int dk, int dv, int n_values, int page_size, float scale, int num_pages,
                         int num_segments, float* __restrict__ partials, int max_chunks, int window, int keep_first, float cap,
-                        const float* __restrict__ head_bias) {
+                        const float* __restrict__ head_bias, const float* __restrict__ out_gate) {
   extern __shared__ float smem[];
   pdl_launch_dependents();
   pdl_wait();
@@ -255,8 +255,9 @@ attention_scored_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
   for (int g = 0; g < GC; ++g) {
     if (g < gcount) {
       float l = L[g];
-      const float w = sink ? add_sink(M[g], l, sink[first_head + g]) : 1.f;
+      float w = sink ? add_sink(M[g], l, sink[first_head + g]) : 1.f;
       if (head_bias) l = 1.f;
+      if (out_gate) w *= out_gate[(size_t)t * n_q + first_head + g];
 #pragma unroll
       for (int i = 0; i < DPT; ++i) {
         const int d = tid + i * THREADS;
@@ -273,7 +274,7 @@ __global__ void __launch_bounds__(MAX_D)
 attention_scored_merge_kernel(const float* __restrict__ partials, TO* __restrict__ out,
                               const int* __restrict__ segment_of_token, const int* __restrict__ positions,
                               const float* __restrict__ sink, int n_values, int dv, int max_chunks, int num_segments,
-                              int window, int keep_first, int unnormalised) {
+                              int window, int keep_first, int unnormalised, const float* __restrict__ out_gate) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, item = blockIdx.y, d = threadIdx.x;
@@ -290,8 +291,9 @@ attention_scored_merge_kernel(const float* __restrict__ partials, TO* __restrict
     merge_parts(M, L, part[dv], part[dv + 1], wa, wb);
     total = fmaf(part[d], wb, total * wa);
   }
-  const float w = sink ? add_sink(M, L, sink[item / n_values]) : 1.f;
+  float w = sink ? add_sink(M, L, sink[item / n_values]) : 1.f;
   if (unnormalised) L = 1.f;
+  if (out_gate) w *= out_gate[(size_t)t * (gridDim.y / n_values) + item / n_values];
   out[((size_t)t * gridDim.y + item) * dv + d] = from_f32<TO>(total * w / L);
 }
 
@@ -422,7 +424,7 @@ int launch_scored(const void* q, const void* k_cache, const void* v_cache, void*
                   int bt_stride, const int* segment_of_token, const int* positions, const float* r1, const float* r2,
                   const float* sink, int tokens, int n_q, int n_kv, int dk, int dv, int n_values, int page_size,
                   float scale, int num_pages, int num_segments, float* partials, int max_chunks, int window, int keep_first,
-                  float cap, const float* head_bias, cudaStream_t stream) {
+                  float cap, const float* head_bias, const float* out_gate, cudaStream_t stream) {
   const int group = n_q / n_kv;
   const int gchunks = (group + GC - 1) / GC;
   const bool split = partials != nullptr;
@@ -441,14 +443,16 @@ int launch_scored(const void* q, const void* k_cache, const void* v_cache, void*
   if (split) {
     lse_launch(attention_scored_kernel<T, TO, true>, grid, THREADS, smem, stream, (const T*)q, (const T*)k_cache,
                (const T*)v_cache, (TO*)out, block_tables, bt_stride, segment_of_token, positions, r1, r2, sink, n_q, n_kv,
-               dk, dv, n_values, page_size, scale, num_pages, num_segments, partials, max_chunks, window, keep_first, cap, head_bias);
+               dk, dv, n_values, page_size, scale, num_pages, num_segments, partials, max_chunks, window, keep_first, cap, head_bias,
+               (const float*)nullptr);
     lse_launch(attention_scored_merge_kernel<TO>, dim3(tokens, n_q * n_values), ((dv + 31) / 32) * 32, 0, stream,
                (const float*)partials, (TO*)out, segment_of_token, positions, sink, n_values, dv, max_chunks,
-               num_segments, window, keep_first, (int)(head_bias != nullptr));
+               num_segments, window, keep_first, (int)(head_bias != nullptr), out_gate);
   } else {
     lse_launch(attention_scored_kernel<T, TO, false>, grid, THREADS, smem, stream, (const T*)q, (const T*)k_cache,
                (const T*)v_cache, (TO*)out, block_tables, bt_stride, segment_of_token, positions, r1, r2, sink, n_q, n_kv,
-               dk, dv, n_values, page_size, scale, num_pages, num_segments, (float*)nullptr, 0, window, keep_first, cap, head_bias);
+               dk, dv, n_values, page_size, scale, num_pages, num_segments, (float*)nullptr, 0, window, keep_first, cap, head_bias,
+               out_gate);
   }
   return (int)cudaGetLastError();
 }
@@ -462,15 +466,17 @@ extern "C" int lse_attention_scored_chunk(void) { return CHUNK; }
 // (dv + 2) floats, and max_chunks chunks cover the longest context that the block tables can describe.
 // window > 0: a row reads its last `window` keys only, and with keep_first > 0 the request's first keep_first; cap > 0: scores capped by cap * tanh(s / cap); head_bias (float32
 // [n_q] or null): weights sigmoid(s + head_bias_h) without a softmax (no sink then).
+// out_gate (float32 [T, n_q] or null; not with cross): head h's output of row t is multiplied by out_gate[t, h].
 extern "C" int lse_attention_scored_windowed(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype,
                                              int out_f32, const int* block_tables, int bt_stride,
                                              const int* segment_of_token, const int* positions, const float* r1,
                                              const float* r2, const float* sink, int tokens, int n_q, int n_kv, int dk,
                                              int dv, int cross, int page_size, float scale, int num_pages,
                                              int num_segments, float* partials, int max_chunks, int window,
-                                             int keep_first, float cap, const float* head_bias, cudaStream_t stream) {
+                                             int keep_first, float cap, const float* head_bias, const float* out_gate,
+                                             cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if ((head_bias && sink) || keep_first < 0) return LSE_ERR_BAD_ARGUMENT;
+  if ((head_bias && sink) || keep_first < 0 || (out_gate && cross)) return LSE_ERR_BAD_ARGUMENT;
   if (window <= 0) keep_first = 0;     // every key is read anyway
   if (dk <= 0 || dk > MAX_D || dv <= 0 || dv > MAX_D || n_kv <= 0 || n_q % n_kv || page_size <= 0 || (!r1) != (!r2))
     return LSE_ERR_BAD_ARGUMENT;
@@ -481,7 +487,8 @@ extern "C" int lse_attention_scored_windowed(const void* q, const void* k_cache,
   if ((long long)(partials ? max_chunks : 1) * n_values * gchunks > 65535 || n_kv > 65535 || n_q * n_values > 65535)
     return LSE_ERR_TOO_LARGE;
 #define LSE_SCORED_ARGS q, k_cache, v_cache, out, block_tables, bt_stride, segment_of_token, positions, r1, r2, sink, tokens, \
-  n_q, n_kv, dk, dv, n_values, page_size, scale, num_pages, num_segments, partials, max_chunks, window, keep_first, cap, head_bias, stream
+  n_q, n_kv, dk, dv, n_values, page_size, scale, num_pages, num_segments, partials, max_chunks, window, keep_first, cap, head_bias, \
+  out_gate, stream
   if (dtype == LSE_DTYPE_F32) return launch_scored<float, float>(LSE_SCORED_ARGS);
   if (dtype == LSE_DTYPE_BF16 && out_f32) return launch_scored<__nv_bfloat16, float>(LSE_SCORED_ARGS);
   if (dtype == LSE_DTYPE_BF16) return launch_scored<__nv_bfloat16, __nv_bfloat16>(LSE_SCORED_ARGS);
@@ -497,17 +504,17 @@ extern "C" int lse_attention_scored(const void* q, const void* k_cache, const vo
                                     cudaStream_t stream) {
   return lse_attention_scored_windowed(q, k_cache, v_cache, out, dtype, out_f32, block_tables, bt_stride, segment_of_token,
                                        positions, r1, r2, sink, tokens, n_q, n_kv, dk, dv, cross, page_size, scale,
-                                       num_pages, num_segments, partials, max_chunks, 0, 0, 0.f, nullptr, stream);
+                                       num_pages, num_segments, partials, max_chunks, 0, 0, 0.f, nullptr, nullptr, stream);
 }
 
 // The second half of a launch with partials, for kernels of other files that leave partials in the same layout
 // ([t][head][value slot][chunk][dv + 2]: sums, maximum, total): out [T, n_q, n_values, dv] in bfloat16 or float32.
-// window, keep_first, unnormalised: as the launch that left the partials had them (chunks before the window hold nothing).
+// window, keep_first, unnormalised, out_gate: as the launch that left the partials had them (chunks before the window hold nothing).
 extern "C" int lse_attention_scored_merge_windowed(const float* partials, void* out, int out_dtype,
                                                    const int* segment_of_token, const int* positions, const float* sink,
                                                    int tokens, int n_q, int n_values, int dv, int max_chunks,
                                                    int num_segments, int window, int keep_first, int unnormalised,
-                                                   cudaStream_t stream) {
+                                                   const float* out_gate, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (dv <= 0 || dv > MAX_D || n_q * n_values > 65535 || max_chunks <= 0 || keep_first < 0) return LSE_ERR_BAD_ARGUMENT;
   if (window <= 0) keep_first = 0;
@@ -515,10 +522,10 @@ extern "C" int lse_attention_scored_merge_windowed(const float* partials, void* 
   const int threads = ((dv + 31) / 32) * 32;
   if (out_dtype == LSE_DTYPE_F32)
     lse_launch(attention_scored_merge_kernel<float>, grid, threads, 0, stream, partials, (float*)out, segment_of_token,
-               positions, sink, n_values, dv, max_chunks, num_segments, window, keep_first, unnormalised);
+               positions, sink, n_values, dv, max_chunks, num_segments, window, keep_first, unnormalised, out_gate);
   else if (out_dtype == LSE_DTYPE_BF16)
     lse_launch(attention_scored_merge_kernel<__nv_bfloat16>, grid, threads, 0, stream, partials, (__nv_bfloat16*)out,
-               segment_of_token, positions, sink, n_values, dv, max_chunks, num_segments, window, keep_first, unnormalised);
+               segment_of_token, positions, sink, n_values, dv, max_chunks, num_segments, window, keep_first, unnormalised, out_gate);
   else
     return LSE_ERR_BAD_ARGUMENT;
   LSE_LAUNCH_CHECK();
@@ -528,7 +535,7 @@ extern "C" int lse_attention_scored_merge(const float* partials, void* out, int 
                                           const int* positions, const float* sink, int tokens, int n_q, int n_values,
                                           int dv, int max_chunks, int num_segments, cudaStream_t stream) {
   return lse_attention_scored_merge_windowed(partials, out, out_dtype, segment_of_token, positions, sink, tokens, n_q,
-                                             n_values, dv, max_chunks, num_segments, 0, 0, 0, stream);
+                                             n_values, dv, max_chunks, num_segments, 0, 0, 0, nullptr, stream);
 }
 
 // wide [T, n_q, n_values, dv] (n_values = n_kv when cross, else 1) in float32, or in bfloat16 (wide_bf16; only shapes

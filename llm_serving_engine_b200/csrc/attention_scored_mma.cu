@@ -1,5 +1,6 @@
 // The attention of attention_scored.cu (distance penalty, sink, values of every group) on the tensor cores, for
-// bfloat16 and head sizes that are multiples of 16 (keys and values of one size: 32, 48, 64, 96 or 128).
+// bfloat16 and head sizes that are multiples of 16 (keys and values of one size: 32, 48, 64, 96 or 128, and some pairs of
+// two sizes; see lse_attention_scored_mma_supported).
 //
 // One block = (tile of consecutive rows of one request, key head, value slot[, chunk of keys]).  The 64 rows of its
 // score matrix are (row, query head of the group) pairs, so the keys of a key head are loaded once for all its query
@@ -15,6 +16,8 @@
 // request's first keys are read by every row behind them as well; the walk then takes the tiles that hold them first and
 // goes on with the tiles of the window.  cap > 0: scores are capped by
 // cap * tanh(s / cap).  head_bias: no softmax, a key's weight is sigmoid(s + head_bias_h) and the sums are not divided.
+//
+// out_gate (per row and head, or null) multiplies a head's finished output (without partials here, else in the merge).
 //
 // With `partials` the keys of a tile of rows are cut into chunks of 256 (counted from key 0) with a block each, which
 // leaves (sums, max, total) per row, head, value slot and chunk in the layout of attention_scored.cu; that file's
@@ -44,7 +47,8 @@ attention_scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
                             const int* __restrict__ segment_first_pos, int num_segments, const float* __restrict__ r1,
                             const float* __restrict__ r2, const float* __restrict__ sink, int n_q, int n_kv,
                             int n_values, int page_size, float scale_log2e, int rows_per_tile, int num_pages,
-                            int max_chunks, int window, int keep_first, float cap, const float* __restrict__ head_bias) {
+                            int max_chunks, int window, int keep_first, float cap, const float* __restrict__ head_bias,
+                            const float* __restrict__ out_gate) {
   constexpr int CHK = DK / 8, CHV = DV / 8;
   constexpr int K_BYTES = tile_bytes<DK>(BN), V_BYTES = tile_bytes<DV>(BN);
   extern __shared__ __align__(128) unsigned char smem[];
@@ -317,7 +321,11 @@ attention_scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     l0 = l0 * w0 + fast_exp2(sa - na);
     l1 = l1 * w1 + fast_exp2(sb - nb);
   }
-  const float inv0 = unnormalised ? 1.f : w0 / l0, inv1 = unnormalised ? 1.f : w1 / l1;
+  float inv0 = unnormalised ? 1.f : w0 / l0, inv1 = unnormalised ? 1.f : w1 / l1;
+  if (out_gate) {
+    if (rla < nrows) inv0 *= out_gate[(size_t)(row_base + rla) * n_q + head_a];
+    if (rlb < nrows) inv1 *= out_gate[(size_t)(row_base + rlb) * n_q + head_b];
+  }
 #pragma unroll
   for (int i = 0; i < DV / 8; ++i) {
     const int d = i * 8 + (lane & 3) * 2;
@@ -334,19 +342,19 @@ attention_scored_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   }
 }
 
-template <int D>
+template <int DK, int DV>
 int launch_scored_mma(const void* q, const void* kc, const void* vc, void* out, int out_is_f32, float* partials,
                       const int* block_tables, int bt_stride, const int* segment_start, const int* segment_first_pos,
                       int num_segments, const float* r1, const float* r2, const float* sink, int tokens, int n_q, int n_kv,
                       int n_values, int page_size, float scale, int num_pages, int max_chunks, int window, int keep_first,
-                      float cap, const float* head_bias, cudaStream_t stream) {
+                      float cap, const float* head_bias, const float* out_gate, cudaStream_t stream) {
   const int group = n_q / n_kv;
   const int rows_per_tile = BM / group;
-  const size_t tiles_bytes = (size_t)tile_bytes<D>(BM) + 2 * (size_t)(tile_bytes<D>(BN) + tile_bytes<D>(BN));
+  const size_t tiles_bytes = (size_t)tile_bytes<DK>(BM) + 2 * (size_t)(tile_bytes<DK>(BN) + tile_bytes<DV>(BN));
   const size_t smem = tiles_bytes + sizeof(float) * (size_t)group * (BN + rows_per_tile);
   static bool configured = false;
   if (!configured) {   // room for the largest penalty table (64 heads a group) once
-    cudaError_t err = cudaFuncSetAttribute(attention_scored_mma_kernel<D, D>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t err = cudaFuncSetAttribute(attention_scored_mma_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                            (int)(tiles_bytes + sizeof(float) * BM * (BN + 1)));
     if (err != cudaSuccess) return (int)err;
     configured = true;
@@ -355,18 +363,21 @@ int launch_scored_mma(const void* q, const void* kc, const void* vc, void* out, 
   const long long depth = (long long)n_values * (partials ? max_chunks : 1);
   if (depth > 65535 || n_kv > 65535) return LSE_ERR_TOO_LARGE;
   dim3 grid(tiles, n_kv, (unsigned)depth);
-  lse_launch(attention_scored_mma_kernel<D, D>, grid, 128, smem, stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)kc,
+  lse_launch(attention_scored_mma_kernel<DK, DV>, grid, 128, smem, stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)kc,
              (const __nv_bfloat16*)vc, out_is_f32 ? (__nv_bfloat16*)nullptr : (__nv_bfloat16*)out,
              out_is_f32 ? (float*)out : (float*)nullptr, partials, block_tables, bt_stride, segment_start, segment_first_pos,
              num_segments, r1, r2, sink, n_q, n_kv, n_values, page_size, scale * LOG2E, rows_per_tile, num_pages, max_chunks,
-             window, keep_first, cap, head_bias);
+             window, keep_first, cap, head_bias, out_gate);
   return (int)cudaGetLastError();
 }
 }  // namespace
 
 // Whether the tensor-core kernel takes this shape (else the caller uses the general kernel).
 extern "C" int lse_attention_scored_mma_supported(int dk, int dv, int n_q, int n_kv) {
-  if (dk != dv || (dk != 32 && dk != 48 && dk != 64 && dk != 96 && dk != 128)) return 0;
+  const bool equal = dk == dv && (dk == 32 || dk == 48 || dk == 64 || dk == 96 || dk == 128);
+  const bool narrow = (dv == 32 && (dk == 64 || dk == 96 || dk == 128)) || (dv == 64 && (dk == 96 || dk == 128)) || (dv == 96 && dk == 128);
+  const bool wide = dk == 64 && dv == 128;
+  if (!equal && !narrow && !wide) return 0;
   if (n_kv <= 0 || n_q % n_kv) return 0;
   return (n_q / n_kv) <= BM ? 1 : 0;
 }
@@ -380,9 +391,9 @@ extern "C" int lse_attention_scored_mma_windowed(const void* q, const void* k_ca
                                                  const float* r1, const float* r2, const float* sink, int tokens, int n_q,
                                                  int n_kv, int dk, int dv, int cross, int page_size, float scale,
                                                  int num_pages, float* partials, int max_chunks, int window, int keep_first, float cap,
-                                                 const float* head_bias, cudaStream_t stream) {
+                                                 const float* head_bias, const float* out_gate, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if ((head_bias && sink) || keep_first < 0) return LSE_ERR_BAD_ARGUMENT;
+  if ((head_bias && sink) || keep_first < 0 || (out_gate && cross)) return LSE_ERR_BAD_ARGUMENT;
   if (window <= 0) keep_first = 0;
   if (!lse_attention_scored_mma_supported(dk, dv, n_q, n_kv) || page_size <= 0 || (!r1) != (!r2)) return LSE_ERR_BAD_ARGUMENT;
   if (partials && (max_chunks <= 0 || (long long)max_chunks * CHUNK < (long long)bt_stride * page_size))
@@ -390,13 +401,21 @@ extern "C" int lse_attention_scored_mma_windowed(const void* q, const void* k_ca
   const int n_values = cross ? n_kv : 1;
 #define LSE_SCORED_MMA_ARGS q, k_cache, v_cache, out, out_f32, partials, block_tables, bt_stride, segment_start, \
   segment_first_pos, num_segments, r1, r2, sink, tokens, n_q, n_kv, n_values, page_size, scale, num_pages, max_chunks, \
-  window, keep_first, cap, head_bias, stream
-  switch (dk) {
-    case 32: return launch_scored_mma<32>(LSE_SCORED_MMA_ARGS);
-    case 48: return launch_scored_mma<48>(LSE_SCORED_MMA_ARGS);
-    case 64: return launch_scored_mma<64>(LSE_SCORED_MMA_ARGS);
-    case 96: return launch_scored_mma<96>(LSE_SCORED_MMA_ARGS);
-    default: return launch_scored_mma<128>(LSE_SCORED_MMA_ARGS);
+  window, keep_first, cap, head_bias, out_gate, stream
+  switch (dk * 1000 + dv) {
+    case 32032: return launch_scored_mma<32, 32>(LSE_SCORED_MMA_ARGS);
+    case 48048: return launch_scored_mma<48, 48>(LSE_SCORED_MMA_ARGS);
+    case 64064: return launch_scored_mma<64, 64>(LSE_SCORED_MMA_ARGS);
+    case 96096: return launch_scored_mma<96, 96>(LSE_SCORED_MMA_ARGS);
+    case 128128: return launch_scored_mma<128, 128>(LSE_SCORED_MMA_ARGS);
+    case 64032: return launch_scored_mma<64, 32>(LSE_SCORED_MMA_ARGS);
+    case 96032: return launch_scored_mma<96, 32>(LSE_SCORED_MMA_ARGS);
+    case 128032: return launch_scored_mma<128, 32>(LSE_SCORED_MMA_ARGS);
+    case 96064: return launch_scored_mma<96, 64>(LSE_SCORED_MMA_ARGS);
+    case 128064: return launch_scored_mma<128, 64>(LSE_SCORED_MMA_ARGS);
+    case 128096: return launch_scored_mma<128, 96>(LSE_SCORED_MMA_ARGS);
+    case 64128: return launch_scored_mma<64, 128>(LSE_SCORED_MMA_ARGS);
+    default: return LSE_ERR_BAD_ARGUMENT;
   }
 #undef LSE_SCORED_MMA_ARGS
 }
@@ -409,5 +428,5 @@ extern "C" int lse_attention_scored_mma(const void* q, const void* k_cache, cons
                                         cudaStream_t stream) {
   return lse_attention_scored_mma_windowed(q, k_cache, v_cache, out, out_f32, block_tables, bt_stride, segment_start,
                                            segment_first_pos, num_segments, r1, r2, sink, tokens, n_q, n_kv, dk, dv, cross,
-                                           page_size, scale, num_pages, partials, max_chunks, 0, 0, 0.f, nullptr, stream);
+                                           page_size, scale, num_pages, partials, max_chunks, 0, 0, 0.f, nullptr, nullptr, stream);
 }

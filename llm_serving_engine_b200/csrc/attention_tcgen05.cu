@@ -105,7 +105,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                        const int* __restrict__ segment_first_pos, int num_segments, int n_q, int n_kv, int page_size,
                        float scale_log2e, int num_pages, int skip_single, int parts, float* __restrict__ scratch,
                        int* __restrict__ counters, const float* __restrict__ r1, const float* __restrict__ r2,
-                       const float* __restrict__ sink, int n_values, float cap) {
+                       const float* __restrict__ sink, int n_values, float cap,
+                       const float* __restrict__ out_gate) {
   constexpr bool PEN = MODE == 1, SIG = MODE == 2;
   constexpr int HALVES = D / 64;
   constexpr uint32_t Q_BYTES = HALVES * HALF_BYTES, KV_BYTES = HALVES * HALF_BYTES, P_BYTES = 2 * HALF_BYTES;
@@ -493,6 +494,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         inv = w_rows / fmaf(l_all, w_rows, exp2_fast(sink2 - m_fin));
       }
     }
+    const float gate = out_gate && row < nrows ? out_gate[(size_t)(row_base + row) * n_q + head] : 1.0f;
+    if (!shared) inv *= gate;
     const float w0 = (g == 0 ? w_mine : w_other) * inv, w1 = (g == 0 ? w_other : w_mine) * inv;
     // both groups' last products must have landed (group 1 has none when there is a single tile)
     const int n0 = (n_local + 1) / 2, n1 = n_local / 2;
@@ -578,7 +581,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
           if (p < sharing) sum = fmaf(__ldcg(parts_base + (size_t)p * PART_FLOATS + BM * D + BM + row), weight[p], sum);
         }
         if (sink) sum += exp2_fast(sink2 - m_tile);
-        const float inv_sum = SIG ? 1.0f : 1.0f / sum;
+        const float inv_sum = (SIG ? 1.0f : 1.0f / sum) * gate;
         if (row < nrows) {
 #pragma unroll 2
           for (int c = 0; c < OD; c += 8) {
@@ -619,7 +622,8 @@ int launch_prefill_tc(const void* q, const void* kc, const void* vc, void* out, 
                       const int* segment_start, const int* segment_first_pos, int num_segments, int tokens,
                       long long num_pages, int n_q, int n_kv, int page_size, float scale, int skip_single,
                       int max_portions, float* scratch, int* counters, long long scratch_slots, const float* r1,
-                      const float* r2, const float* sink, int n_values, cudaStream_t stream, float cap = 0.f) {
+                      const float* r2, const float* sink, int n_values, cudaStream_t stream, float cap = 0.f,
+                      const float* out_gate = nullptr) {
   const size_t smem = attn_tc_smem<D>();
   static bool configured = false;
   if (!configured) {
@@ -655,7 +659,7 @@ int launch_prefill_tc(const void* q, const void* kc, const void* vc, void* out, 
   cudaError_t err = lse_launch(attn_prefill_tc_kernel<D, MODE>, grid, THREADS, smem, stream, map_q, map_k, map_v,
                                (__nv_bfloat16*)out, block_tables, bt_stride, segment_start, segment_first_pos,
                                num_segments, n_q, n_kv, page_size, scale * LOG2E, (int)num_pages, skip_single, parts,
-                               scratch, counters, r1, r2, sink, n_values, cap);
+                               scratch, counters, r1, r2, sink, n_values, cap, out_gate);
   if (err != cudaSuccess) return (int)err;
   return (int)cudaGetLastError();
 }
@@ -723,21 +727,22 @@ extern "C" int lse_paged_attention_prefill_tc(const void* q, const void* k_cache
 
 // The same kernel with learned changes to its scores or weights (see attention_scored.cu): r1, r2 (together, float32
 // [n_q], or null): the distance penalty; sink (float32 [n_q] or null); cross != 0: out is [tokens, n_q, n_kv, D] and slot
-// c of a head holds its weights applied to the values of key/value head c.  Every request's rows are worked on (single
+// c of a head holds its weights applied to the values of key/value head c; out_gate (float32 [tokens, n_q] or null, not with
+// cross): head h's output of row t is multiplied by out_gate[t, h].  Every request's rows are worked on (single
 // tokens take a tile of their own).
 extern "C" int lse_attention_scored_tc(const void* q, const void* k_cache, const void* v_cache, void* out,
                                        const int* block_tables, int bt_stride, const int* segment_start,
                                        const int* segment_first_pos, int num_segments, int tokens, long long num_pages,
                                        int n_q, int n_kv, int head_dim, int page_size, float scale, const float* r1,
                                        const float* r2, const float* sink, int cross, float* scratch, int* counters,
-                                       long long scratch_slots, cudaStream_t stream) {
+                                       long long scratch_slots, const float* out_gate, cudaStream_t stream) {
   if (tokens <= 0 || num_segments <= 0) return 0;
-  if (!lse_attention_tc_supported(head_dim, n_q, n_kv, page_size) || num_pages <= 0 || !(scale > 0.f) || (!r1) != (!r2) ||
+  if (!lse_attention_tc_supported(head_dim, n_q, n_kv, page_size) || num_pages <= 0 || !(scale > 0.f) || (!r1) != (!r2) || (out_gate && cross) ||
       (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) & 15))
     return LSE_ERR_BAD_ARGUMENT;
   const int n_values = cross ? n_kv : 1;
 #define LSE_SCORED_TC_ARGS q, k_cache, v_cache, out, block_tables, bt_stride, segment_start, segment_first_pos, num_segments, \
-  tokens, num_pages, n_q, n_kv, page_size, scale, 0, 0, scratch, counters, scratch_slots, r1, r2, sink, n_values, stream
+  tokens, num_pages, n_q, n_kv, page_size, scale, 0, 0, scratch, counters, scratch_slots, r1, r2, sink, n_values, stream, 0.f, out_gate
   if (head_dim == 128) return r1 ? launch_prefill_tc<128, 1>(LSE_SCORED_TC_ARGS) : launch_prefill_tc<128, 0>(LSE_SCORED_TC_ARGS);
   return r1 ? launch_prefill_tc<64, 1>(LSE_SCORED_TC_ARGS) : launch_prefill_tc<64, 0>(LSE_SCORED_TC_ARGS);
 #undef LSE_SCORED_TC_ARGS

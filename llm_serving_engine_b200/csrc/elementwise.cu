@@ -13,10 +13,11 @@ LSE_TL_DEFINE(lse_timeline_elementwise)
 LSE_CHECK_DEFINE(lse_check_elementwise)
 
 // ------------------------------------------------------------------ embedding
-// residual[t, :] = float(table[ids[t], :]) * scale
+// residual[t, :] = float(table[ids[t], :]) * scale; hidden_out (or null, one copy only) receives the same row rounded
 template <typename T>
 __global__ void embedding_kernel(const T* __restrict__ table, const int* __restrict__ ids,
-                                 float* __restrict__ out, int hidden, int vocab, int copies, float scale) {
+                                 float* __restrict__ out, T* __restrict__ hidden_out, int hidden, int vocab, int copies,
+                                 float scale) {
   LSE_TL_BEGIN(1)
   pdl_launch_dependents();
   pdl_wait();
@@ -26,28 +27,38 @@ __global__ void embedding_kernel(const T* __restrict__ table, const int* __restr
   float* dst = out + (size_t)t * hidden * copies;   // a row holds `copies` copies of the embedding, side by side
   if (id < 0 || id >= vocab) {  // padding row of a fixed-shape batch
     for (int i = threadIdx.x; i < hidden * copies; i += blockDim.x) dst[i] = 0.f;
+    if (hidden_out)
+      for (int i = threadIdx.x; i < hidden; i += blockDim.x) hidden_out[(size_t)t * hidden + i] = from_f32<T>(0.f);
     return;
   }
   const T* src = table + (size_t)id * hidden;
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
     const float v = to_f32<T>(src[i]) * scale;
     for (int c = 0; c < copies; ++c) dst[(size_t)c * hidden + i] = v;
+    if (hidden_out) hidden_out[(size_t)t * hidden + i] = from_f32<T>(v);
   }
   LSE_TL_MARK(3)
 }
 
-extern "C" int lse_embedding_scaled(const void* table, int table_dtype, const int* ids, float* out, int tokens,
-                                    int hidden, int vocab, int copies, float scale, cudaStream_t stream) {
+extern "C" int lse_embedding_hidden(const void* table, int table_dtype, const int* ids, float* out, void* hidden_out,
+                                    int tokens, int hidden, int vocab, int copies, float scale, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (copies <= 0) return LSE_ERR_BAD_ARGUMENT;
+  if (copies <= 0 || (hidden_out && copies != 1)) return LSE_ERR_BAD_ARGUMENT;
   const int threads = hidden >= 1024 ? 256 : 128;
   if (table_dtype == LSE_DTYPE_F32)
-    lse_launch(embedding_kernel<float>, tokens, threads, 0, stream, (const float*)table, ids, out, hidden, vocab, copies, scale);
+    lse_launch(embedding_kernel<float>, tokens, threads, 0, stream, (const float*)table, ids, out, (float*)hidden_out, hidden,
+               vocab, copies, scale);
   else if (table_dtype == LSE_DTYPE_BF16)
-    lse_launch(embedding_kernel<__nv_bfloat16>, tokens, threads, 0, stream, (const __nv_bfloat16*)table, ids, out, hidden, vocab, copies, scale);
+    lse_launch(embedding_kernel<__nv_bfloat16>, tokens, threads, 0, stream, (const __nv_bfloat16*)table, ids, out,
+               (__nv_bfloat16*)hidden_out, hidden, vocab, copies, scale);
   else
     return LSE_ERR_BAD_ARGUMENT;
   LSE_LAUNCH_CHECK();
+}
+
+extern "C" int lse_embedding_scaled(const void* table, int table_dtype, const int* ids, float* out, int tokens,
+                                    int hidden, int vocab, int copies, float scale, cudaStream_t stream) {
+  return lse_embedding_hidden(table, table_dtype, ids, out, nullptr, tokens, hidden, vocab, copies, scale, stream);
 }
 
 extern "C" int lse_embedding_copies(const void* table, int table_dtype, const int* ids, float* out,

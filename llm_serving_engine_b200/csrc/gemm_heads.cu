@@ -1,4 +1,4 @@
-// A product per head: out[t][h][n] = gate[t][h] * sum_k a[t][h][k] * w[h](k, n), the heads' matrices
+// A product per head: out[t][h][n] = gate[t][h] (or gate[t][h][n]) * sum_k a[t][h][k] * w[h](k, n), the heads' matrices
 // side by side in one tensor.  It is what folds a per-head up-projection into the queries of an attention
 // over a shared latent (w[h] read as [k][n]) and what expands the attended latent into a head's values
 // afterwards (w[h] stored [n][k]): the strides of w say which.  float32 accumulation in k order (one chain
@@ -13,7 +13,7 @@ template <typename TA, typename TW, typename TO>
 __global__ void __launch_bounds__(HG_THREADS)
 head_gemm_kernel(const TA* __restrict__ a, long long a_t, long long a_h, const TW* __restrict__ w, long long w_h,
                  long long w_k, long long w_n, TO* __restrict__ out, long long o_t, long long o_h,
-                 const float* __restrict__ gate, int T, int N, int K) {
+                 const float* __restrict__ gate, int gate_wide, int T, int N, int K) {
   __shared__ float a_s[HG_K][HG_TILE + 4], w_s[HG_K][HG_TILE + 4];
   pdl_launch_dependents();
   pdl_wait();
@@ -55,10 +55,10 @@ head_gemm_kernel(const TA* __restrict__ a, long long a_t, long long a_h, const T
   for (int i = 0; i < 4; ++i) {
     const int t = t0 + ty * 4 + i;
     if (t >= T) continue;
-    const float g = gate ? gate[(size_t)t * gridDim.z + h] : 1.f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
+      const float g = gate && n < N ? gate[gate_wide ? ((size_t)t * gridDim.z + h) * N + n : (size_t)t * gridDim.z + h] : 1.f;
       if (n < N) out[(size_t)t * o_t + (size_t)h * o_h + n] = from_f32<TO>(acc[i][j] * g);
     }
   }
@@ -94,7 +94,7 @@ template <typename TA, typename TW, typename TO, bool KSIDE>
 __global__ void __launch_bounds__(HF_THREADS)
 head_gemm_few_kernel(const TA* __restrict__ a, long long a_t, long long a_h, const TW* __restrict__ w, long long w_h,
                      long long w_k, long long w_n, TO* __restrict__ out, long long o_t, long long o_h,
-                     const float* __restrict__ gate, int T, int N, int K) {
+                     const float* __restrict__ gate, int gate_wide, int T, int N, int K) {
   extern __shared__ __align__(16) float a_sh[];   // [HF_ROWS][K], then (columns side by side) [4][HF_ROWS][32] parts
   pdl_launch_dependents();
   pdl_wait();
@@ -145,7 +145,8 @@ head_gemm_few_kernel(const TA* __restrict__ a, long long a_t, long long a_h, con
 #pragma unroll
           for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
           if (lane == 0 && r < rows && n0 + c < N) {
-            const float g = gate ? gate[(size_t)(t0 + r) * gridDim.y + h] : 1.f;
+            const size_t at = (size_t)(t0 + r) * gridDim.y + h;
+            const float g = gate ? gate[gate_wide ? at * N + n0 + c : at] : 1.f;
             out[(size_t)(t0 + r) * o_t + (size_t)h * o_h + n0 + c] = from_f32<TO>(v * g);
           }
         }
@@ -174,20 +175,68 @@ head_gemm_few_kernel(const TA* __restrict__ a, long long a_t, long long a_h, con
           float v = 0.f;
 #pragma unroll
           for (int p = 0; p < 4; ++p) v += part_s[(p * HF_ROWS + r) * 32 + c];
-          const float g = gate ? gate[(size_t)(t0 + r) * gridDim.y + h] : 1.f;
+          const size_t at = (size_t)(t0 + r) * gridDim.y + h;
+          const float g = gate ? gate[gate_wide ? at * N + blockIdx.x * 32 + c : at] : 1.f;
           out[(size_t)(t0 + r) * o_t + (size_t)h * o_h + blockIdx.x * 32 + c] = from_f32<TO>(v * g);
         }
       }
     }
   }
 }
+
+// out[t][h * N + n] = product[h][t][n] * sigmoid(gate columns): what follows the library's batched product over many rows.
+// A block per token, eight columns of one head a thread (by_eight) or one.
+template <typename TI>
+__global__ void __launch_bounds__(256)
+gate_heads_kernel(const TI* __restrict__ product, const TI* __restrict__ proj, long long ld, TI* __restrict__ out, int T, int heads,
+                  int N, int by_eight) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, width = heads * N;
+  const TI* g_row = proj + (size_t)t * ld;
+  if (by_eight) {
+    for (int i = threadIdx.x * 8; i < width; i += blockDim.x * 8) {
+      const int h = i / N, n = i % N;
+      float x[8], z[8];
+      load_w8<TI>(product + ((size_t)h * T + t) * N + n, x);
+      load_w8<TI>(g_row + i, z);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] *= 1.0f / (1.0f + __expf(-z[e]));
+      uint4 raw;
+      __nv_bfloat162* packed = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) packed[e] = __floats2bfloat162_rn(x[2 * e], x[2 * e + 1]);
+      *reinterpret_cast<uint4*>(out + (size_t)t * width + i) = raw;
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    const int h = i / N, n = i % N;
+    const float z = to_f32<TI>(g_row[i]);
+    out[(size_t)t * width + i] = from_f32<TI>(to_f32<TI>(product[((size_t)h * T + t) * N + n]) / (1.0f + expf(-z)));
+  }
+}
 }  // namespace
 
+// product [heads][T][N], proj: row t's gate columns at t * ld; out [T][heads * N]; all bfloat16.
+extern "C" int lse_gate_heads(const void* product, const void* proj, long long ld, void* out, int T, int heads, int N,
+                              cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (heads <= 0 || N <= 0) return LSE_ERR_BAD_ARGUMENT;
+  const int by_eight = N % 8 == 0 && ld % 8 == 0 && (((uintptr_t)product | (uintptr_t)proj | (uintptr_t)out) & 15) == 0;
+  const int threads = heads * N >= 2048 ? 256 : 128;
+  lse_launch(gate_heads_kernel<__nv_bfloat16>, T, threads, 0, stream, (const __nv_bfloat16*)product, (const __nv_bfloat16*)proj, ld,
+             (__nv_bfloat16*)out, T, heads, N, by_eight);
+  LSE_LAUNCH_CHECK();
+}
+
 // a: element (t, h, k) at t * a_t + h * a_h + k; w: element (h, k, n) at h * w_h + k * w_k + n * w_n;
-// out: element (t, h, n) at t * o_t + h * o_h + n; gate: float32 [T][heads] or null.
+// out: element (t, h, n) at t * o_t + h * o_h + n; gate: float32 [T][heads], or [T][heads][N] (gate_wide),
+// or null.
 extern "C" int lse_head_gemm(const void* a, int a_dtype, long long a_t, long long a_h, const void* w, int w_dtype,
                              long long w_h, long long w_k, long long w_n, void* out, int out_dtype, long long o_t,
-                             long long o_h, const float* gate, int T, int heads, int N, int K, cudaStream_t stream) {
+                             long long o_h, const float* gate, int gate_wide, int T, int heads, int N, int K,
+                             cudaStream_t stream) {
   if (T <= 0) return 0;
   if (heads <= 0 || heads > 65535 || N <= 0 || K <= 0) return LSE_ERR_BAD_ARGUMENT;
   dim3 grid((N + HG_TILE - 1) / HG_TILE, (T + HG_TILE - 1) / HG_TILE, heads);
@@ -201,13 +250,13 @@ extern "C" int lse_head_gemm(const void* a, int a_dtype, long long a_t, long lon
 #define LSE_HG_CASE(TA, TW, TO)                                                                                 \
   if (few && k_side)                                                                                            \
     lse_launch(head_gemm_few_kernel<TA, TW, TO, true>, few_grid, HF_THREADS, few_smem, stream, (const TA*)a,    \
-               a_t, a_h, (const TW*)w, w_h, w_k, w_n, (TO*)out, o_t, o_h, gate, T, N, K);                        \
+               a_t, a_h, (const TW*)w, w_h, w_k, w_n, (TO*)out, o_t, o_h, gate, gate_wide, T, N, K);                        \
   else if (few)                                                                                                 \
     lse_launch(head_gemm_few_kernel<TA, TW, TO, false>, few_grid, HF_THREADS, few_smem, stream, (const TA*)a,   \
-               a_t, a_h, (const TW*)w, w_h, w_k, w_n, (TO*)out, o_t, o_h, gate, T, N, K);                        \
+               a_t, a_h, (const TW*)w, w_h, w_k, w_n, (TO*)out, o_t, o_h, gate, gate_wide, T, N, K);                        \
   else                                                                                                          \
     lse_launch(head_gemm_kernel<TA, TW, TO>, grid, HG_THREADS, 0, stream, (const TA*)a, a_t, a_h, (const TW*)w,  \
-               w_h, w_k, w_n, (TO*)out, o_t, o_h, gate, T, N, K);
+               w_h, w_k, w_n, (TO*)out, o_t, o_h, gate, gate_wide, T, N, K);
   typedef __nv_bfloat16 bf;
   const int code = (a_dtype == LSE_DTYPE_BF16 ? 4 : 0) | (w_dtype == LSE_DTYPE_BF16 ? 2 : 0) | (out_dtype == LSE_DTYPE_BF16 ? 1 : 0);
   switch (code) {

@@ -98,18 +98,19 @@ moe_route_kernel(const float* __restrict__ logits, int n_partials, long long par
   if (lane == 0) identity_weight[t] = identity_sum;
 }
 
-// A router whose scores are sigmoids, chosen within the best groups of experts (a warp per token, float32):
-//   s_e = sigmoid(z_e);  c_e = s_e + correction_e  (the choice score);
+// A router that chooses within the best groups of experts (a warp per token, float32):
+//   s_e = sigmoid(z_e), or softmax(z)_e over all experts (softmax);  c_e = s_e + correction_e  (the choice score);
 //   the experts form `group_count` equal groups of neighbours; a group's score is the sum of its two largest c (of its
-//   one c when a group is a single expert); only the `group_keep` best groups' experts can be chosen (group_count <= 1:
+//   one c when a group is a single expert), or its largest c (group_best); only the `group_keep` best groups' experts can be chosen (group_count <= 1:
 //   all experts);  the `top` largest c among them are chosen (ties: the lower index);
-//   weight_e = s_e / (sum of the chosen s + 1e-20) * scale.
+//   weight_e = s_e / (sum of the chosen s + 1e-20) * scale, or s_e * scale (without normalise).
 // Leaves what moe_route_kernel leaves: the dense row of weights, the choices, a zero identity weight, the shared gate.
 __global__ void __launch_bounds__(ROUTE_THREADS)
-moe_route_sigmoid_kernel(const float* __restrict__ logits, int n_partials, long long partial_stride, int ld,
+moe_route_groups_kernel(const float* __restrict__ logits, int n_partials, long long partial_stride, int ld,
                          const float* __restrict__ correction, int has_shared_gate, float* __restrict__ expert_weights,
                          float* __restrict__ identity_weight, float* __restrict__ shared_gate, int* __restrict__ chosen_out,
-                         int tokens, int experts, int top, int group_count, int group_keep, float scale) {
+                         int tokens, int experts, int top, int group_count, int group_keep, float scale, int softmax,
+                        int group_best, int normalise) {
   extern __shared__ float smem[];   // per warp: [experts] scores, [experts] choice scores, [groups] group scores
   pdl_launch_dependents();
   pdl_wait();
@@ -126,8 +127,15 @@ moe_route_sigmoid_kernel(const float* __restrict__ logits, int n_partials, long 
     for (int p = 0; p < n_partials; ++p) sum += row[(size_t)p * partial_stride + e];
     return sum;
   };
+  float top_z = -INFINITY, z_sum = 0.f;
+  if (softmax) {
+    for (int e = lane; e < experts; e += 32) { const float z = logit(e); score[e] = z; top_z = fmaxf(top_z, z); }
+    top_z = warp_max(top_z);
+    for (int e = lane; e < experts; e += 32) z_sum += expf(score[e] - top_z);
+    z_sum = warp_sum(z_sum);
+  }
   for (int e = lane; e < experts; e += 32) {
-    const float sg = 1.0f / (1.0f + expf(-logit(e)));
+    const float sg = softmax ? expf(score[e] - top_z) / z_sum : 1.0f / (1.0f + expf(-logit(e)));
     score[e] = sg;
     choice[e] = correction ? sg + correction[e] : sg;
     expert_weights[(size_t)t * experts + e] = 0.f;
@@ -143,7 +151,7 @@ moe_route_sigmoid_kernel(const float* __restrict__ logits, int n_partials, long 
         if (c > first) { second = first; first = c; }
         else if (c > second) second = c;
       }
-      group_score[g] = per > 1 ? first + second : first;
+      group_score[g] = per > 1 && !group_best ? first + second : first;
     }
     __syncwarp();
     // a group is kept when fewer than group_keep groups come before it (a larger score, or an equal one at a lower index)
@@ -160,7 +168,6 @@ moe_route_sigmoid_kernel(const float* __restrict__ logits, int n_partials, long 
     __syncwarp();
   }
   float chosen_sum = 0.f;
-  int taken = 0;
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
     int best_e = 0x7fffffff;
@@ -180,7 +187,6 @@ moe_route_sigmoid_kernel(const float* __restrict__ logits, int n_partials, long 
       break;
     }
     chosen_sum += score[best_e];
-    ++taken;
     if (lane == 0) {
       choice[best_e] = -INFINITY;
       expert_weights[(size_t)t * experts + best_e] = score[best_e];
@@ -188,10 +194,9 @@ moe_route_sigmoid_kernel(const float* __restrict__ logits, int n_partials, long 
     }
     __syncwarp();
   }
-  const float factor = scale / (chosen_sum + 1e-20f);
+  const float factor = normalise ? scale / (chosen_sum + 1e-20f) : scale;
   for (int e = lane; e < experts; e += 32) expert_weights[(size_t)t * experts + e] *= factor;
   if (lane == 0) identity_weight[t] = 0.f;
-  (void)taken;
 }
 
 template <typename T> __device__ __forceinline__ void moe_load8(const T* p, float (&v)[8]);
@@ -462,20 +467,21 @@ extern "C" int lse_moe_route_biased(const float* logits, int n_partials, long lo
   LSE_LAUNCH_CHECK();
 }
 
-// As lse_moe_route, for sigmoid scores chosen within the best groups (see moe_route_sigmoid_kernel); no identity experts.
-extern "C" int lse_moe_route_sigmoid(const float* logits, int n_partials, long long partial_stride, int ld,
-                                     const float* correction, int has_shared_gate, float* expert_weights,
-                                     float* identity_weight, float* shared_gate, int* chosen, int tokens, int experts,
-                                     int top, int group_count, int group_keep, float scale, cudaStream_t stream) {
+// As lse_moe_route, for a choice within the best groups (see moe_route_groups_kernel); no identity experts.
+extern "C" int lse_moe_route_groups(const float* logits, int n_partials, long long partial_stride, int ld,
+                                    const float* correction, int has_shared_gate, float* expert_weights,
+                                    float* identity_weight, float* shared_gate, int* chosen, int tokens, int experts,
+                                    int top, int group_count, int group_keep, float scale, int softmax, int group_best,
+                                    int normalise, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (experts <= 0 || top <= 0 || n_partials < 1 || ld < experts + (has_shared_gate ? 1 : 0)) return LSE_ERR_BAD_ARGUMENT;
   if (group_count > 1 && (experts % group_count || group_keep <= 0)) return LSE_ERR_BAD_ARGUMENT;
   if (experts > 1024) return LSE_ERR_TOO_LARGE;
   const int warps = ROUTE_THREADS / 32;
   const size_t smem = sizeof(float) * (2 * (size_t)experts + (group_count > 1 ? group_count : 1)) * warps;
-  lse_launch(moe_route_sigmoid_kernel, (tokens + warps - 1) / warps, ROUTE_THREADS, smem, stream, logits, n_partials,
+  lse_launch(moe_route_groups_kernel, (tokens + warps - 1) / warps, ROUTE_THREADS, smem, stream, logits, n_partials,
              partial_stride, ld, correction, has_shared_gate, expert_weights, identity_weight, shared_gate, chosen, tokens,
-             experts, top, group_count, group_keep, scale);
+             experts, top, group_count, group_keep, scale, softmax, group_best, normalise);
   LSE_LAUNCH_CHECK();
 }
 

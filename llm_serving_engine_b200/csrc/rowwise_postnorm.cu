@@ -8,6 +8,7 @@
 // An input that comes from a matrix product may be a stack of float32 partial sums, added in index order first.
 // All arithmetic is float32; a value is rounded once, when it is stored in a bfloat16 tensor.
 #include "common.cuh"
+#include "rotary.cuh"
 
 LSE_CHECK_DEFINE(lse_check_rowwise_postnorm)
 
@@ -358,6 +359,173 @@ head_norm_rope_kv_write_kernel(const TI* __restrict__ proj, int n_partials, long
   }
 }
 
+// The same for heads that are rotated in neighbouring pairs (values 2i and 2i + 1 by the angle position * freq[i]), with what an
+// attention of that kind may take from the same projected row: values mixed with those of an earlier layer,
+//   v <- (1 - a) v + a first[t]        (mix = &a, float32 on the device; first_in: that layer's values, float32 [T, n_kv * dv]),
+// the layer's own values left for later layers (first_out), and a gate per head, sigmoid of the columns gate_column .. + n_q.
+// A block owns some of a token's items (query heads, key heads, value heads, then the gates), a warp one at a time; sines and
+// cosines are taken once a block.  A lane holds both values of its pairs, so nothing passes through shared memory.
+struct PairHeadArgs {
+  int n_partials;
+  long long partial_stride, ld;
+  const float *bias, *q_norm, *k_norm;
+  float eps;
+  const int *slot_mapping, *positions;
+  const double* freq;
+  float rot_factor;
+  int rot_dims, n_q, n_kv, dk, dv, page_size, num_pages, gate_column;
+  float* gate;
+  const float *mix, *first_in;
+  float* first_out;
+  int items, items_a_block, aligned;
+};
+constexpr int PAIR_THREADS = 128, PAIR_MAX_WIDTH = 256;
+
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(PAIR_THREADS)
+head_norm_pair_rope_kernel(PairHeadArgs a, const TI* __restrict__ proj, TO* __restrict__ q_out, TO* __restrict__ k_cache,
+                           TO* __restrict__ v_cache) {
+  __shared__ float cos_s[PAIR_MAX_WIDTH / 2], sin_s[PAIR_MAX_WIDTH / 2];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int slot = LSE_CHECKED(a.slot_mapping[t], -1, a.num_pages * a.page_size, -1, LSE_CHECK_CACHE_SLOT);
+  if (slot < 0) return;   // padding row
+  const int first = blockIdx.y * a.items_a_block, last = min(a.items, first + a.items_a_block);
+  if (first < a.n_q + a.n_kv) {
+    const int position = a.positions[t];
+    for (int i = threadIdx.x; i < a.rot_dims / 2; i += PAIR_THREADS)
+      rotary_sincos(position, a.freq[i], a.rot_factor, sin_s[i], cos_s[i]);
+    __syncthreads();
+  }
+  const int page = slot / a.page_size, offset = slot % a.page_size;
+  const TI* row = proj + (size_t)t * a.ld;
+  for (int item = first + warp; item < last; item += PAIR_THREADS / 32) {
+    if (item == a.n_q + 2 * a.n_kv) {
+      for (int h = lane; h < a.n_q; h += 32) {
+        const float z = sum_partials<TI>(row + a.gate_column + h, a.n_partials, a.partial_stride);
+        a.gate[(size_t)t * a.n_q + h] = 1.0f / (1.0f + expf(-z));
+      }
+      continue;
+    }
+    int column, width;
+    const float* norm_w = nullptr;
+    TO* dst;
+    int value_at = -1;     // a value head: its first column among the values
+    if (item < a.n_q) {
+      column = item * a.dk; width = a.dk; norm_w = a.q_norm;
+      dst = q_out + ((size_t)t * a.n_q + item) * a.dk;
+    } else if (item < a.n_q + a.n_kv) {
+      const int h = item - a.n_q;
+      column = item * a.dk; width = a.dk; norm_w = a.k_norm;
+      dst = k_cache + (((size_t)page * a.n_kv + h) * a.page_size + offset) * a.dk;
+    } else {
+      const int h = item - a.n_q - a.n_kv;
+      column = (a.n_q + a.n_kv) * a.dk + h * a.dv; width = a.dv; value_at = h * a.dv;
+      dst = v_cache + (((size_t)page * a.n_kv + h) * a.page_size + offset) * a.dv;
+    }
+    const TI* src = row + column;
+    const size_t value_row = (size_t)t * a.n_kv * a.dv;
+    const float share = value_at >= 0 && a.mix ? *a.mix : 0.f;
+    if (a.aligned && width % 4 == 0 && column % 4 == 0) {     // four consecutive values a lane and piece
+      float v[2][4], sq = 0.f;
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        const int i = (lane + 32 * k) * 4;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[k][e] = 0.f;
+        if (i < width) {
+          int p = 0;
+          for (; p + 4 <= a.n_partials; p += 4) {
+            float x[4][4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) postnorm_load4<TI>(src + (size_t)(p + j) * a.partial_stride + i, x[j]);
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+              for (int e = 0; e < 4; ++e) v[k][e] += x[j][e];
+          }
+          for (; p < a.n_partials; ++p) {
+            float x[4];
+            postnorm_load4<TI>(src + (size_t)p * a.partial_stride + i, x);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[k][e] += x[e];
+          }
+          if (a.bias) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[k][e] += a.bias[column + i + e];
+          }
+#pragma unroll
+          for (int e = 0; e < 4; ++e) sq = fmaf(v[k][e], v[k][e], sq);
+        }
+      }
+      const float inv = norm_w ? 1.0f / sqrtf(warp_sum(sq) / (float)width + a.eps) : 1.f;
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        const int i = (lane + 32 * k) * 4;
+        if (i >= width) continue;
+        if (norm_w) {
+          float w[4];
+          postnorm_load4<float>(norm_w + i, w);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) v[k][e] = (v[k][e] * inv) * w[e];
+        }
+        if (value_at >= 0) {
+          if (a.first_out) postnorm_store4<float>(a.first_out + value_row + value_at + i, v[k]);
+          if (a.mix) {
+            float f[4];
+            postnorm_load4<float>(a.first_in + value_row + value_at + i, f);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[k][e] = fmaf(share, f[e], (1.0f - share) * v[k][e]);
+          }
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; e += 2) {
+            if (i + e < a.rot_dims) {
+              const float c = cos_s[(i + e) / 2], s = sin_s[(i + e) / 2], x = v[k][e], y = v[k][e + 1];
+              v[k][e] = x * c - y * s;
+              v[k][e + 1] = y * c + x * s;
+            }
+          }
+        }
+        postnorm_store4<TO>(dst + i, v[k]);
+      }
+      continue;
+    }
+    float v[4][2], sq = 0.f;      // pairs lane, lane + 32, ... (the last may be half a pair)
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int i = 2 * (lane + 32 * k) + e;
+        v[k][e] = i < width ? sum_partials<TI>(src + i, a.n_partials, a.partial_stride) + (a.bias ? a.bias[column + i] : 0.f) : 0.f;
+        sq = fmaf(v[k][e], v[k][e], sq);
+      }
+    const float inv = norm_w ? 1.0f / sqrtf(warp_sum(sq) / (float)width + a.eps) : 1.f;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int i = 2 * (lane + 32 * k);
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        if (i + e >= width) continue;
+        if (norm_w) v[k][e] = (v[k][e] * inv) * norm_w[i + e];
+        if (value_at >= 0) {
+          if (a.first_out) a.first_out[value_row + value_at + i + e] = v[k][e];
+          if (a.mix) v[k][e] = fmaf(share, a.first_in[value_row + value_at + i + e], (1.0f - share) * v[k][e]);
+        }
+      }
+      if (value_at < 0 && i < a.rot_dims) {
+        const float c = cos_s[i / 2], s = sin_s[i / 2], x = v[k][0], y = v[k][1];
+        v[k][0] = x * c - y * s;
+        v[k][1] = y * c + x * s;
+      }
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+        if (i + e < width) dst[i + e] = from_f32<TO>(v[k][e]);
+    }
+  }
+}
+
 __global__ void softcap_kernel(float* __restrict__ values, long long count, float cap) {
   pdl_launch_dependents();
   pdl_wait();
@@ -464,6 +632,39 @@ extern "C" int lse_head_norm_rope_kv_write(const void* proj, int in_dtype, int n
   else if (in_dtype == LSE_DTYPE_F32 && out_dtype == LSE_DTYPE_BF16) LSE_HEADROPE_CASE(float, __nv_bfloat16);
   else return LSE_ERR_BAD_ARGUMENT;
 #undef LSE_HEADROPE_CASE
+  LSE_LAUNCH_CHECK();
+}
+
+// As lse_head_norm_rope_kv_write with neighbouring pairs (see head_norm_pair_rope_kernel): first_out, or mix and first_in
+// (float32 [tokens, n_kv * dv]; mix one float on the device), or neither; gate float32 [tokens, n_q] from the columns
+// gate_column .. (counted like the row's), or null.  Heads up to 256 wide.
+extern "C" int lse_head_norm_pair_rope_kv_write(const void* proj, int in_dtype, int n_partials, long long partial_stride,
+                                                long long ld, const float* bias, const float* q_norm, const float* k_norm,
+                                                float eps, const int* slot_mapping, const int* positions, const double* freq,
+                                                float rot_factor, int rot_dims, void* q_out, void* k_cache, void* v_cache,
+                                                int out_dtype, int tokens, int n_q, int n_kv, int dk, int dv, int page_size,
+                                                int num_pages, int gate_column, float* gate, const float* mix,
+                                                const float* first_in, float* first_out, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (n_q <= 0 || n_kv <= 0 || dk <= 0 || dv <= 0 || n_partials < 1 || dk > PAIR_MAX_WIDTH || dv > PAIR_MAX_WIDTH) return LSE_ERR_BAD_ARGUMENT;
+  if (rot_dims < 0 || rot_dims % 2 || rot_dims > dk || (rot_dims > 0 && (!freq || !positions))) return LSE_ERR_BAD_ARGUMENT;
+  if (!k_cache || !v_cache || !slot_mapping || page_size <= 0 || (!mix) != (!first_in) || (mix && first_out)) return LSE_ERR_BAD_ARGUMENT;
+  const int items = n_q + 2 * n_kv + (gate ? 1 : 0);
+  const int items_a_block = tokens >= 512 ? items : 4;     // few tokens: a warp an item, as many blocks as that takes
+  const int in_align = in_dtype == LSE_DTYPE_F32 ? 16 : 8;
+  const int aligned = ld % 4 == 0 && partial_stride % 4 == 0 && (uintptr_t)proj % in_align == 0;
+  const PairHeadArgs args = {n_partials, partial_stride, ld, bias, q_norm, k_norm, eps, slot_mapping, positions, freq, rot_factor,
+                             rot_dims, n_q, n_kv, dk, dv, page_size, num_pages, gate_column, gate, mix, first_in, first_out,
+                             items, items_a_block, aligned};
+  const dim3 grid(tokens, (items + items_a_block - 1) / items_a_block);
+#define LSE_PAIRROPE_CASE(TI, TO)                                                                                      \
+  lse_launch(head_norm_pair_rope_kernel<TI, TO>, grid, PAIR_THREADS, 0, stream, args, (const TI*)proj, (TO*)q_out,     \
+             (TO*)k_cache, (TO*)v_cache)
+  if (in_dtype == LSE_DTYPE_F32 && out_dtype == LSE_DTYPE_F32) LSE_PAIRROPE_CASE(float, float);
+  else if (in_dtype == LSE_DTYPE_BF16 && out_dtype == LSE_DTYPE_BF16) LSE_PAIRROPE_CASE(__nv_bfloat16, __nv_bfloat16);
+  else if (in_dtype == LSE_DTYPE_F32 && out_dtype == LSE_DTYPE_BF16) LSE_PAIRROPE_CASE(float, __nv_bfloat16);
+  else return LSE_ERR_BAD_ARGUMENT;
+#undef LSE_PAIRROPE_CASE
   LSE_LAUNCH_CHECK();
 }
 

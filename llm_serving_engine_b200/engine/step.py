@@ -65,6 +65,7 @@ class StepContext:
         self.segment_context: torch.Tensor = None    # [S] keys of the request after this step
         self.segment_state_slot: torch.Tensor = None  # [S]
         self.want_rows: torch.Tensor = None          # [W]
+        self.carried: dict = {}                      # what a layer leaves for later layers of this step (by the mixers' own keys)
         self.max_segment_tokens = 0
         self.max_context = 0                         # None: not known on the host (a replayed graph)
         self.decode_only = False                     # every segment brings exactly one token

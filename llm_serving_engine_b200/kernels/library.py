@@ -16,6 +16,20 @@ from ..csrc import build
 _lib = None
 
 _SIGNATURES = {
+    "lse_moe_route_groups": [c_void_p, c_int, c_longlong, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                             c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p],
+    "lse_head_norm_pair_rope_kv_write": [c_void_p, c_int, c_int, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p,
+                                         c_float, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p,
+                                         c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                                         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
+    "lse_gate_heads": [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_void_p],
+    "lse_latent_front": [c_void_p, c_int, c_int, c_longlong, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                         c_float, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                         c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
+    "lse_layer_norm": [c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_float, c_int,
+                       c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "lse_embedding_hidden": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
+                             c_void_p],
     "lse_embedding": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "lse_embedding_copies": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "lse_streams_update_rmsnorm": [c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_float, c_void_p, c_void_p,
@@ -40,9 +54,9 @@ _SIGNATURES = {
                                    c_int, c_int, c_void_p],
     "lse_latent_attention_mma_supported": [c_int, c_int],
     "lse_latent_attention_mma": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
-                                 c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_void_p],
+                                 c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_void_p],
     "lse_head_gemm": [c_void_p, c_int, c_longlong, c_longlong, c_void_p, c_int, c_longlong, c_longlong, c_longlong,
-                      c_void_p, c_int, c_longlong, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+                      c_void_p, c_int, c_longlong, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "lse_add_rmsnorm": [c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int,
                         c_int, c_float, c_int, c_int, c_void_p],
     "lse_rope_kv_write": [c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -109,7 +123,7 @@ _SIGNATURES = {
     "lse_head_mix_gate_stages": [c_int, c_int, c_int],
     "lse_attention_scored_tc": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
                                 c_longlong, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int,
-                                c_void_p, c_void_p, c_longlong, c_void_p],
+                                c_void_p, c_void_p, c_longlong, c_void_p, c_void_p],
     "lse_embedding_scaled": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p],
     "lse_tanh_norm": [c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                       c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
@@ -167,7 +181,7 @@ _SIGNATURES = {
     "lse_attention_scored_windowed": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p,
                                       c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                       c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p,
-                                      c_void_p],
+                                      c_void_p, c_void_p],
     "lse_gated_linear_attention_scan_shared": [c_void_p, c_int, c_int, c_longlong, c_longlong, c_int, c_int, c_int,
                                                c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                                c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
@@ -181,13 +195,11 @@ _SIGNATURES = {
     "lse_gated_group_rmsnorm": [c_void_p, c_void_p, c_int, c_int, c_longlong, c_longlong, c_int, c_void_p, c_longlong,
                                 c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_longlong, c_int, c_int, c_int,
                                 c_float, c_float, c_int, c_int, c_void_p, c_void_p],
-    "lse_moe_route_sigmoid": [c_void_p, c_int, c_longlong, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                              c_int, c_int, c_int, c_int, c_int, c_float, c_void_p],
     "lse_attention_scored_mma_windowed": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                           c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                          c_float, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
+                                          c_float, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p],
     "lse_attention_scored_merge_windowed": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                                            c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+                                            c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "lse_attention_sigmoid_tc": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
                                  c_longlong, c_int, c_int, c_int, c_int, c_float, c_void_p, c_float, c_void_p, c_void_p,
                                  c_longlong, c_void_p],

@@ -45,14 +45,17 @@ def sm_count(device=None) -> int:
     return count
 
 
-def embedding(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, copies: int = 1, scale: float = 1.0) -> torch.Tensor:
-    """out[t] = float32(table[ids[t]]) * scale, ``copies`` times side by side; ids int32 [T], out float32 [T, copies * H]."""
-    _need_cuda(table, ids, out)
+def embedding(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, copies: int = 1, scale: float = 1.0,
+              hidden_out: torch.Tensor | None = None) -> torch.Tensor:
+    """out[t] = float32(table[ids[t]]) * scale, ``copies`` times side by side; ids int32 [T], out float32 [T, copies * H].
+    ``hidden_out`` ([T, H] in the table's dtype, one copy only): receives the same rows rounded."""
+    _need_cuda(table, ids, out, hidden_out)
     vocab, hidden = table.shape
     assert ids.dtype == torch.int32 and out.dtype == torch.float32 and table.is_contiguous()
     assert out.shape == (ids.shape[0], copies * hidden) and out.is_contiguous()
+    assert hidden_out is None or (copies == 1 and hidden_out.shape == out.shape and hidden_out.dtype == table.dtype and hidden_out.is_contiguous())
     lib = library.load()
-    check(lib.lse_embedding_scaled(table.data_ptr(), dtype_code(table.dtype), ids.data_ptr(), out.data_ptr(),
+    check(lib.lse_embedding_hidden(table.data_ptr(), dtype_code(table.dtype), ids.data_ptr(), out.data_ptr(), _ptr(hidden_out),
                                    ids.shape[0], hidden, vocab, int(copies), float(scale), _stream()), "embedding")
     return out
 
@@ -675,10 +678,35 @@ def latent_query(proj: torch.Tensor, q_off: int, heads: int, dim: int, rot: int,
                                tokens, _stream()), "latent_query")
 
 
-def latent_attention_mma_supported(dk: int, dv: int, dtype: torch.dtype, window: int = 0) -> bool:
-    """Whether the tensor-core kernel takes this shape (bfloat16, DK a multiple of 16, DV a multiple of 8 up to 512,
-    no window); other shapes, and float32, run the general kernel."""
-    if dtype != torch.bfloat16 or window > 0:
+def latent_front(proj: torch.Tensor, step_positions: torch.Tensor, slot_mapping: torch.Tensor, eps: float, *, q_off: int,
+                 heads: int, dim: int, rot: int, rot_dims: int, freq: torch.Tensor, rot_factor: float, kv_off: int, rank: int,
+                 kv_norm: torch.Tensor, q_plain: torch.Tensor, q_wide: torch.Tensor, cache: torch.Tensor, g_off: int = -1,
+                 gate: torch.Tensor | None = None) -> None:
+    """:func:`latent_prepare` and :func:`latent_query` in one launch, for layers whose one projection ``proj`` holds the queries
+    (from column q_off), the latent with the shared key part (kv_off) and the gates (g_off): the queries' unrotated parts go
+    to ``q_plain`` [T, heads, dim], their rotated parts behind column ``rank`` of ``q_wide`` [T, heads, wide], the normed latent
+    and the rotated shared part into the token's row of ``cache``, sigmoid of the gate columns into ``gate`` float32 (its
+    size gives their number; None: none)."""
+    _need_cuda(proj, step_positions, slot_mapping, freq, kv_norm, q_plain, q_wide, cache, gate)
+    proj, code, n_partials, stride, ld = _projection(proj)
+    tokens = proj.shape[-2]
+    assert q_plain.shape == (tokens, heads, dim) and q_plain.is_contiguous() and q_wide.is_contiguous()
+    assert q_wide.shape[:2] == (tokens, heads) and rank + rot <= q_wide.shape[2] and q_wide.dtype == q_plain.dtype == cache.dtype
+    assert freq.dtype == torch.float64 and freq.shape[0] >= rot_dims // 2
+    assert cache.is_contiguous() and cache.shape[-1] == rank + rot and kv_norm.dtype == torch.float32 and kv_norm.shape == (rank,)
+    assert gate is None or (gate.dtype == torch.float32 and gate.is_contiguous() and gate.shape[0] == tokens)
+    check(library.load().lse_latent_front(
+        proj.data_ptr(), code, n_partials, stride, ld, q_off, heads, dim, rot, rot_dims, freq.data_ptr(), float(rot_factor), kv_off,
+        rank, kv_norm.data_ptr(), float(eps), step_positions.data_ptr(), slot_mapping.data_ptr(), q_plain.data_ptr(),
+        q_wide.data_ptr(), q_wide.shape[2], cache.data_ptr(), dtype_code(q_plain.dtype), g_off,
+        0 if gate is None else gate.numel() // max(tokens, 1), _ptr(gate), tokens, cache.shape[0] * cache.shape[1], _stream()),
+        "latent_front")
+
+
+def latent_attention_mma_supported(dk: int, dv: int, dtype: torch.dtype) -> bool:
+    """Whether the tensor-core kernel takes this shape (bfloat16, DK a multiple of 16, DV a multiple of 8 up to 512); other
+    shapes, and float32, run the general kernel."""
+    if dtype != torch.bfloat16:
         return False
     return bool(library.load().lse_latent_attention_mma_supported(int(dk), int(dv)))
 
@@ -690,7 +718,8 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, bl
                      segment_first_position: torch.Tensor | None = None, tensor_cores: bool = True) -> torch.Tensor:
     """Attention of every row of the step over its request's cached latent rows: q [T, heads, DK], cache
     [pages, page_size, DK], out [T, heads, DV] with DV <= DK: the first DV columns of a row are its value.
-    ``sink`` float32 [heads]: exp(sink_h) joins the softmax's denominator.  ``split``: every chunk of 256 keys of a
+    ``sink`` float32 [heads]: exp(sink_h) joins the softmax's denominator.  ``window`` > 0: a row reads its last ``window``
+    rows only, itself included.  ``split``: every chunk of 256 keys of a
     row gets a block of its own and a second kernel merges them (default: with few rows).  Given the step's
     ``segment_start`` (int32 [S + 1]) and ``segment_first_position`` (int32 [S]), bfloat16 shapes that the
     tensor-core kernel takes run there (``tensor_cores=False``: the general kernel, for comparisons)."""
@@ -707,21 +736,23 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, bl
     if split if split is not None else tokens <= GENERIC_SPLIT_MAX_ROWS:
         chunk = int(lib.lse_latent_attention_chunk())
         max_chunks = max(1, -(-(block_tables.stride(0) * page_size) // chunk))
+        if window > 0:     # chunks that the window of a tile of up to 32 rows can touch
+            max_chunks = min(max_chunks, (window + 30) // chunk + 2)
         partials = torch.empty(tokens * heads * max_chunks * (dv + 2), dtype=torch.float32, device=q.device)
     if (tensor_cores and segment_start is not None and segment_first_position is not None
-            and latent_attention_mma_supported(dk, dv, q.dtype, window)):
+            and latent_attention_mma_supported(dk, dv, q.dtype)):
         segments = segment_first_position.shape[0]
         assert segment_start.dtype == torch.int32 and segment_start.shape[0] == segments + 1
         assert segments == block_tables.shape[0]
         check(lib.lse_latent_attention_mma(q.data_ptr(), cache.data_ptr(), out.data_ptr(), block_tables.data_ptr(),
                                            block_tables.stride(0), segment_start.data_ptr(),
                                            segment_first_position.data_ptr(), _ptr(sink), tokens, segments, heads, dk,
-                                           dv, page_size, float(scale), cache.shape[0], _ptr(partials), max_chunks,
-                                           _stream()), "latent_attention_mma")
+                                           dv, page_size, float(scale), int(window), cache.shape[0], _ptr(partials),
+                                           max_chunks, _stream()), "latent_attention_mma")
         if partials is not None:
             check(lib.lse_latent_attention_merge(partials.data_ptr(), out.data_ptr(), dtype_code(out.dtype),
                                                  segment_of_token.data_ptr(), positions.data_ptr(), _ptr(sink), tokens,
-                                                 heads, dv, 0, max_chunks, block_tables.shape[0], _stream()),
+                                                 heads, dv, int(window), max_chunks, block_tables.shape[0], _stream()),
                   "latent_attention_merge")
         return out
     check(lib.lse_latent_attention(q.data_ptr(), cache.data_ptr(), out.data_ptr(), dtype_code(q.dtype),
@@ -735,18 +766,32 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, bl
 def head_gemm(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gate: torch.Tensor | None = None) -> torch.Tensor:
     """out[t, h, n] = gate[t, h] * sum_k a[t, h, k] * weight[h, k, n]: a product per head.  a [T, heads, K] and out
     [T, heads, N] may be views with strided rows and heads (innermost contiguous); weight [heads, K, N] any strides
-    (pass a transposed view for matrices stored [N, K]); gate float32 [T, heads] or None."""
+    (pass a transposed view for matrices stored [N, K]); gate float32 [T, heads] (one number a head), [T, heads, N] (one
+    an output) or None."""
     _need_cuda(a, weight, out, gate)
     tokens, heads, k = a.shape
     n = out.shape[2]
     assert weight.shape == (heads, k, n) and out.shape[:2] == (tokens, heads)
     assert a.stride(2) == 1 and out.stride(2) == 1
-    assert gate is None or (gate.dtype == torch.float32 and gate.shape == (tokens, heads) and gate.is_contiguous())
+    assert gate is None or (gate.dtype == torch.float32 and gate.is_contiguous()
+                            and gate.shape in ((tokens, heads), (tokens, heads, n)))
     lib = library.load()
     check(lib.lse_head_gemm(a.data_ptr(), dtype_code(a.dtype), a.stride(0), a.stride(1), weight.data_ptr(),
                             dtype_code(weight.dtype), weight.stride(0), weight.stride(1), weight.stride(2),
-                            out.data_ptr(), dtype_code(out.dtype), out.stride(0), out.stride(1), _ptr(gate), tokens,
-                            heads, n, k, _stream()), "head_gemm")
+                            out.data_ptr(), dtype_code(out.dtype), out.stride(0), out.stride(1), _ptr(gate),
+                            int(gate is not None and gate.dim() == 3), tokens, heads, n, k, _stream()), "head_gemm")
+    return out
+
+
+def gate_heads(product: torch.Tensor, proj: torch.Tensor, g_off: int, out: torch.Tensor) -> torch.Tensor:
+    """out[t, h, n] = product[h, t, n] * sigmoid(proj[t, g_off + h * N + n]): product [heads, T, N] (a batched product's
+    result), proj [T, width], out [T, heads, N], all bfloat16."""
+    _need_cuda(product, proj, out)
+    heads, tokens, n = product.shape
+    assert product.dtype == proj.dtype == out.dtype == torch.bfloat16 and product.is_contiguous() and out.is_contiguous()
+    assert out.shape == (tokens, heads, n) and proj.dim() == 2 and proj.stride(1) == 1 and proj.shape[1] >= g_off + heads * n
+    check(library.load().lse_gate_heads(product.data_ptr(), proj.data_ptr() + g_off * 2, proj.stride(0), out.data_ptr(), tokens,
+                                        heads, n, _stream()), "gate_heads")
     return out
 
 
@@ -855,13 +900,46 @@ def head_norm_rope_kv_write(proj: torch.Tensor, bias: torch.Tensor | None, q_nor
         "head_norm_rope_kv_write")
 
 
+def head_norm_pair_rope_kv_write(proj: torch.Tensor, bias: torch.Tensor | None, q_norm: torch.Tensor | None,
+                                 k_norm: torch.Tensor | None, eps: float, slot_mapping: torch.Tensor, positions: torch.Tensor,
+                                 freq: torch.Tensor, rot_factor: float, q_out: torch.Tensor, k_cache: torch.Tensor,
+                                 v_cache: torch.Tensor, n_q: int, n_kv: int, dk: int, dv: int, offset: int = 0,
+                                 gate_column: int = 0, gate: torch.Tensor | None = None, mix: torch.Tensor | None = None,
+                                 first_in: torch.Tensor | None = None, first_out: torch.Tensor | None = None) -> None:
+    """As :func:`head_norm_rope_kv_write` with neighbouring pairs: values 2i and 2i + 1 of a head are rotated by
+    position * freq[i].  ``gate`` (float32 [T, n_q]) receives the sigmoid of the columns ``gate_column`` .. (counted from
+    ``offset``).  ``first_out`` (float32 [T, n_kv * dv]) receives the row's values; or, with ``first_in`` of that shape and
+    ``mix`` (float32, one number), the values become (1 - mix) v + mix first_in."""
+    _need_cuda(proj, bias, q_norm, k_norm, slot_mapping, positions, freq, q_out, k_cache, v_cache, gate, mix, first_in, first_out)
+    proj, code, n_partials, stride, ld = _projection(proj)
+    tokens = proj.shape[-2]
+    assert q_out.shape == (tokens, n_q, dk) and q_out.is_contiguous()
+    assert bias is None or bias.dtype == torch.float32
+    for weight in (q_norm, k_norm):
+        assert weight is None or (weight.dtype == torch.float32 and weight.shape == (dk,))
+    assert freq.dtype == torch.float64 and freq.is_contiguous() and positions.dtype == torch.int32
+    assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == v_cache.dtype == q_out.dtype
+    assert k_cache.shape[1] == n_kv and k_cache.shape[3] == dk and v_cache.shape[3] == dv
+    assert slot_mapping.dtype == torch.int32 and slot_mapping.shape[0] >= tokens
+    assert gate is None or (gate.dtype == torch.float32 and gate.shape == (tokens, n_q) and gate.is_contiguous())
+    assert mix is None or (mix.dtype == torch.float32 and mix.numel() == 1)
+    for values in (first_in, first_out):
+        assert values is None or (values.dtype == torch.float32 and values.shape == (tokens, n_kv * dv) and values.is_contiguous())
+    check(library.load().lse_head_norm_pair_rope_kv_write(
+        proj.data_ptr() + int(offset) * proj.element_size(), code, n_partials, stride, ld, _ptr(bias), _ptr(q_norm), _ptr(k_norm),
+        float(eps), slot_mapping.data_ptr(), positions.data_ptr(), freq.data_ptr() if freq.numel() else None, float(rot_factor),
+        2 * freq.numel(), q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), dtype_code(q_out.dtype), tokens, n_q, n_kv,
+        dk, dv, k_cache.shape[2], k_cache.shape[0], int(gate_column), _ptr(gate), _ptr(mix), _ptr(first_in), _ptr(first_out),
+        _stream()), "head_norm_pair_rope_kv_write")
+
+
 def attention_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor,
                      block_tables: torch.Tensor, segment_of_token: torch.Tensor, positions: torch.Tensor, scale: float,
                      r1: torch.Tensor | None = None, r2: torch.Tensor | None = None, sink: torch.Tensor | None = None,
                      cross: bool = False, split: bool | None = None, segment_start: torch.Tensor | None = None,
                      segment_first_position: torch.Tensor | None = None, tensor_cores: bool = True,
                      window: int = 0, cap: float = 0.0, head_bias: torch.Tensor | None = None,
-                     keep_first: int = 0) -> torch.Tensor:
+                     keep_first: int = 0, out_gate: torch.Tensor | None = None) -> torch.Tensor:
     """Causal attention of every row of the step over its request's pages, with the scores or weights changed:
     s_ij = q_i . k_j * scale - r1_h ln(1 + r2_h (i - j)) (``r1``, ``r2`` float32 [n_q]); exp(sink_h) in the
     denominator (``sink`` float32 [n_q]).  q [T, n_q, dk]; k_cache [pages, n_kv, page, dk]; v_cache [.., dv];
@@ -872,9 +950,10 @@ def attention_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     ``window`` > 0: a row reads its last ``window`` keys only (itself included) and, with ``keep_first`` > 0, of those before
     them the request's first ``keep_first``.  ``cap`` > 0: scores become
     cap * tanh(s / cap).  ``head_bias`` (float32 [n_q]): no softmax; a key's weight is sigmoid(s + head_bias_h) and the
-    weights are not normalised over the keys."""
+    weights are not normalised over the keys.  ``out_gate`` (float32 [T, n_q], not with ``cross``): head h's output of row t is
+    multiplied by out_gate[t, h]."""
     _need_cuda(q, k_cache, v_cache, out, block_tables, segment_of_token, positions, r1, r2, sink, segment_start,
-               segment_first_position, head_bias)
+               segment_first_position, head_bias, out_gate)
     tokens, n_q, dk = q.shape
     n_kv, page_size, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
     n_values = n_kv if cross else 1
@@ -888,6 +967,7 @@ def attention_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     assert block_tables.dtype == torch.int32 and block_tables.dim() == 2 and block_tables.stride(1) == 1
     for vector in (r1, r2, sink, head_bias):
         assert vector is None or (vector.dtype == torch.float32 and vector.shape == (n_q,))
+    _check_out_gate(out_gate, tokens, n_q, cross)
     lib = library.load()
     partials, max_chunks = None, 0
     if split if split is not None else tokens <= GENERIC_SPLIT_MAX_ROWS:
@@ -903,20 +983,28 @@ def attention_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
             block_tables.data_ptr(), block_tables.stride(0), segment_start.data_ptr(), segment_first_position.data_ptr(),
             segments, _ptr(r1), _ptr(r2), _ptr(sink), tokens, n_q, n_kv, dk, dv, int(cross), page_size, float(scale),
             k_cache.shape[0], _ptr(partials), max_chunks, int(window), int(keep_first), float(cap), _ptr(head_bias),
-            _stream()), "attention_scored_mma")
+            _ptr(out_gate), _stream()), "attention_scored_mma")
         if partials is not None:
             check(lib.lse_attention_scored_merge_windowed(
                 partials.data_ptr(), out.data_ptr(), dtype_code(out.dtype), segment_of_token.data_ptr(),
                 positions.data_ptr(), _ptr(sink), tokens, n_q, n_values, dv, max_chunks, block_tables.shape[0],
-                int(window), int(keep_first), int(head_bias is not None), _stream()), "attention_scored_merge")
+                int(window), int(keep_first), int(head_bias is not None), _ptr(out_gate), _stream()), "attention_scored_merge")
         return out
     check(lib.lse_attention_scored_windowed(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), dtype_code(q.dtype),
         int(out.dtype == torch.float32 and q.dtype != torch.float32), block_tables.data_ptr(), block_tables.stride(0),
         segment_of_token.data_ptr(), positions.data_ptr(), _ptr(r1), _ptr(r2), _ptr(sink), tokens, n_q, n_kv, dk, dv,
         int(cross), page_size, float(scale), k_cache.shape[0], block_tables.shape[0], _ptr(partials), max_chunks,
-        int(window), int(keep_first), float(cap), _ptr(head_bias), _stream()), "attention_scored")
+        int(window), int(keep_first), float(cap), _ptr(head_bias), _ptr(out_gate), _stream()), "attention_scored")
     return out
+
+
+def _check_out_gate(out_gate: torch.Tensor | None, tokens: int, n_q: int, cross: bool) -> None:
+    if out_gate is None:
+        return
+    if cross:
+        raise KernelError("attention: a gate per head belongs to outputs of one value slot")
+    assert out_gate.dtype == torch.float32 and out_gate.shape == (tokens, n_q) and out_gate.is_contiguous()
 
 
 def head_mix_gate_stages(n_q: int, n_values: int, dv: int) -> bool:
@@ -927,12 +1015,14 @@ def head_mix_gate_stages(n_q: int, n_values: int, dv: int) -> bool:
 def attention_scored_tc(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor,
                         block_tables: torch.Tensor, segment_start: torch.Tensor, segment_first_position: torch.Tensor,
                         scale: float, r1: torch.Tensor | None = None, r2: torch.Tensor | None = None,
-                        sink: torch.Tensor | None = None, cross: bool = False) -> torch.Tensor:
+                        sink: torch.Tensor | None = None, cross: bool = False,
+                        out_gate: torch.Tensor | None = None) -> torch.Tensor:
     """:func:`attention_scored` for prompt portions on the 5th-generation tensor cores (the kernel of
     :func:`paged_attention_prefill_tc` with the penalty, the sink and the value head as a grid dimension): bfloat16,
     keys and values of one size, 64 or 128, pages of 8 to 128 keys.  out [T, n_q, dv] or, with ``cross``,
     [T, n_q, n_kv, dv], bfloat16.  Every request of the step is worked on in tiles of 128 rows."""
-    _need_cuda(q, k_cache, v_cache, out, block_tables, segment_start, segment_first_position, r1, r2, sink)
+    _need_cuda(q, k_cache, v_cache, out, block_tables, segment_start, segment_first_position, r1, r2, sink, out_gate)
+    _check_out_gate(out_gate, q.shape[0], q.shape[1], cross)
     tokens, n_q, head_dim = q.shape
     pages, n_kv, page_size = k_cache.shape[0], k_cache.shape[1], k_cache.shape[2]
     segments = segment_first_position.shape[0]
@@ -948,8 +1038,8 @@ def attention_scored_tc(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
                                                  block_tables.data_ptr(), block_tables.stride(0), segment_start.data_ptr(),
                                                  segment_first_position.data_ptr(), segments, tokens, pages, n_q, n_kv,
                                                  head_dim, page_size, float(scale), _ptr(r1), _ptr(r2), _ptr(sink),
-                                                 int(cross), _ptr(scratch), _ptr(counters), counters.shape[0], _stream()),
-          "attention_scored_tc")
+                                                 int(cross), _ptr(scratch), _ptr(counters), counters.shape[0], _ptr(out_gate),
+                                                 _stream()), "attention_scored_tc")
     return out
 
 
@@ -980,7 +1070,7 @@ def attention_sigmoid_tc(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
 
 def attention_scored_mma_supported(dk: int, dv: int, n_q: int, n_kv: int, dtype: torch.dtype) -> bool:
     """Whether the tensor-core form of :func:`attention_scored` takes this shape (bfloat16; keys and values of one
-    size, 32, 48, 64, 96 or 128; at most 64 query heads a group)."""
+    size, 32, 48, 64, 96 or 128, or one of the pairs that were built; at most 64 query heads a group)."""
     if dtype != torch.bfloat16:
         return False
     return bool(library.load().lse_attention_scored_mma_supported(int(dk), int(dv), int(n_q), int(n_kv)))
@@ -1041,13 +1131,15 @@ def moe_route(logits: torch.Tensor, correction: torch.Tensor | None, outputs: in
     return expert_weights, identity_weight, gate
 
 
-def moe_route_sigmoid(logits: torch.Tensor, correction: torch.Tensor | None, experts: int, top: int, group_count: int,
-                      group_keep: int, scale: float, shared_gate: bool = False, chosen: torch.Tensor | None = None):
-    """A router with sigmoid scores, in float32: s = sigmoid(z); the choice goes by s + ``correction`` and is confined to
-    the ``group_keep`` best of ``group_count`` equal groups of neighbouring experts (a group's score: the sum of its two
-    largest choice scores); the ``top`` largest choice scores are chosen; weights s / (sum of the chosen s + 1e-20) *
-    ``scale``.  ``group_count`` <= 1: no groups.  Arguments and results otherwise as :func:`moe_route` (no identity
-    experts: the second result is zeros)."""
+def moe_route_groups(logits: torch.Tensor, correction: torch.Tensor | None, experts: int, top: int, group_count: int,
+                     group_keep: int, scale: float, shared_gate: bool = False, chosen: torch.Tensor | None = None,
+                     softmax: bool = False, group_best: bool = False, normalise: bool = True):
+    """A router that chooses within the best groups of experts, in float32: s = sigmoid(z), or softmax(z) over the experts
+    (``softmax``); the choice goes by s + ``correction`` and is confined to the ``group_keep`` best of ``group_count`` equal
+    groups of neighbouring experts (a group's score: the sum of its two largest choice scores, or with ``group_best`` the
+    largest); the ``top`` largest choice scores are chosen; weights s / (sum of the chosen s + 1e-20) * ``scale``, or without
+    ``normalise`` s * ``scale``.  ``group_count`` <= 1: no groups.  Arguments and results otherwise as :func:`moe_route` (no
+    identity experts: the second result is zeros)."""
     _need_cuda(logits, correction, chosen)
     logits, code, n_partials, stride, ld = _projection(logits)
     tokens = logits.shape[-2]
@@ -1057,10 +1149,11 @@ def moe_route_sigmoid(logits: torch.Tensor, correction: torch.Tensor | None, exp
     expert_weights = torch.empty((tokens, experts), dtype=torch.float32, device=logits.device)
     identity_weight = torch.empty((tokens,), dtype=torch.float32, device=logits.device)
     gate = torch.empty((tokens,), dtype=torch.float32, device=logits.device) if shared_gate else None
-    check(library.load().lse_moe_route_sigmoid(logits.data_ptr(), n_partials, stride, ld, _ptr(correction),
-                                               int(shared_gate), expert_weights.data_ptr(), identity_weight.data_ptr(),
-                                               _ptr(gate), _ptr(chosen), tokens, int(experts), int(top), int(group_count),
-                                               int(group_keep), float(scale), _stream()), "moe_route_sigmoid")
+    check(library.load().lse_moe_route_groups(logits.data_ptr(), n_partials, stride, ld, _ptr(correction),
+                                              int(shared_gate), expert_weights.data_ptr(), identity_weight.data_ptr(),
+                                              _ptr(gate), _ptr(chosen), tokens, int(experts), int(top), int(group_count),
+                                              int(group_keep), float(scale), int(softmax), int(group_best), int(normalise),
+                                              _stream()), "moe_route_groups")
     return expert_weights, identity_weight, gate
 
 
@@ -1133,6 +1226,30 @@ def moe_combine(down: torch.Tensor, row_of: torch.Tensor, chosen: torch.Tensor, 
                                          tokens, x.shape[1], top, expert_weights.shape[1], int(accumulate), _stream()),
           "moe_combine")
     return y
+
+
+# ------------------------------------------------------------------ layer norm
+def layer_norm(residual: torch.Tensor, delta: torch.Tensor | None, bias: torch.Tensor | None, weight: torch.Tensor,
+               shift: torch.Tensor, eps: float, out: torch.Tensor | None, rows: torch.Tensor | None = None,
+               write_residual: bool = True, after: bool = False) -> None:
+    """With LN(v) = (v - mean) / sqrt(variance + eps) * weight + shift and d = delta + bias (each may be None): x = residual + d,
+    out = LN(x), the residual becomes x (``write_residual``); with ``rows`` (int32 row indices) only these rows, the residual
+    left alone.  ``after``: the residual becomes residual + LN(d), and ``out`` (or None) receives it rounded.
+    residual float32 [T, H]; delta [T, H] or a float32 stack of partial sums [P, T, H]; bias, weight, shift float32 [H]."""
+    _need_cuda(residual, delta, bias, weight, shift, out, rows)
+    tokens, hidden = residual.shape
+    assert residual.dtype == torch.float32 and residual.is_contiguous()
+    for vector in (bias, weight, shift):
+        assert vector is None or (vector.dtype == torch.float32 and vector.shape == (hidden,) and vector.is_contiguous())
+    delta, n_partials, stride = _partials(delta, tokens, hidden)
+    n_rows = tokens if rows is None else rows.shape[0]
+    assert out is None or (out.shape == (n_rows, hidden) and out.is_contiguous())
+    assert rows is None or (rows.dtype == torch.int32 and not after)
+    out_code = dtype_code(out.dtype) if out is not None else F32
+    delta_code = dtype_code(delta.dtype) if delta is not None else out_code
+    check(library.load().lse_layer_norm(residual.data_ptr(), _ptr(delta), delta_code, n_partials, stride, _ptr(bias), weight.data_ptr(),
+                                        shift.data_ptr(), float(eps), int(after), _ptr(out), out_code, _ptr(rows), n_rows, hidden,
+                                        tokens, int(write_residual and rows is None), _stream()), "layer_norm")
 
 
 # ------------------------------------------------------------------ the tanh norm

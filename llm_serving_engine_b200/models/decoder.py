@@ -204,6 +204,7 @@ class DecoderModel:
         """Run the step's rows through the layers and return float32 logits
         [number of wanted rows, vocab] (an empty tensor when nothing is wanted)."""
         tokens = step.num_tokens
+        step.carried = {}      # what a layer leaves for later layers of the same step
         copies = self.spec.residual_streams
         residual = torch.empty((tokens, copies * self.spec.hidden_size), dtype=torch.float32, device=self.device)
         if self.position_table is not None:
@@ -216,8 +217,13 @@ class DecoderModel:
             stream.hidden = hidden
         else:
             # every copy starts as the embedding
-            ops.embedding(self.embedding, step.token_ids, residual, copies, scale=self.spec.embedding_scale)
+            hidden = None
+            if copies == 1 and getattr(self.blocks[self.spec.order[0]], "reads_residual", False):
+                hidden = residual if self.dtype == torch.float32 else torch.empty_like(residual, dtype=self.dtype)
+            ops.embedding(self.embedding, step.token_ids, residual, copies, scale=self.spec.embedding_scale,
+                          hidden_out=None if hidden is residual else hidden)
             stream = ResidualStream(residual, copies=copies)
+            stream.hidden = hidden
         if self.spec.embedding_again and copies != 1:
             raise ops.KernelError("the embedding is added again to one copy of the residual only")
         for position, index in enumerate(self.spec.order):   # caches run along the order

@@ -218,6 +218,7 @@ class TokenInput(Part):
 class Block:
     graph_safe = False     # as for ``Part``: the arrangement itself launches nothing that depends on the step's contents
     kernel_sources: tuple[str, ...] = ()   # as for ``Part``: what the arrangement itself launches
+    reads_residual = False                 # the branches read the residual itself: the model keeps ``stream.hidden`` from the embedding on
 
     def __init__(self, params, mixer_norm: Norm, mixer: Mixer, feed_forward_norm: Norm | None,
                  feed_forward: FeedForward | None, weights: dict | None = None, ctx: BuildContext | None = None) -> None:

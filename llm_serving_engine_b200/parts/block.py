@@ -83,6 +83,7 @@ class PostNormResidualBlock(Block):
     it, in the compute dtype as ``stream.hidden``, the branches' input; a layer may have no feed-forward."""
 
     graph_safe = True
+    reads_residual = True
 
     def forward(self, stream: ResidualStream, step, cache) -> None:
         if stream.hidden is None:    # the model's embedding left float32 rows only
@@ -95,6 +96,25 @@ class PostNormResidualBlock(Block):
             stream.delta = self.feed_forward.forward(x)
             stream.delta_row_scale = self.feed_forward.row_scale
             self.feed_forward_norm.forward(stream)
+
+
+@register_block("normed_branch_residual")
+class NormedBranchResidualBlock(Block):
+    """h = h + norm1(mixer(h)); h = h + norm2(feed_forward(h)): the branches read the residual itself, their outputs are normed
+    before they are added (the norms have ``add_branch``: ``layernorm``).  The residual is kept in float32 and, beside it, in
+    the compute dtype as ``stream.hidden``, the branches' input; a layer may have no feed-forward."""
+
+    graph_safe = True
+    reads_residual = True
+
+    def forward(self, stream: ResidualStream, step, cache) -> None:
+        stream.delta = self.mixer.forward(stream.hidden, step, cache)
+        stream.delta_bias = self.mixer.output_bias
+        x = self.mixer_norm.add_branch(stream)
+        if self.feed_forward is not None:
+            stream.delta = self.feed_forward.forward(x)
+            stream.delta_row_scale = self.feed_forward.row_scale
+            self.feed_forward_norm.add_branch(stream)
 
 
 @register_block("sandwich_residual")

@@ -203,7 +203,7 @@ class SelectiveStateSpace(BranchMixer):
 
 
 _HEAD_NORM_NAMES = {"q": "q", "k": "k", "v": "v", "out": "o", "q_norm": "q.norm", "k_norm": "k.norm",
-                    "bias_suffix": ".b", "head_bias": "pb", "head_factor": "temp"}
+                    "bias_suffix": ".b", "head_bias": "pb", "head_factor": "temp", "gate": "g", "value_mix": "vmix"}
 
 
 @register_mixer("head_norm_rotary_attention")
@@ -218,11 +218,17 @@ class HeadNormRotaryAttention(BranchMixer):
     left to the norm that adds the output), ``head_factor`` (head h's scores are multiplied by a learned number before the
     cap: its queries are), ``values`` ("own", the default, or "keys": no value projection, a value is its key as projected,
     before norm and rotation), ``keep_first`` (with a window: the request's first so many keys are read as well, their pages
-    stay), ``unit_sink`` (one is added to the softmax's denominator), ``tensor_names``.
+    stay), ``unit_sink`` (one is added to the softmax's denominator), ``pairing`` ("half", the default: value i is rotated with value
+    i + dims / 2; or "neighbours": value 2i with value 2i + 1), ``gate`` (head h's output is multiplied by sigmoid(w_g,h x)),
+    ``value_mix`` (None; "first": the layer's values are left in the step for later layers; or "later": v <- (1 - a) v + a v_first,
+    a learned number a and the values of the layer that left them, of the same token; the mixed values are what the pages
+    keep), ``tensor_names``.
 
     With ``head_norm`` every head of q and of k is RMS-normed over its ``dim`` values with one weight vector for all heads,
-    before the rotation.  One kernel sums the projection, adds the biases, norms, rotates and writes the pages; the attention is
-    the engine's paged attention for changed scores (window, cap and sigmoid weights are arguments of its kernels)."""
+    before the rotation.  One kernel sums the projection, adds the biases, norms, rotates and writes the pages (and, with
+    neighbouring pairs, mixes the values and takes the gates' sigmoids); the attention is the engine's paged attention for
+    changed scores (window, cap, sigmoid weights and gates are arguments of its kernels).  Long prompt portions of the forms
+    without a window run on the tcgen05 kernel, if their scores are not capped or their weights are sigmoids."""
 
     graph_safe = True
     kernel_sources = ("attention_scored", "attention_scored_mma", "attention_tcgen05", "rowwise_postnorm",)
@@ -249,7 +255,20 @@ class HeadNormRotaryAttention(BranchMixer):
         if p.get("unit_sink", False) and self.sigmoid:
             raise ops.KernelError("attention: a sink belongs to the softmax")
         roles = ("q", "k") if self.tied else ("q", "k", "v")
-        self.in_weight = torch.cat([weights[names[role]] for role in roles], dim=0).contiguous()
+        self.neighbours = self._pairing(p) == "neighbours"
+        self.value_mix, self.has_gate = self._value_mix(p), bool(p.get("gate", False))
+        if (self.value_mix or self.has_gate) and (not self.neighbours or self.tied):
+            raise ops.KernelError("attention: gates and mixed values belong to heads rotated in neighbouring pairs, with values of their own")
+        if self.neighbours and (p.get("head_factor", False) or self.tied):
+            raise ops.KernelError("attention: head factors and tied values belong to heads rotated in halves")
+        stacked = [weights[names[role]] for role in roles]
+        self.gate_column = sum(w.shape[0] for w in stacked)
+        if self.has_gate:      # whole tiles of the products, aligned rows of their results
+            stacked.append(weights[names["gate"]])
+            pad = -sum(w.shape[0] for w in stacked) % 16
+            if pad:
+                stacked.append(stacked[0].new_zeros((pad, stacked[0].shape[1])))
+        self.in_weight = torch.cat(stacked, dim=0).contiguous()
         self.in_bias = (torch.cat([weights[names[role] + names["bias_suffix"]].to(torch.float32) for role in roles]).contiguous()
                         if p.get("bias", False) else None)
         def vector(role, used):
@@ -262,7 +281,22 @@ class HeadNormRotaryAttention(BranchMixer):
         self.sink = torch.zeros(self.n_q, dtype=torch.float32, device=ctx.device) if p.get("unit_sink", False) else None
         self.output_bias = (weights[names["out"] + names["bias_suffix"]].to(torch.float32).contiguous()
                             if p.get("output_bias", False) else None)
+        self.share = weights[names["value_mix"]].to(torch.float32).reshape(1).contiguous() if self.value_mix == "later" else None
         self.out_weight = weights[names["out"]].contiguous()
+
+    @staticmethod
+    def _pairing(params) -> str:
+        kind = params.get("pairing", "half")
+        if kind not in ("half", "neighbours"):
+            raise ops.KernelError(f"attention: pairing {kind!r} must be half or neighbours")
+        return kind
+
+    @staticmethod
+    def _value_mix(params):
+        kind = params.get("value_mix")
+        if kind not in (None, "first", "later"):
+            raise ops.KernelError(f"attention: value_mix {kind!r} must be first or later")
+        return kind
 
     @staticmethod
     def _values_kind(params) -> str:
@@ -300,6 +334,10 @@ class HeadNormRotaryAttention(BranchMixer):
                 out[names[role] + names["bias_suffix"]] = TensorSpec((out[names[role]].shape[0],), "bias")
         if cls._weights_kind(p) == "sigmoid":
             out[names["head_bias"]] = TensorSpec((n_q,), "bias")
+        if p.get("gate", False):
+            out[names["gate"]] = TensorSpec((n_q, hidden_size))
+        if cls._value_mix(p):          # the first such layer has the number too, and does not use it
+            out[names["value_mix"]] = TensorSpec((), "positive")
         return out
 
     @classmethod
@@ -310,8 +348,8 @@ class HeadNormRotaryAttention(BranchMixer):
                        int(params.get("keep_first", 0)) if window > 0 else 0)
 
     def _on_tcgen05(self, segment_counts, page_size=None) -> bool:
-        """Long prompt portions of the sigmoid-weighted form without a window run on the tcgen05 kernel."""
-        if not self.sigmoid or self.window > 0:
+        """Long prompt portions without a window run on the tcgen05 kernel: sigmoid weights, or a softmax of uncapped scores."""
+        if self.window > 0 or (self.sigmoid and self.has_gate) or (not self.sigmoid and self.softcap > 0):
             return False
         if not prompt_shape_for_tcgen05(self.ctx.dtype, self.dk, self.dv, segment_counts):
             return False
@@ -324,22 +362,39 @@ class HeadNormRotaryAttention(BranchMixer):
         pages = cache
         tokens = out.shape[0]
         q = torch.empty((tokens, self.n_q, self.dk), dtype=out.dtype, device=out.device)
-        ops.head_norm_rope_kv_write(proj, self.in_bias, self.q_norm, self.k_norm, self.eps, pages.slot_mapping,
-                                    step.positions, self.freq, self.rot_factor, q, pages.keys, pages.values, self.n_q,
-                                    self.n_kv, self.dk, self.dv, offset=offset, q_factor=self.head_factor,
-                                    values_are_keys=self.tied)
+        gate = torch.empty((tokens, self.n_q), dtype=torch.float32, device=out.device) if self.has_gate else None
+        if self.neighbours:
+            first_out = first_in = None
+            if self.value_mix == "first":
+                first_out = torch.empty((tokens, self.n_kv * self.dv), dtype=torch.float32, device=out.device)
+                step.carried["first_values"] = first_out
+            elif self.value_mix == "later":
+                first_in = step.carried["first_values"]
+            ops.head_norm_pair_rope_kv_write(proj, self.in_bias, self.q_norm, self.k_norm, self.eps, pages.slot_mapping,
+                                             step.positions, self.freq, self.rot_factor, q, pages.keys, pages.values, self.n_q,
+                                             self.n_kv, self.dk, self.dv, offset=offset, gate_column=self.gate_column, gate=gate,
+                                             mix=self.share, first_in=first_in, first_out=first_out)
+        else:
+            ops.head_norm_rope_kv_write(proj, self.in_bias, self.q_norm, self.k_norm, self.eps, pages.slot_mapping,
+                                        step.positions, self.freq, self.rot_factor, q, pages.keys, pages.values, self.n_q,
+                                        self.n_kv, self.dk, self.dv, offset=offset, q_factor=self.head_factor,
+                                        values_are_keys=self.tied)
         straight = scale == 1.0 and out.is_contiguous()      # the attention's own output is the branch's
         attended = (out.view(tokens, self.n_q, self.dv) if straight
                     else torch.empty((tokens, self.n_q, self.dv), dtype=out.dtype, device=out.device))
         if (not step.decode_only and step.segments
                 and self._on_tcgen05([segment.count for segment in step.segments], pages.keys.shape[2])):
-            ops.attention_sigmoid_tc(q, pages.keys, pages.values, attended, pages.block_tables, step.segment_start,
-                                     step.segment_first_position, self.scale, self.head_bias, self.softcap)
+            if self.sigmoid:
+                ops.attention_sigmoid_tc(q, pages.keys, pages.values, attended, pages.block_tables, step.segment_start,
+                                         step.segment_first_position, self.scale, self.head_bias, self.softcap)
+            else:
+                ops.attention_scored_tc(q, pages.keys, pages.values, attended, pages.block_tables, step.segment_start,
+                                        step.segment_first_position, self.scale, sink=self.sink, out_gate=gate)
         else:
             ops.attention_scored(q, pages.keys, pages.values, attended, pages.block_tables, step.segment_of_token,
                                  step.positions, self.scale, segment_start=step.segment_start,
                                  segment_first_position=step.segment_first_position, window=self.window, cap=self.softcap,
-                                 head_bias=self.head_bias, sink=self.sink, keep_first=self.keep_first)
+                                 head_bias=self.head_bias, sink=self.sink, keep_first=self.keep_first, out_gate=gate)
         if not straight:
             ops.head_gate_scale(attended, None, out, scale, step.segment_of_token)
 

@@ -46,7 +46,9 @@ class LatentAttention(Mixer):
     ``kv_rank`` (the latent), ``q_rank`` (0: queries are projected directly; else they go through a normed latent of
     this size), ``scale`` (on the scores), ``rot`` ({base, dims, scaling}: see :func:`rotary_frequencies`; the first
     ``dims`` of the ``rot_dim`` values are rotated in interleaved pairs), ``eps`` (of the latent norms), ``sink`` (a
-    learned number per head in the softmax's denominator), ``gate`` (head h's output times sigmoid(W_g x)_h),
+    learned number per head in the softmax's denominator), ``gate`` (true, or "head": head h's output times sigmoid(W_g x)_h;
+    "elements": the concatenated heads times sigmoid(W_g x), W_g with a row per value), ``window`` (> 0: a row reads its last
+    ``window`` keys, itself included; older pages are given back),
     ``own_cache`` (false: the layer reads the latent rows of another layer, ``LayerSpec.cache_from``, and has no
     down-projection of its own), ``tensor_names``.
 
@@ -88,15 +90,26 @@ class LatentAttention(Mixer):
             self.kv_norm = weights[names["kv_down_norm"]].to(torch.float32).contiguous()
             self.kv_off = width
             width += self.rank + self.rot_dim
-        if p.get("gate", False):
+        self.gates = self._gates(p)
+        if self.gates:
             stacked.append(weights[names["gate"]])
             self.g_off = width
-            width += self.heads
+            width += self.gates
+        if self.gates > self.heads and width % 16:       # whole tiles of the product, aligned rows of its result
+            stacked.append(stacked[0].new_zeros((-width % 16, stacked[0].shape[1])))
         self.in_weight = torch.cat(stacked, dim=0).contiguous()
         self.k_up = weights[names["k_up"]].contiguous().view(self.heads, self.dim, self.rank)
         self.v_up = weights[names["v_up"]].contiguous().view(self.heads, self.vdim, self.rank).transpose(1, 2)
         self.sink = weights[names["sink"]].to(torch.float32).contiguous() if p.get("sink", False) else None
         self.out_weight = weights[names["out"]].contiguous()
+
+    @staticmethod
+    def _gates(params) -> int:
+        """Rows of the gate's matrix: none, one per head, or one per value."""
+        kind = params.get("gate", False)
+        if kind not in (False, None, True, "head", "elements"):
+            raise ops.KernelError(f"latent attention: gate {kind!r} must be false, head or elements")
+        return int(params["heads"]) * (int(params["vdim"]) if kind == "elements" else 1) if kind else 0
 
     @classmethod
     def expected_tensors(cls, params, hidden_size):
@@ -118,8 +131,8 @@ class LatentAttention(Mixer):
         out[names["v_up"]] = TensorSpec((heads * vdim, rank))
         if p.get("sink", False):
             out[names["sink"]] = TensorSpec((heads,), "bias")
-        if p.get("gate", False):
-            out[names["gate"]] = TensorSpec((heads, hidden_size))
+        if cls._gates(p):
+            out[names["gate"]] = TensorSpec((cls._gates(p), hidden_size))
         out[names["out"]] = TensorSpec((hidden_size, heads * vdim))
         return out
 
@@ -127,41 +140,62 @@ class LatentAttention(Mixer):
     def cache_requirement(cls, params, hidden_size):
         return PagedLatent(int(params["kv_rank"]) + int(params["rot_dim"]), int(params.get("window", 0)))
 
-    @staticmethod
-    def _per_head(a, weight, out, gate) -> None:
-        """out[t, h] = gate[t, h] * a[t, h] @ weight[h]: many bfloat16 rows go to the library's batched product (the
-        tensor cores), few rows and float32 to the engine's own kernel (true float32, one summation order)."""
-        if a.dtype == torch.bfloat16 and a.shape[0] > PER_HEAD_LIBRARY_ROWS:
-            product = torch.bmm(a.transpose(0, 1), weight)            # [heads, T, N], float32 accumulation
-            if gate is None:
-                out.copy_(product.transpose(0, 1))
-            else:
-                torch.mul(product.transpose(0, 1), gate.unsqueeze(-1), out=out)
+    def _fold_queries(self, q_plain, q_wide) -> None:
+        """q_wide[t, h, :rank] = W_uk,h^T q_plain[t, h]: many bfloat16 rows go to the library's batched product (the tensor
+        cores), few rows and float32 to the engine's own kernel (true float32, one summation order)."""
+        if q_plain.dtype == torch.bfloat16 and q_plain.shape[0] > PER_HEAD_LIBRARY_ROWS:
+            torch.bmm(q_plain.transpose(0, 1), self.k_up, out=q_wide[:, :, :self.rank].transpose(0, 1))
         else:
-            ops.head_gemm(a, weight, out, gate)
+            ops.head_gemm(q_plain, self.k_up, q_wide[:, :, :self.rank])
+
+    def _expand_values(self, attended, values, gate, proj) -> None:
+        """values[t, h] = gate * W_uv,h attended[t, h]; ``gate`` [T, heads], [T, heads, vdim], or None (without gates, or when
+        the gate columns of ``proj`` are still to be taken)."""
+        if attended.dtype == torch.bfloat16 and attended.shape[0] > PER_HEAD_LIBRARY_ROWS:
+            if gate is None and self.g_off < 0:
+                torch.bmm(attended.transpose(0, 1), self.v_up, out=values.transpose(0, 1))
+                return
+            product = torch.bmm(attended.transpose(0, 1), self.v_up)            # [heads, T, vdim], float32 accumulation
+            if gate is None:
+                ops.gate_heads(product, proj, self.g_off, values)
+            else:
+                torch.mul(product.transpose(0, 1), gate if gate.dim() == 3 else gate.unsqueeze(-1), out=values)
+        else:
+            ops.head_gemm(attended, self.v_up, values, gate)
 
     def forward(self, x, step, cache):
         tokens, heads = x.shape[0], self.heads
         proj = linear_partials(x, self.in_weight)
-        q_latent = torch.empty((tokens, self.q_rank), dtype=x.dtype, device=x.device) if self.q_rank else None
-        gate = torch.empty((tokens, heads), dtype=torch.float32, device=x.device) if self.g_off >= 0 else None
-        if self.q_rank or self.own_cache or gate is not None:
-            ops.latent_prepare(proj, step.positions, cache.slot_mapping, self.eps,
-                               q_off=self.q_off, q_rank=self.q_rank, q_norm=self.q_norm if self.q_rank else None,
-                               q_latent=q_latent, kv_off=self.kv_off, rank=self.rank, kv_norm=self.kv_norm,
-                               rot=self.rot_dim, rot_dims=self.rot_dims, freq=self.freq, rot_factor=self.rot_factor,
-                               cache=cache.keys, g_off=self.g_off, heads=heads, gate=gate)
-        queries = linear_partials(q_latent, self.q_up) if self.q_rank else proj
         wide = self.rank + self.rot_dim
         q_plain = torch.empty((tokens, heads, self.dim), dtype=x.dtype, device=x.device)
         q_wide = torch.empty((tokens, heads, wide), dtype=x.dtype, device=x.device)
-        ops.latent_query(queries, 0, heads, self.dim, self.rot_dim, self.rot_dims, self.freq, self.rot_factor,
-                         step.positions, step.segment_of_token, q_plain, q_wide, self.rank)
-        self._per_head(q_plain, self.k_up, q_wide[:, :, :self.rank], None)
+        # many rows: the kernel behind the values' product takes the gates from the projection itself
+        late_gates = self.gates > heads and x.dtype == torch.bfloat16 and proj.dim() == 2 and tokens > PER_HEAD_LIBRARY_ROWS
+        gate = (torch.empty((tokens, self.gates), dtype=torch.float32, device=x.device)
+                if self.gates and not late_gates else None)
+        if not self.q_rank and self.own_cache:
+            ops.latent_front(proj, step.positions, cache.slot_mapping, self.eps, q_off=self.q_off, heads=heads, dim=self.dim,
+                             rot=self.rot_dim, rot_dims=self.rot_dims, freq=self.freq, rot_factor=self.rot_factor,
+                             kv_off=self.kv_off, rank=self.rank, kv_norm=self.kv_norm, q_plain=q_plain, q_wide=q_wide,
+                             cache=cache.keys, g_off=self.g_off, gate=gate)
+        else:
+            q_latent = torch.empty((tokens, self.q_rank), dtype=x.dtype, device=x.device) if self.q_rank else None
+            if self.q_rank or self.own_cache or gate is not None:
+                ops.latent_prepare(proj, step.positions, cache.slot_mapping, self.eps,
+                                   q_off=self.q_off, q_rank=self.q_rank, q_norm=self.q_norm if self.q_rank else None,
+                                   q_latent=q_latent, kv_off=self.kv_off, rank=self.rank, kv_norm=self.kv_norm,
+                                   rot=self.rot_dim, rot_dims=self.rot_dims, freq=self.freq, rot_factor=self.rot_factor,
+                                   cache=cache.keys, g_off=self.g_off, heads=self.gates, gate=gate)
+            queries = linear_partials(q_latent, self.q_up) if self.q_rank else proj
+            ops.latent_query(queries, 0, heads, self.dim, self.rot_dim, self.rot_dims, self.freq, self.rot_factor,
+                             step.positions, step.segment_of_token, q_plain, q_wide, self.rank)
+        self._fold_queries(q_plain, q_wide)
         attended = torch.empty((tokens, heads, self.rank), dtype=x.dtype, device=x.device)
         ops.latent_attention(q_wide, cache.keys, attended, cache.block_tables, step.segment_of_token, step.positions,
                              self.scale, self.sink, self.window, segment_start=step.segment_start,
                              segment_first_position=step.segment_first_position)
         values = torch.empty((tokens, heads, self.vdim), dtype=x.dtype, device=x.device)
-        self._per_head(attended, self.v_up, values, gate)
+        if gate is not None and self.gates > heads:
+            gate = gate.view(tokens, heads, self.vdim)
+        self._expand_values(attended, values, gate, proj)
         return linear_partials(values.view(tokens, heads * self.vdim), self.out_weight)

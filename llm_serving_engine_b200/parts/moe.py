@@ -1,5 +1,5 @@
 """Mixture-of-experts feed-forward: a softmax router over experts and identity experts, clamped gated experts, and a
-gated shared expert."""
+shared expert with or without a gate."""
 from __future__ import annotations
 
 import os
@@ -30,8 +30,10 @@ class ClampedMoE(FeedForward):
     y = W_down (silu(W_gate x) * (W_up x)), nothing clamped, ``limit`` not read; or "squared_relu": experts without a
     gate matrix, y = W_down relu(W_up x)^2), ``scores`` ("softmax", the default, or "sigmoid": scores are sigmoids of the
     logits, the chosen experts' scores are divided by their sum and multiplied by ``router_scale``, and with ``groups``
-    {"count", "keep"} the choice is confined to the ``keep`` best of ``count`` equal groups of neighbouring experts, a
-    group's score being the sum of its two largest corrected scores), ``tensor_names``.
+    {"count", "keep"} the choice is confined to the ``keep`` best of ``count`` equal groups of neighbouring experts;
+    ``groups`` and ``router_scale`` go with "softmax" too, whose weights stay as they are, times ``router_scale``),
+    ``group_score`` (of a group: "two_best", the default, the sum of its two largest corrected scores, or "best", the
+    largest), ``shared_gate`` (default true; false: the shared expert is added as it is and has no gate row), ``tensor_names``.
 
     Expert: g = min(W_gate x, limit), u = clamp(W_up x, -limit, limit), y = W_down (g sigmoid(1.702 g) (u + 1)).
     Router: s = softmax(W_router x) over all outputs, in float32; the ``top`` outputs with the largest s + correction
@@ -67,12 +69,17 @@ class ClampedMoE(FeedForward):
         groups = p.get("groups") or {}
         self.group_count, self.group_keep = int(groups.get("count", 1)), int(groups.get("keep", 1))
         self.router_scale = float(p.get("router_scale", 1.0))
-        if self.sigmoid_scores and (self.identity or self.over_chosen or p.get("router_bias", False)):
-            raise ops.KernelError("mixture of experts: sigmoid scores come without identity experts, a router bias or softmax_chosen")
+        self.group_best = self._group_score(p) == "best"
+        # the router that chooses within groups (one group: all experts)
+        self.in_groups = self.sigmoid_scores or self.group_count > 1 or self.router_scale != 1.0
+        if self.in_groups and (self.identity or self.over_chosen or p.get("router_bias", False)):
+            raise ops.KernelError("mixture of experts: sigmoid scores, groups and a router scale come without identity experts, "
+                                  "a router bias or softmax_chosen")
         self.columns = 1 if self.activation in ops.MOE_UNGATED else 2    # input columns per column of an expert
         self.ff, self.limit = int(p["ff"]), float(p.get("limit", 0.0))
         shared = p.get("shared")
         self.shared_ff = int(shared["ff"]) if shared else 0
+        self.shared_gated = bool(shared) and bool(p.get("shared_gate", True))
         self.shared_limit = float(shared.get("limit", 0.0)) if shared else 0.0
         names = {**_DEFAULT_NAMES, **p.get("tensor_names", {})}
         prefixes = [names["expert"].format(index=index) for index in range(self.experts)]
@@ -85,7 +92,7 @@ class ClampedMoE(FeedForward):
         self.down_weight = torch.cat([weights[prefix + names["down"]] for prefix in prefixes], dim=1).contiguous() if prefixes else None
         # the router's rows, then the shared expert's gate row, padded with zero rows to a multiple of 16: one product
         # gives every logit that the routing kernel reads
-        rows = [weights[names["router"]]] + ([weights[names["shared"] + names["shared_gate"]].reshape(1, -1)] if shared else [])
+        rows = [weights[names["router"]]] + ([weights[names["shared"] + names["shared_gate"]].reshape(1, -1)] if self.shared_gated else [])
         self.outputs = self.experts + self.identity
         pad = -(self.outputs + len(rows) - 1) % 16
         if pad:
@@ -117,7 +124,8 @@ class ClampedMoE(FeedForward):
         sized = [(names["expert"].format(index=index), ff) for index in range(experts)]
         if p.get("shared"):
             sized.append((names["shared"], int(p["shared"]["ff"])))
-            out[names["shared"] + names["shared_gate"]] = TensorSpec((1, hidden_size))
+            if p.get("shared_gate", True):
+                out[names["shared"] + names["shared_gate"]] = TensorSpec((1, hidden_size))
         gated = p.get("activation", "clamped_swish") not in ops.MOE_UNGATED
         for prefix, width in sized:
             if gated:
@@ -125,6 +133,13 @@ class ClampedMoE(FeedForward):
             out[prefix + names["up"]] = TensorSpec((width, hidden_size))
             out[prefix + names["down"]] = TensorSpec((hidden_size, width))
         return out
+
+    @staticmethod
+    def _group_score(params) -> str:
+        kind = params.get("group_score", "two_best")
+        if kind not in ("two_best", "best"):
+            raise ops.KernelError(f"mixture of experts: group_score {kind!r} must be two_best or best")
+        return kind
 
     def _grouped(self, x):
         """Rows grouped by expert (see the class)."""
@@ -160,11 +175,12 @@ class ClampedMoE(FeedForward):
             logits = ops.gemm_bf16_skinny(x, self.router)     # float32 partial sums, added up by the routing kernel
         else:
             logits = linear(x, self.router, out_dtype=torch.float32)
-        if self.sigmoid_scores:
-            return ops.moe_route_sigmoid(logits, self.correction, self.experts, self.top, self.group_count,
-                                         self.group_keep, self.router_scale, shared_gate=self.shared_ff > 0, chosen=chosen)
+        if self.in_groups:
+            return ops.moe_route_groups(logits, self.correction, self.experts, self.top, self.group_count, self.group_keep,
+                                        self.router_scale, shared_gate=self.shared_gated, chosen=chosen,
+                                        softmax=not self.sigmoid_scores, group_best=self.group_best, normalise=self.sigmoid_scores)
         return ops.moe_route(logits, self.correction, self.outputs, self.identity, self.top,
-                             shared_gate=self.shared_ff > 0, chosen=chosen, logit_bias=self.router_bias,
+                             shared_gate=self.shared_gated, chosen=chosen, logit_bias=self.router_bias,
                              over_chosen=self.over_chosen)
 
     def forward(self, x):

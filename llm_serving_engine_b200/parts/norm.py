@@ -1,4 +1,4 @@
-"""RMSNorm fused with the residual sum (reference ``src/llmserve/model.py:14-23``)."""
+"""Norms fused with the residual sum (RMSNorm: reference ``src/llmserve/model.py:14-23``)."""
 from __future__ import annotations
 
 import torch
@@ -151,3 +151,54 @@ class DynamicTanh(Norm):
         if rows is None:
             stream.delta = stream.delta_norm = None
         return out
+
+
+@register_norm("layernorm")
+class LayerNorm(Norm):
+    """params: ``eps``, ``weight_name`` (default "weight"), ``bias_name`` (default: the weight's name + ".b").
+
+    y = (x - mean) / sqrt(variance + eps) * w + b over a row, in float32, the variance being the mean of the squared
+    deviations.  As a layer's norm before a branch (``forward``) x is the residual after the pending output has been added.
+    ``add_branch`` is the other use, for a layer that norms what a branch puts out: residual += norm(pending output)."""
+
+    graph_safe = True
+    kernel_sources = ("layer_norm",)
+
+    def __init__(self, params, weights, ctx) -> None:
+        super().__init__(params, weights, ctx)
+        weight, bias = self._names(params)
+        self.eps = float(params["eps"])
+        self.weight = weights[weight].to(torch.float32).contiguous()
+        self.bias = weights[bias].to(torch.float32).contiguous()
+
+    @staticmethod
+    def _names(params) -> tuple[str, str]:
+        weight = params.get("weight_name", "weight")
+        return weight, params.get("bias_name", weight + ".b")
+
+    @classmethod
+    def expected_tensors(cls, params, hidden_size):
+        weight, bias = cls._names(params)
+        return {weight: TensorSpec((hidden_size,), "norm"), bias: TensorSpec((hidden_size,), "bias")}
+
+    @staticmethod
+    def _check(stream: ResidualStream) -> None:
+        if not stream.plain or stream.delta_norm is not None or stream.delta_row_scale is not None:
+            raise ops.KernelError("layernorm: one copy of the residual, branch outputs without a norm or factors of their own")
+
+    def forward(self, stream: ResidualStream, rows: torch.Tensor | None = None) -> torch.Tensor:
+        self._check(stream)
+        n_rows = stream.residual.shape[0] if rows is None else rows.shape[0]
+        out = torch.empty((n_rows, self.weight.shape[0]), dtype=self.ctx.dtype, device=stream.residual.device)
+        ops.layer_norm(stream.residual, stream.delta, stream.delta_bias, self.weight, self.bias, self.eps, out, rows=rows)
+        if rows is None:
+            stream.delta = stream.delta_bias = None
+        return out
+
+    def add_branch(self, stream: ResidualStream) -> torch.Tensor:
+        """residual += norm(pending output); the new rows, in ``stream.hidden`` (the compute dtype)."""
+        self._check(stream)
+        copy = stream.hidden if stream.hidden is not stream.residual else None
+        ops.layer_norm(stream.residual, stream.delta, stream.delta_bias, self.weight, self.bias, self.eps, copy, after=True)
+        stream.delta = stream.delta_bias = None
+        return stream.hidden

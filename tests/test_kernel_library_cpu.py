@@ -1,6 +1,7 @@
 """Which CUDA sources a model has compiled: every entry point belongs to one source, a source's key follows the headers it
 includes, and a model names the sources of its parts and no others."""
 import ctypes
+import re
 
 import pytest
 import torch
@@ -16,6 +17,25 @@ def test_every_declared_entry_point_belongs_to_one_source():
             assert name not in owners, f"{name} in {path.stem} and {owners[name]}"
             owners[name] = path.stem
     assert set(library._SIGNATURES) <= set(owners)
+
+
+def test_declared_argument_types_are_those_of_the_sources():
+    kinds = {"int": ctypes.c_int, "long long": ctypes.c_longlong, "float": ctypes.c_float, "unsigned": ctypes.c_uint,
+             "unsigned int": ctypes.c_uint, "cudaStream_t": ctypes.c_void_p}
+    checked = set()
+    for path in build.sources():
+        for name, arguments in re.findall(r'extern "C" int\s+(lse_\w+)\s*\(([^)]*)\)', path.read_text()):
+            if name not in library._SIGNATURES:
+                continue
+            want = []
+            for argument in re.sub(r"//[^\n]*", "", arguments).split(","):
+                words = argument.split()
+                if not words or words == ["void"]:
+                    continue
+                want.append(ctypes.c_void_p if "*" in argument else kinds[" ".join(words[:-1])])
+            assert library._SIGNATURES[name] == want, name
+            checked.add(name)
+    assert checked == set(library._SIGNATURES)
 
 
 def test_a_sources_key_follows_what_it_includes(tmp_path, monkeypatch):

@@ -749,7 +749,7 @@ def test_router_chooses_within_the_best_groups(experts, top, count, keep):
         router["groups"] = {"count": count, "keep": keep}
     chosen_want, weights_want = plain.route(logits[:, :experts].double(), w, "p.", router)
     chosen = torch.empty(rows, top, dtype=torch.int32, device="cuda")
-    weights, _, gate = ops.moe_route_sigmoid(logits.cuda(), correction.cuda(), experts, top, count, keep, scale,
+    weights, _, gate = ops.moe_route_groups(logits.cuda(), correction.cuda(), experts, top, count, keep, scale,
                                              shared_gate=True, chosen=chosen)
     assert torch.equal(chosen.cpu().long().sort(dim=1).values, chosen_want.sort(dim=1).values)
     want = torch.zeros(rows, experts, dtype=torch.float64).scatter(1, chosen_want, weights_want)
