@@ -138,6 +138,23 @@ def route(logits: torch.Tensor, top: int, groups: dict | None, scale: float) -> 
     return torch.zeros_like(scores).scatter_(1, chosen, scores.gather(1, chosen)) * scale
 
 
+def routing_margin(logits: torch.Tensor, top: int, groups: dict | None) -> torch.Tensor:
+    """[T]: how far (in logits) a token's choice of experts is from another one: the smaller of the gaps between the last
+    kept group's best expert and the first dropped one's, and between the last chosen expert and the next it could have been."""
+    far = torch.full((logits.shape[0],), float("inf"), dtype=logits.dtype)
+    allowed = logits
+    if groups and int(groups["keep"]) < int(groups["count"]):
+        count, keep = int(groups["count"]), int(groups["keep"])
+        best = logits.view(logits.shape[0], count, -1)
+        order = best.amax(-1).sort(dim=-1, descending=True)
+        far = torch.minimum(far, order.values[:, keep - 1] - order.values[:, keep])
+        allowed = best.gather(1, order.indices[:, :keep, None].expand(-1, -1, best.shape[2])).flatten(1)
+    if top < allowed.shape[1]:
+        ranked = allowed.sort(dim=-1, descending=True).values
+        far = torch.minimum(far, ranked[:, top - 1] - ranked[:, top])
+    return far
+
+
 def mixture(x, w, prefix, mlp) -> torch.Tensor:
     router = mlp["router"]
     weights = route(x @ w[prefix + "router"].t(), int(router["top"]), router.get("groups"), float(router.get("scale", 1.0)))
@@ -148,8 +165,9 @@ def mixture(x, w, prefix, mlp) -> torch.Tensor:
 
 
 # --------------------------------------------------------------------------- the model
-def forward_layers(cfg: dict, w: dict, tokens: list[int]) -> list[torch.Tensor]:
-    """The residual after the embedding and after every layer: a list of [T, W]."""
+def forward_layers(cfg: dict, w: dict, tokens: list[int], margins: list | None = None) -> list[torch.Tensor]:
+    """The residual after the embedding and after every layer: a list of [T, W].  ``margins``: every mixture adds its tokens'
+    routing margins to it."""
     eps = float(cfg["norm"]["eps"])
     x = w["embed"][torch.tensor(tokens, dtype=torch.long)]
     seen, first_values = [x], None
@@ -165,6 +183,9 @@ def forward_layers(cfg: dict, w: dict, tokens: list[int]) -> list[torch.Tensor]:
             raise ValueError(f"layer {index}: unknown type {layer['type']!r}")
         x = x + layer_norm(y, w[p + "norm1"], w[p + "norm1.b"], eps)
         if layer.get("mlp") is not None:
+            if margins is not None:
+                router = layer["mlp"]["router"]
+                margins.append(routing_margin(x @ w[p + "mlp.router"].t(), int(router["top"]), router.get("groups")))
             x = x + layer_norm(mixture(x, w, p + "mlp.", layer["mlp"]), w[p + "norm2"], w[p + "norm2.b"], eps)
         seen.append(x)
     return seen
@@ -230,14 +251,15 @@ def tensor_shapes(cfg: dict) -> dict[str, tuple]:
 
 
 def random_weights(cfg: dict, seed: int) -> dict[str, torch.Tensor]:
-    """Random weights, rounded to bfloat16 values: large enough that every mechanism moves the logits."""
+    """Random weights, rounded to bfloat16 values: large enough that every mechanism moves the logits, the branches' norms small
+    enough that a branch whose output is small (and is blown up by its norm) does not drown the residual in rounding."""
     generator = torch.Generator().manual_seed(seed)
     out = {}
     for name, (shape, kind) in tensor_shapes(cfg).items():
         draw = torch.randn(shape, generator=generator)
         uniform = torch.rand(shape, generator=generator) - 0.5
-        out[name] = {"matrix": lambda: draw / math.sqrt(shape[-1]), "embed": lambda: draw, "norm": lambda: 0.8 + 0.4 * uniform,
-                     "bias": lambda: 0.2 * draw, "head_norm": lambda: 1.2 + 0.8 * uniform,
+        out[name] = {"matrix": lambda: draw / math.sqrt(shape[-1]), "embed": lambda: draw, "norm": lambda: 0.4 + 0.3 * uniform,
+                     "bias": lambda: 0.1 * draw, "head_norm": lambda: 1.2 + 0.8 * uniform,
                      "share": lambda: 0.5 + 0.6 * uniform}[kind]().to(torch.bfloat16)
     return out
 

@@ -417,7 +417,7 @@ def write_safetensors(path, tensors: dict[str, torch.Tensor]) -> None:
     header, blobs, offset = {}, [], 0
     for name, tensor in tensors.items():
         tensor = tensor.contiguous()
-        blob = tensor.view(torch.uint8).numpy().tobytes() if tensor.numel() else b""
+        blob = tensor.reshape(-1).view(torch.uint8).numpy().tobytes() if tensor.numel() else b""
         header[name] = {"dtype": names[tensor.dtype], "shape": list(tensor.shape), "data_offsets": [offset, offset + len(blob)]}
         blobs.append(blob)
         offset += len(blob)
