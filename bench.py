@@ -466,8 +466,6 @@ def other_points(args, peak: dict) -> tuple[dict, dict]:
 def run_ours(args) -> dict:
     import torch
 
-    import __graft_entry__
-    __graft_entry__.build()
     torch.cuda.set_device(0)
     layers = args.layers or FULL_LAYERS
     sizes = {"7b": QWEN25_7B_SIZES, "14b": QWEN25_14B_SIZES}.get(args.sizes)
@@ -593,8 +591,17 @@ KOFIPEL_SIZES = {
     "w2048": dict(width=2048, heads=16, ff=8192),
     "w4096": dict(width=4096, heads=32, ff=16384),
 }
+# Daferax at layer sizes that resemble real models of the kind: six layers, attention and latent attention in turn; attention
+# heads of 128 in groups of eight, the whole head rotated; latent heads of 128 + 64 rotated over a latent of 512 and a window
+# of 512 keys; mixtures of eight experts in four groups (two kept) of a third of the dense size of which a token uses two,
+# beside a shared expert of a third, so that a token's feed-forward work equals the dense layer's.  The closest existing models
+# are Fororax (normed heads, a mixture with a shared expert, a norm at the end of every sublayer) and Givelix (latent attention).
+DAFERAX_SIZES = {
+    "w2048": dict(width=2048, heads=16, ff=8192),
+    "w4096": dict(width=4096, heads=32, ff=16384),
+}
 DESIGN_SIZES = {"givelix": GIVELIX_SIZES, "fororax": FORORAX_SIZES, "tufevik": TUFEVIK_SIZES, "sebudra": SEBUDRA_SIZES,
-                "kofipel": KOFIPEL_SIZES}
+                "kofipel": KOFIPEL_SIZES, "daferax": DAFERAX_SIZES}
 
 
 def fororax_config(width: int, heads: int, ff: int, vocab: int = 32768, context: int = 4096) -> dict:
@@ -655,6 +662,20 @@ def kofipel_config(width: int, heads: int, ff: int, vocab: int = 32768, context:
             "max_position_embeddings": context}
 
 
+def daferax_config(width: int, heads: int, ff: int, vocab: int = 32768, context: int = 4096) -> dict:
+    expert_ff = (ff // 3) // 64 * 64
+    mlp = {"kind": "moe", "router": {"experts": 8, "top": 2, "scale": 1.5, "groups": {"count": 4, "keep": 2}},
+           "expert": {"ff": expert_ff}, "shared": {"ff": ff - 2 * expert_ff}}
+    attention = {"heads": heads, "kv_heads": max(2, heads // 8), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "v_mix": True,
+                 "rot": {"base": 1000000.0, "dims": 128}}
+    latent = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5, "mask": {"size": 512},
+              "rot": {"base": 1000000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 2048, "fast": 16.0, "slow": 1.0}}}
+    layers = [{"type": kind, "mixer": mixer, "mlp": mlp}
+              for kind, mixer in (("attention", attention), ("latent_attention", latent)) * 3]
+    return {"architecture": "Daferax", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": 1e-6},
+            "max_position_embeddings": context}
+
+
 def kernel_times(run, repeats: int = 3) -> dict:
     """Device microseconds per kernel name (a mean over ``repeats`` calls of ``run``), from the profiler's records."""
     import torch
@@ -692,8 +713,6 @@ def run_design(args) -> dict:
     decode step, with roofline fractions of the kernels that the two designs do not share."""
     import torch
 
-    import __graft_entry__
-    __graft_entry__.build()
     torch.cuda.set_device(0)
     from llm_serving_engine_b200.cache.manager import CacheManager
     from llm_serving_engine_b200.config.runtime_config import CacheConfig
@@ -704,12 +723,13 @@ def run_design(args) -> dict:
     fma_tflops = 2 * 128 * torch.cuda.get_device_properties(0).multi_processor_count * 1.965e9 / 1e12   # float32 FMA pipe
     design = args.design
     make_config = {"givelix": givelix_config, "fororax": fororax_config, "tufevik": tufevik_config,
-                   "sebudra": sebudra_config, "kofipel": kofipel_config}[design]
+                   "sebudra": sebudra_config, "kofipel": kofipel_config, "daferax": daferax_config}[design]
     rooflines = {"givelix": design_rooflines, "fororax": fororax_rooflines, "tufevik": tufevik_rooflines,
-                 "sebudra": sebudra_rooflines, "kofipel": kofipel_rooflines}[design]
+                 "sebudra": sebudra_rooflines, "kofipel": kofipel_rooflines, "daferax": daferax_rooflines}[design]
     # designs that are set beside another model than Qwen2 as well: (label, config maker)
     beside = {"sebudra": [("tufevik_equal_size", tufevik_config)],
-              "kofipel": [("sebudra_equal_size", sebudra_config)]}.get(design, [])
+              "kofipel": [("sebudra_equal_size", sebudra_config)],
+              "daferax": [("fororax_equal_size", fororax_config), ("givelix_equal_size", lambda **shape: givelix_config(**shape, q_rank=shape["width"] * 3 // 4))]}.get(design, [])
     batch, out = args.batch, {"design": design, "peaks": dict(peak, fp32_fma_tflops=round(fma_tflops, 1)), "sizes": {}}
     names = [args.design_size] if args.design_size else list(DESIGN_SIZES[design])
     with ClockSampler() as clocks:
@@ -1118,6 +1138,84 @@ def kofipel_rooflines(shape: dict, entry: dict, batch: int, peak: dict, fma_tflo
     return out
 
 
+def daferax_rooflines(shape: dict, entry: dict, batch: int, peak: dict, fma_tflops: float) -> dict:
+    """As :func:`design_rooflines`, for Daferax beside Fororax and Givelix (the closest existing models) at equal size: every
+    kind of kernel that is not a plain product, each against the slower of the bytes it must move and the operations it must
+    do (row-wise kernels against the bytes, attention against the measured bfloat16 tensor throughput).  The other models'
+    entries are their own tables', and those of their kernels that are the like of one here."""
+    heads, width, tokens = shape["heads"], shape["width"], PROMPT
+    kv_heads = max(2, heads // 8)
+    config = daferax_config(**shape)
+    latent, mlp = config["layers"][1]["mixer"], config["layers"][0]["mlp"]
+    rank, rot, dim, vdim, window = latent["kv_rank"], latent["rot_dim"], latent["dim"], latent["vdim"], latent["mask"]["size"]
+    experts, top, expert_ff, shared_ff = mlp["router"]["experts"], mlp["router"]["top"], mlp["expert"]["ff"], mlp["shared"]["ff"]
+    bandwidth, tensor, fma = peak["hbm_gbs"] * 1e9, peak["bf16_tflops"] * 1e12, fma_tflops * 1e12
+
+    def frac(kernels: dict, keys, launches_of_work: float, bytes_each: float, flops_each: float, pipe: float, without=()):
+        keys = (keys,) if isinstance(keys, str) else keys
+        found = [(name, value) for name, value in kernels.items()
+                 if any(key in name for key in keys) and not any(key in name for key in without)]
+        if not found:
+            return None
+        us = sum(value["us"] for _, value in found)
+        count = sum(value["launches"] for _, value in found)
+        bound = max(bytes_each / bandwidth, flops_each / pipe) * launches_of_work
+        return {"us": round(us, 1), "launches": count, "bound_us": round(bound * 1e6, 2), "frac": round(bound * 1e6 / us, 4)}
+
+    pairs = tokens * (tokens + 1) / 2
+    windowed = tokens * window - window * (window - 1) / 2
+    row, wide = (heads + 2 * kv_heads) * 128, rank + rot
+    layers, each = len(config["layers"]), 3
+    d, f, g = entry["daferax"], entry["fororax_equal_size"], entry["givelix_equal_size"]
+    out = {"prefill": {}, "decode": {}}
+
+    def front(rows: int, stored: int) -> float:      # queries, latent and shared part of a latent layer: read, written
+        return rows * (heads * (dim + rot) + wide) * (stored + 2)
+
+    def per_head(rows: int) -> tuple[float, float]:  # both products: matrices, operands, results; operations
+        sizes = heads * (dim + vdim) * rank
+        return sizes * 2 + rows * heads * (dim + vdim + 2 * rank) * 2, 2 * rows * sizes
+
+    prompt, step = d["prefill_kernels"], d["decode_kernels"]
+    out["prefill"]["daferax attention (tcgen05, gates in its epilogue, 3 layers)"] = frac(
+        prompt, "attn_prefill_tc", each, tokens * row * 2 * 2, 4 * pairs * heads * 128, tensor)
+    out["prefill"]["daferax latent attention over a window (3 layers)"] = frac(
+        prompt, "latent_attention", each, tokens * heads * (wide + rank) * 2, 2 * windowed * heads * (wide + rank), tensor)
+    out["prefill"]["daferax head norm, rotation, value mixing, gates, page write"] = frac(
+        prompt, "head_norm_pair", each, tokens * row * (4 + 2) + tokens * kv_heads * 128 * 4, 0, fma)
+    out["prefill"]["daferax latent queries, norm, rotation, cached row"] = frac(prompt, "latent_front", each, front(tokens, 2), 0, fma)
+    out["prefill"]["daferax gates of the latent layers' values"] = frac(prompt, "gate_heads", each, tokens * heads * vdim * 6, 0, fma)
+    out["prefill"]["daferax layer norm and sum"] = frac(prompt, "layer_norm", 2 * layers, tokens * width * (4 * 2 + 3 + 2), 0, fma)
+    out["prefill"]["daferax rows of the mixture (route, place, gather, activation, combine)"] = frac(
+        prompt, ("moe_",), layers, tokens * width * 2 * (1 + 2 * top) + tokens * (top * expert_ff + shared_ff) * 2 * 3 + tokens * width * 4 * 2, 0, fma)
+    out["decode"]["daferax attention (mma.sync, chunks + merge, 3 layers)"] = frac(
+        step, ("attention_scored",), each, batch * tokens * 2 * kv_heads * 128 * 2, 4 * batch * tokens * heads * 128, tensor)
+    out["decode"]["daferax latent attention over a window (chunks + merge, 3 layers)"] = frac(
+        step, "latent_attention", each, batch * window * wide * 2, 2 * batch * window * heads * (wide + rank), tensor)
+    out["decode"]["daferax head norm, rotation, value mixing, gates, page write"] = frac(
+        step, "head_norm_pair", each, batch * row * 4 * 5, 0, fma)
+    out["decode"]["daferax latent queries, norm, rotation, cached row, gates"] = frac(
+        step, "latent_front", each, front(batch, 4 * 4) + batch * heads * vdim * 4 * 5, 0, fma)
+    out["decode"]["daferax per-head products (few rows)"] = frac(step, "head_gemm", each, per_head(batch)[0], per_head(batch)[1], tensor)
+    out["decode"]["daferax layer norm and sum"] = frac(step, "layer_norm", 2 * layers, batch * width * (4 * 2 + 4 * 4 + 2), 0, fma)
+    out["decode"]["daferax rows of the mixture (route, activation)"] = frac(
+        step, ("moe_",), layers, (experts + 1) * width * 2 + batch * (experts * expert_ff + shared_ff) * 2 * 3, 0, fma)
+    qwen = {"qwen2_equal_size": entry["qwen2_equal_size"]}
+    for other in (fororax_rooflines(shape, {"fororax": f, **qwen}, batch, peak, fma_tflops),
+                  design_rooflines(shape, {"givelix": g, **qwen}, batch, peak, fma_tflops)):
+        for part in ("prefill", "decode"):
+            out[part].update({key: value for key, value in other[part].items() if value is not None and "frac" in value})
+    g_latents = 4      # Givelix's latent layers, two of them with a query latent and one without a cache of its own: counted alike
+    out["prefill"]["givelix latent queries, norms, rotation, cached row"] = frac(
+        g["prefill_kernels"], ("latent_prepare", "latent_query"), g_latents, front(tokens, 2), 0, fma)
+    out["decode"]["givelix latent queries, norms, rotation, cached row"] = frac(
+        g["decode_kernels"], ("latent_prepare", "latent_query"), g_latents, front(batch, 4 * 4), 0, fma)
+    out["decode"]["fororax head_norm_kv_write"] = frac(f["decode_kernels"], "head_norm_kv_write", 6, batch * row * 4 * 5, 0, fma)
+    for part in ("prefill", "decode"):
+        out[part] = {key: value for key, value in out[part].items() if value is not None}
+    return out
+
+
 def bench_config(config: dict, layers: int, batch: int) -> dict:
     """The ``config`` of the bench line: every size, flat; the same dict in both arms."""
     return {
@@ -1438,7 +1536,7 @@ def main() -> int:
                         help="with --only: the true float32 path instead of the serving precision")
     parser.add_argument("--quick", action="store_true", help="the headline, its points and the end-to-end number only "
                                                              "(no other model sizes, no float32 point, no kernel table)")
-    parser.add_argument("--design", choices=("givelix", "fororax", "tufevik", "sebudra", "kofipel"), default=None,
+    parser.add_argument("--design", choices=("givelix", "fororax", "tufevik", "sebudra", "kofipel", "daferax"), default=None,
                         help="instead of the default workload: the named design at layer sizes of real models beside the "
                              "Qwen2 model of equal size (prefill and decode throughput, kernel times, rooflines)")
     parser.add_argument("--design-size", choices=tuple(sorted({name for sizes in DESIGN_SIZES.values() for name in sizes})),
