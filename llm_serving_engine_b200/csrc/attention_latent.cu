@@ -205,6 +205,89 @@ latent_front_kernel(const TI* __restrict__ proj, int n_partials, long long parti
   for (int i = threadIdx.x; i < rank; i += PREP_THREADS) dst[i] = from_f32<TO>((row_s[i] * inv) * kv_norm[i]);
 }
 
+// The same over the rows of a prompt's portion (bfloat16, one set of sums, no gates; every size and offset a multiple of 8, rank
+// at most 8 * ROWS_THREADS, rot at most 256): a block per token, sines and cosines taken once, sixteen bytes a load and store.
+constexpr int ROWS_THREADS = 256;
+__device__ __forceinline__ void lat_unpack8(const uint4& raw, float (&v)[8]) {
+  const __nv_bfloat162* two = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(two[i]); v[2 * i] = f.x; v[2 * i + 1] = f.y; }
+}
+__device__ __forceinline__ uint4 lat_pack8(const float (&v)[8]) {
+  uint4 raw;
+  __nv_bfloat162* two = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) two[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+  return raw;
+}
+__device__ __forceinline__ uint4 lat_turn8(const uint4& raw, const float* cs, const float* sn) {   // four pairs from the table
+  float v[8], y[8];
+  lat_unpack8(raw, v);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    y[2 * i] = v[2 * i] * cs[i] - v[2 * i + 1] * sn[i];
+    y[2 * i + 1] = v[2 * i + 1] * cs[i] + v[2 * i] * sn[i];
+  }
+  return lat_pack8(y);
+}
+
+__global__ void __launch_bounds__(ROWS_THREADS)
+latent_front_rows_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int q_off, int heads, int dim, int rot, int rot_dims,
+                         const double* __restrict__ freq, float rot_factor, int kv_off, int rank, const float* __restrict__ kv_norm,
+                         float eps, const int* __restrict__ positions, const int* __restrict__ slot_mapping,
+                         __nv_bfloat16* __restrict__ q_plain, __nv_bfloat16* __restrict__ q_wide, int wide,
+                         __nv_bfloat16* __restrict__ cache, int num_slots) {
+  __shared__ float scratch[32], cs_s[128], sn_s[128];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  const int slot = LSE_CHECKED(slot_mapping[t], -1, num_slots, -1, LSE_CHECK_CACHE_SLOT);
+  if (slot < 0) return;
+  const uint4* row = reinterpret_cast<const uint4*>(proj + (size_t)t * ld);
+  uint4 latent = make_uint4(0, 0, 0, 0);       // this thread's eight values of the latent
+  const bool holds = (int)threadIdx.x * 8 < rank;
+  if (holds) latent = row[kv_off / 8 + threadIdx.x];
+  const int position = positions[t];
+  for (int i = threadIdx.x; i < rot / 2; i += ROWS_THREADS) {
+    float sn = 0.f, cs = 1.f;
+    if (2 * i + 1 < rot_dims) rotary_sincos(position, freq[i], rot_factor, sn, cs);
+    sn_s[i] = sn;
+    cs_s[i] = cs;
+  }
+  float v[8];
+  lat_unpack8(latent, v);
+  float sq = 0.f;
+#pragma unroll
+  for (int e = 0; e < 8; ++e) sq = fmaf(v[e], v[e], sq);
+  const float inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)rank + eps);     // its barriers publish the table too
+  uint4* held = reinterpret_cast<uint4*>(cache + (size_t)slot * (rank + rot));
+  if (holds) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] = (v[e] * inv) * kv_norm[threadIdx.x * 8 + e];
+    held[threadIdx.x] = lat_pack8(v);
+  }
+  for (int i = threadIdx.x; i < rot / 8; i += ROWS_THREADS)
+    held[rank / 8 + i] = lat_turn8(row[(kv_off + rank) / 8 + i], cs_s + 4 * i, sn_s + 4 * i);
+  const int plain8 = dim / 8, pieces = (dim + rot) / 8, total = heads * pieces;
+  uint4* plain = reinterpret_cast<uint4*>(q_plain + (size_t)t * heads * dim);
+  uint4* turned = reinterpret_cast<uint4*>(q_wide + (size_t)t * heads * wide + rank);
+  const uint4* queries = row + q_off / 8;
+  for (int base = threadIdx.x; base < total; base += 4 * ROWS_THREADS) {      // four loads in flight
+    uint4 raw[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      if (base + k * ROWS_THREADS < total) raw[k] = queries[base + k * ROWS_THREADS];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int at = base + k * ROWS_THREADS;
+      if (at >= total) continue;
+      const int h = at / pieces, c = at % pieces;
+      if (c < plain8) plain[h * plain8 + c] = raw[k];
+      else turned[(size_t)h * (wide / 8) + c - plain8] = lat_turn8(raw[k], cs_s + 4 * (c - plain8), sn_s + 4 * (c - plain8));
+    }
+  }
+}
+
 // ------------------------------------------------------------------ the attention
 constexpr int KT = 32;        // keys per tile (one warp lane per key)
 constexpr int CHUNK = 256;    // keys per chunk (a multiple of KT)
@@ -392,7 +475,7 @@ __global__ void __launch_bounds__(256)
 latent_attention_merge_kernel(const float* __restrict__ partials, T* __restrict__ out,
                               const int* __restrict__ segment_of_token, const int* __restrict__ positions,
                               const float* __restrict__ sink, int n_q, int DV, int window, int max_chunks,
-                              int num_segments) {
+                              int num_segments, int chunk_keys) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, head = blockIdx.y;
@@ -403,8 +486,8 @@ latent_attention_merge_kernel(const float* __restrict__ partials, T* __restrict_
   const float* src = partials + ((size_t)t * n_q + head) * max_chunks * (DV + 2);
   for (int d = threadIdx.x; d < DV; d += blockDim.x) {
     float total = 0.f, M = -INFINITY, L = 0.f;
-    for (int chunk = kv_begin / CHUNK; chunk <= pos / CHUNK; ++chunk) {
-      const float* part = src + (size_t)(chunk - kv_begin / CHUNK) * (DV + 2);
+    for (int chunk = kv_begin / chunk_keys; chunk <= pos / chunk_keys; ++chunk) {
+      const float* part = src + (size_t)(chunk - kv_begin / chunk_keys) * (DV + 2);
       float wa, wb;
       merge_chunk(M, L, part[DV], part[DV + 1], wa, wb);
       total = fmaf(part[d], wb, total * wa);
@@ -472,6 +555,15 @@ extern "C" int lse_latent_front(const void* proj, int in_dtype, int n_partials, 
                                 float* gate, int tokens, int num_slots, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (rot_dims > rot || (rot_dims & 1) || heads <= 0 || rank <= 0 || dim < 0 || wide < rank + rot || n_partials < 1 || !kv_norm) return LSE_ERR_BAD_ARGUMENT;
+  const bool rows_kernel = tokens >= 256 && in_dtype == LSE_DTYPE_BF16 && out_dtype == LSE_DTYPE_BF16 && n_partials == 1 && !gate &&
+                           (dim | rot | rank | wide | q_off | kv_off) % 8 == 0 && ld % 8 == 0 && rank <= 8 * ROWS_THREADS && rot <= 256 &&
+                           (((uintptr_t)proj | (uintptr_t)q_plain | (uintptr_t)q_wide | (uintptr_t)cache) & 15) == 0;
+  if (rows_kernel) {
+    lse_launch(latent_front_rows_kernel, tokens, ROWS_THREADS, 0, stream, (const __nv_bfloat16*)proj, ld, q_off, heads, dim, rot,
+               rot_dims, freq, rot_factor, kv_off, rank, kv_norm, eps, positions, slot_mapping, (__nv_bfloat16*)q_plain,
+               (__nv_bfloat16*)q_wide, wide, (__nv_bfloat16*)cache, num_slots);
+    LSE_LAUNCH_CHECK();
+  }
   const long long parts = (long long)heads + 1 + (gate ? (gates + GATES_A_BLOCK - 1) / GATES_A_BLOCK : 0);
   const size_t smem = (size_t)rank * sizeof(float);
   if (parts > 65535 || smem > 40 * 1024) return LSE_ERR_TOO_LARGE;
@@ -494,17 +586,18 @@ extern "C" int lse_latent_attention_chunk(void) { return CHUNK; }
 // The merge alone: adds up the chunks that a split kernel (this file's, or the tensor-core one) left in `partials`.
 extern "C" int lse_latent_attention_merge(const float* partials, void* out, int dtype, const int* segment_of_token,
                                           const int* positions, const float* sink, int tokens, int n_q, int DV,
-                                          int window, int max_chunks, int num_segments, cudaStream_t stream) {
+                                          int window, int max_chunks, int num_segments, int chunk_keys,
+                                          cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (n_q <= 0 || n_q > 65535 || DV <= 0 || max_chunks <= 0) return LSE_ERR_BAD_ARGUMENT;
+  if (n_q <= 0 || n_q > 65535 || DV <= 0 || max_chunks <= 0 || chunk_keys <= 0) return LSE_ERR_BAD_ARGUMENT;
   const dim3 grid(tokens, n_q);
   const int threads = min(256, ((DV + 31) / 32) * 32);
   if (dtype == LSE_DTYPE_F32)
     lse_launch(latent_attention_merge_kernel<float>, grid, threads, 0, stream, partials, (float*)out, segment_of_token,
-               positions, sink, n_q, DV, window, max_chunks, num_segments);
+               positions, sink, n_q, DV, window, max_chunks, num_segments, chunk_keys);
   else if (dtype == LSE_DTYPE_BF16)
     lse_launch(latent_attention_merge_kernel<__nv_bfloat16>, grid, threads, 0, stream, partials, (__nv_bfloat16*)out,
-               segment_of_token, positions, sink, n_q, DV, window, max_chunks, num_segments);
+               segment_of_token, positions, sink, n_q, DV, window, max_chunks, num_segments, chunk_keys);
   else return LSE_ERR_BAD_ARGUMENT;
   LSE_LAUNCH_CHECK();
 }
@@ -546,7 +639,7 @@ extern "C" int lse_latent_attention(const void* q, const void* cache, void* out,
   if (split) {                                                                                                     \
     LSE_LAT_ONE(T, DPT, true)                                                                                      \
     lse_launch(latent_attention_merge_kernel<T>, merge_grid, merge_threads, 0, stream, (const float*)partials,     \
-               (T*)out, segment_of_token, positions, sink, n_q, DV, window, max_chunks, num_segments);             \
+               (T*)out, segment_of_token, positions, sink, n_q, DV, window, max_chunks, num_segments, (int)CHUNK); \
   } else LSE_LAT_ONE(T, DPT, false)
 #define LSE_LAT_DPT(T)                                    \
   if (DV <= THREADS) { LSE_LAT_CASE(T, 1) }               \

@@ -9,7 +9,7 @@
 //   softmax  per row over the tile, float32: running maximum m and sum l, the factor exp(m_old - m_new)
 //   output   O[32][DV] = O * factor + P[32][64] V[64][DV]     warp w owns DV / 8 columns; P rounded to bfloat16 for
 //            the product, V the first DV columns of the very rows that were the keys
-// With few rows (decoding) every chunk of 256 keys has a block of its own (blockIdx.z) that leaves O, m and l of
+// With few rows (decoding) every chunk of chunk_keys keys (a multiple of 64) has a block of its own (blockIdx.z) that leaves O, m and l of
 // its chunk in the layout of attention_latent.cu's split kernel, whose merge kernel adds the chunks up and lets
 // the sink join the denominator.  window > 0: a row reads its last `window` keys only; a row's chunks are then numbered from
 // the one that holds the first key of its window, and the grid has as many as a tile's window can touch.  With many rows a block walks all its keys and finishes the row itself.
@@ -18,7 +18,7 @@
 LSE_CHECK_DEFINE(lse_check_attention_latent_mma)
 
 namespace {
-constexpr int ROWS = 32, KEYS = 64, THREADS = 256, CHUNK = 256;
+constexpr int ROWS = 32, KEYS = 64, THREADS = 256;
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool pred) {
@@ -69,7 +69,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
                             const int* __restrict__ segment_start, const int* __restrict__ segment_first_position,
                             const float* __restrict__ sink, int num_segments, int n_q, int DK, int DV, int page_size,
                             float scale, int num_pages, float* __restrict__ partials, int max_chunks,
-                            int tokens_per_tile, int heads_per_block, int window) {
+                            int tokens_per_tile, int heads_per_block, int window, int chunk_keys) {
   extern __shared__ __align__(16) unsigned char smem[];
   __shared__ int tile_slot[3];
   pdl_launch_dependents();
@@ -98,11 +98,11 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   const int heads_here = min(heads_per_block, n_q - h0);
   // window > 0: the first key that any row of the tile reads; keys before it are not fetched (their pages may be given back)
   int key_lo = window > 0 ? max(0, first_pos + 1 - window) : 0, key_hi = ctx;
-  const int chunk = key_lo / CHUNK + blockIdx.z;                  // split: the tile's chunks from its first one on
+  const int chunk = key_lo / chunk_keys + blockIdx.z;                  // split: the tile's chunks from its first one on
   if (split) {
-    key_lo = max(key_lo, chunk * CHUNK);
-    key_hi = min(ctx, (chunk + 1) * CHUNK);
-    if (chunk * CHUNK >= ctx) return;
+    key_lo = max(key_lo, chunk * chunk_keys);
+    key_hi = min(ctx, (chunk + 1) * chunk_keys);
+    if (chunk * chunk_keys >= ctx) return;
   }
   const int* bt = block_tables + (size_t)seg * bt_stride;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -262,8 +262,8 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
       if (split) {
         const int row_first = window > 0 ? max(0, pos_s[r] + 1 - window) : 0;
         // the row sees no key of this chunk: the merge does not read it
-        if (pos_s[r] < key_lo || (chunk + 1) * CHUNK <= row_first) continue;
-        float* dst = partials + (row * max_chunks + chunk - row_first / CHUNK) * (DV + 2);   // a row's chunks from its own first one
+        if (pos_s[r] < key_lo || (chunk + 1) * chunk_keys <= row_first) continue;
+        float* dst = partials + (row * max_chunks + chunk - row_first / chunk_keys) * (DV + 2);   // a row's chunks from its own first one
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt) {
           const int c = col_base + nt * 8 + (lane & 3) * 2;
@@ -299,21 +299,21 @@ extern "C" int lse_latent_attention_mma_supported(int DK, int DV) {
 }
 
 // The arguments of lse_latent_attention, with the step's segments instead of its rows' segment numbers.  partials
-// (tokens * n_q * max_chunks * (DV + 2) floats): a block per chunk of 256 keys; the caller then runs the merge of
+// (tokens * n_q * max_chunks * (DV + 2) floats): a block per chunk of chunk_keys keys; the caller then runs the merge of
 // lse_latent_attention_merge.
 extern "C" int lse_latent_attention_mma(const void* q, const void* cache, void* out, const int* block_tables,
                                         int bt_stride, const int* segment_start, const int* segment_first_position,
                                         const float* sink, int tokens, int num_segments, int n_q, int DK, int DV,
                                         int page_size, float scale, int window, int num_pages, float* partials,
-                                        int max_chunks, cudaStream_t stream) {
+                                        int max_chunks, int chunk_keys, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (!lse_latent_attention_mma_supported(DK, DV) || n_q <= 0 || page_size <= 0 || num_segments <= 0) return LSE_ERR_BAD_ARGUMENT;
   const int heads_per_block = min(n_q, ROWS);
   const int tokens_per_tile = max(1, ROWS / heads_per_block);
   const int tiles = min(tokens, tokens / tokens_per_tile + num_segments);       // an upper bound
   const bool split = partials != nullptr;
-  if (split && (max_chunks <= 0 || max_chunks > 65535 ||
-                ((long long)max_chunks * CHUNK < (long long)bt_stride * page_size && (window <= 0 || max_chunks < (window + ROWS - 2) / CHUNK + 2))))
+  if (split && (max_chunks <= 0 || max_chunks > 65535 || chunk_keys <= 0 || chunk_keys % KEYS ||
+                ((long long)max_chunks * chunk_keys < (long long)bt_stride * page_size && (window <= 0 || max_chunks < (window + ROWS - 2) / chunk_keys + 2))))
     return LSE_ERR_BAD_ARGUMENT;
   dim3 grid(tiles, (n_q + heads_per_block - 1) / heads_per_block, split ? max_chunks : 1);
   const size_t smem = Layout(DK).total;
@@ -330,7 +330,7 @@ extern "C" int lse_latent_attention_mma(const void* q, const void* cache, void* 
     lse_launch(latent_attention_mma_kernel<NT>, grid, THREADS, smem, stream, (const __nv_bfloat16*)q,              \
                (const __nv_bfloat16*)cache, (__nv_bfloat16*)out, block_tables, bt_stride, segment_start,           \
                segment_first_position, sink, num_segments, n_q, DK, DV, page_size, scale, num_pages, partials,     \
-               max_chunks, tokens_per_tile, heads_per_block, window);                                                      \
+               max_chunks, tokens_per_tile, heads_per_block, window, chunk_keys);                                                      \
   }
   if (per_warp <= 1) LSE_LMMA_CASE(1)
   else if (per_warp <= 2) LSE_LMMA_CASE(2)

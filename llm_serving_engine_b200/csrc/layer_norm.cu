@@ -186,8 +186,8 @@ extern "C" int lse_layer_norm(float* residual, const void* delta, int delta_dtyp
       (rows && write_residual) || (!after && !out))
     return LSE_ERR_BAD_ARGUMENT;
   const NormArgs args = {residual, n_partials, partial_stride, bias, weight, shift, rows, hidden, tokens, after, write_residual, eps};
-  // rows of many tokens: fewer threads a row, more rows an SM; float32 keeps one block size, hence one order of sums
-  const int threads = (out_dtype == LSE_DTYPE_BF16 && n_rows > 256 && hidden <= 128 * 4 * 8) ? 128 : 256;
+  // narrow rows of many tokens: fewer threads a row, more rows an SM; float32 keeps one block size, hence one order of sums
+  const int threads = (out_dtype == LSE_DTYPE_BF16 && n_rows > 256 && hidden <= 1024) ? 128 : 256;
   const bool aligned = (((uintptr_t)residual | (uintptr_t)delta | (uintptr_t)out | (uintptr_t)weight | (uintptr_t)shift | (uintptr_t)bias) & 15) == 0;
   const int pieces = aligned && hidden % 4 == 0 && partial_stride % 4 == 0 ? (hidden / 4 + threads - 1) / threads : 0;
 #define LSE_LN_LAUNCH(K, TD, TO) lse_launch(K, n_rows, threads, 0, stream, args, (const TD*)delta, (TO*)out)

@@ -51,10 +51,11 @@ _SIGNATURES = {
                              c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p, c_int,
                              c_void_p],
     "lse_latent_attention_merge": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                                   c_int, c_int, c_void_p],
+                                   c_int, c_int, c_int, c_void_p],
     "lse_latent_attention_mma_supported": [c_int, c_int],
     "lse_latent_attention_mma": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
-                                 c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_void_p],
+                                 c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_int,
+                                 c_void_p],
     "lse_head_gemm": [c_void_p, c_int, c_longlong, c_longlong, c_void_p, c_int, c_longlong, c_longlong, c_longlong,
                       c_void_p, c_int, c_longlong, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "lse_add_rmsnorm": [c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int,

@@ -711,6 +711,10 @@ def latent_attention_mma_supported(dk: int, dv: int, dtype: torch.dtype) -> bool
     return bool(library.load().lse_latent_attention_mma_supported(int(dk), int(dv)))
 
 
+LATENT_SMALL_CHUNK = 64               # keys of a chunk of the tensor-core kernel (a tile of keys) over a window up to
+LATENT_SMALL_CHUNK_WINDOW = 1024      # this long; 256 beyond it and without a window
+
+
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_tables: torch.Tensor,
                      segment_of_token: torch.Tensor, positions: torch.Tensor, scale: float,
                      sink: torch.Tensor | None = None, window: int = 0, split: bool | None = None,
@@ -720,7 +724,7 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, bl
     [pages, page_size, DK], out [T, heads, DV] with DV <= DK: the first DV columns of a row are its value.
     ``sink`` float32 [heads]: exp(sink_h) joins the softmax's denominator.  ``window`` > 0: a row reads its last ``window``
     rows only, itself included.  ``split``: every chunk of 256 keys of a
-    row gets a block of its own and a second kernel merges them (default: with few rows).  Given the step's
+    row (of 64 over a short window) gets a block of its own and a second kernel merges them (default: with few rows).  Given the step's
     ``segment_start`` (int32 [S + 1]) and ``segment_first_position`` (int32 [S]), bfloat16 shapes that the
     tensor-core kernel takes run there (``tensor_cores=False``: the general kernel, for comparisons)."""
     _need_cuda(q, cache, out, block_tables, segment_of_token, positions, sink, segment_start, segment_first_position)
@@ -732,15 +736,17 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, bl
     assert block_tables.dtype == torch.int32 and block_tables.dim() == 2 and block_tables.stride(1) == 1
     assert sink is None or (sink.dtype == torch.float32 and sink.shape == (heads,))
     lib = library.load()
-    partials, max_chunks = None, 0
+    on_tensor_cores = (tensor_cores and segment_start is not None and segment_first_position is not None
+                       and latent_attention_mma_supported(dk, dv, q.dtype))
+    partials, max_chunks, chunk = None, 0, int(lib.lse_latent_attention_chunk())
     if split if split is not None else tokens <= GENERIC_SPLIT_MAX_ROWS:
-        chunk = int(lib.lse_latent_attention_chunk())
+        if on_tensor_cores and 0 < window <= LATENT_SMALL_CHUNK_WINDOW:
+            chunk = LATENT_SMALL_CHUNK     # a short walk: a block per tile of keys
         max_chunks = max(1, -(-(block_tables.stride(0) * page_size) // chunk))
         if window > 0:     # chunks that the window of a tile of up to 32 rows can touch
             max_chunks = min(max_chunks, (window + 30) // chunk + 2)
         partials = torch.empty(tokens * heads * max_chunks * (dv + 2), dtype=torch.float32, device=q.device)
-    if (tensor_cores and segment_start is not None and segment_first_position is not None
-            and latent_attention_mma_supported(dk, dv, q.dtype)):
+    if on_tensor_cores:
         segments = segment_first_position.shape[0]
         assert segment_start.dtype == torch.int32 and segment_start.shape[0] == segments + 1
         assert segments == block_tables.shape[0]
@@ -748,11 +754,11 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, bl
                                            block_tables.stride(0), segment_start.data_ptr(),
                                            segment_first_position.data_ptr(), _ptr(sink), tokens, segments, heads, dk,
                                            dv, page_size, float(scale), int(window), cache.shape[0], _ptr(partials),
-                                           max_chunks, _stream()), "latent_attention_mma")
+                                           max_chunks, chunk, _stream()), "latent_attention_mma")
         if partials is not None:
             check(lib.lse_latent_attention_merge(partials.data_ptr(), out.data_ptr(), dtype_code(out.dtype),
                                                  segment_of_token.data_ptr(), positions.data_ptr(), _ptr(sink), tokens,
-                                                 heads, dv, int(window), max_chunks, block_tables.shape[0], _stream()),
+                                                 heads, dv, int(window), max_chunks, block_tables.shape[0], chunk, _stream()),
                   "latent_attention_merge")
         return out
     check(lib.lse_latent_attention(q.data_ptr(), cache.data_ptr(), out.data_ptr(), dtype_code(q.dtype),

@@ -453,29 +453,34 @@ def test_windowed_latent_attention_of_unequal_requests_in_one_launch(split):
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("stacked", [False, True])
-@pytest.mark.parametrize("heads,dim,rot,rot_dims,rank,vdim", [(3, 20, 12, 12, 36, 24), (1, 1, 2, 2, 1, 1), (5, 7, 9, 4, 27, 13), (8, 128, 64, 64, 512, 128)])
-def test_queries_latent_and_gates_in_one_launch(dtype, stacked, heads, dim, rot, rot_dims, rank, vdim):
-    """Positions in the thousands, stretched frequencies, a padding row, rows as partial sums and whole."""
+@pytest.mark.parametrize("rows", [5, 300])
+@pytest.mark.parametrize("heads,dim,rot,rot_dims,rank,vdim", [(3, 20, 12, 12, 36, 24), (1, 1, 2, 2, 1, 1), (5, 7, 9, 4, 27, 13), (8, 128, 64, 64, 512, 128),
+                                                              (3, 24, 16, 12, 40, 8)])
+def test_queries_latent_and_gates_in_one_launch(dtype, stacked, rows, heads, dim, rot, rot_dims, rank, vdim):
+    """Positions in the thousands, stretched frequencies, a padding row, rows as partial sums and whole; few rows, and the many
+    of a portion with and without the gates (which a later kernel may take)."""
     from llm_serving_engine_b200.kernels import ops
     from llm_serving_engine_b200.parts.latent_attention import rotary_frequencies
 
     torch.manual_seed(19)
-    rows, page, first = 5, 8, 4001
+    page, first = 8, 4001
     description = {"base": 3000.0, "dims": rot_dims, "scaling": {"factor": 8.0, "original": 512, "fast": 16.0, "slow": 1.0}}
     wanted, plain_factor = plain.frequencies(description)
     freq, factor = rotary_frequencies(description)
     assert abs(factor - plain_factor) < 1e-12 and float((freq - torch.tensor(wanted, dtype=torch.float64)).abs().max()) < 1e-12
     nq, gates = heads * (dim + rot), heads * vdim
     width = nq + rank + rot + gates
-    whole = torch.randn(rows, width + 3)
+    whole = torch.randn(rows, -(-width // 8) * 8)
     proj = torch.stack([whole * 0.25, whole * 0.5, whole * 0.25]) if stacked else whole.to(dtype)
     seen = (proj.double().sum(0) if stacked else proj.double())[:, :width]
-    slots = torch.tensor([3, 17, -1, 30, 8], dtype=torch.int32)
+    pages = rows // page + 4
+    slots = torch.randperm(pages * page)[:rows].to(torch.int32)
+    slots[2] = -1
     norm = torch.rand(rank) + 0.5
-    cache = torch.zeros(4, page, rank + rot, dtype=dtype, device="cuda")
+    cache = torch.zeros(pages, page, rank + rot, dtype=dtype, device="cuda")
     q_plain = torch.zeros(rows, heads, dim, dtype=dtype, device="cuda")
     q_wide = torch.zeros(rows, heads, rank + rot, dtype=dtype, device="cuda")
-    gate = torch.zeros(rows, gates, device="cuda")
+    gate = torch.zeros(rows, gates, device="cuda") if rows == 5 else None
     ops.latent_front(proj.cuda(), torch.arange(first, first + rows, dtype=torch.int32).cuda(), slots.cuda(), 1e-5, q_off=0, heads=heads,
                      dim=dim, rot=rot, rot_dims=rot_dims, freq=freq.cuda(), rot_factor=factor, kv_off=nq, rank=rank, kv_norm=norm.cuda(),
                      q_plain=q_plain, q_wide=q_wide, cache=cache, g_off=nq + rank + rot, gate=gate)
@@ -484,16 +489,18 @@ def test_queries_latent_and_gates_in_one_launch(dtype, stacked, heads, dim, rot,
     c = plain.rms(seen[:, nq:nq + rank], 1e-5) * norm.double()
     shared = plain.rotate_pairs(seen[:, None, nq + rank:nq + rank + rot], description, first)[:, 0]
     limit = 3e-5 if dtype == torch.float32 else 4e-2
-    for row, slot in enumerate(slots.tolist()):
-        if slot < 0:
-            assert float(q_plain[row].abs().max()) == 0.0
-            continue
-        held = cache[slot // page, slot % page].cpu().double()
-        for got, want in ((q_plain[row], q[row, :, :dim]), (q_wide[row, :, rank:], turned[row]), (held[:rank], c[row]), (held[rank:], shared[row])):
-            assert float((got.cpu().double() - want).abs().max()) <= limit * max(1.0, float(want.abs().max()) / 4)
-        assert float((gate[row].cpu().double() - torch.sigmoid(seen[row, nq + rank + rot:])).abs().max()) <= 2e-6
-    used = {slot for slot in slots.tolist() if slot >= 0}
-    assert all(float(cache[slot // page, slot % page].abs().max()) == 0.0 for slot in range(4 * page) if slot not in used)
+    real = slots >= 0
+    held = cache.cpu().double().view(pages * page, -1)
+    for got, want in ((q_plain.cpu(), q[..., :dim]), (q_wide.cpu()[..., rank:], turned)):
+        assert float((got.double() - want)[real].abs().max()) <= limit * max(1.0, float(want.abs().max()) / 4)
+        assert float(got[2].abs().max()) == 0.0
+    for got, want in ((held[slots[real].long()][:, :rank], c[real]), (held[slots[real].long()][:, rank:], shared[real])):
+        assert float((got - want).abs().max()) <= limit * max(1.0, float(want.abs().max()) / 4)
+    if gate is not None:
+        assert float((gate.cpu().double() - torch.sigmoid(seen[:, nq + rank + rot:]))[real].abs().max()) <= 2e-6
+    free = torch.ones(pages * page, dtype=torch.bool)
+    free[slots[real].long()] = False
+    assert float(held[free].abs().max()) == 0.0
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
