@@ -77,7 +77,7 @@ struct NormArgs {
 
 // Rows whose width is a multiple of 4 up to blockDim * 4 * C: the row stays in registers (a thread owns C float4 pieces).
 template <typename TD, typename TO, int C>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, C <= 4 ? 4 : 2)
 layer_norm_regs_kernel(NormArgs a, const TD* __restrict__ delta, TO* __restrict__ out) {
   __shared__ float scratch[32];
   pdl_launch_dependents();
