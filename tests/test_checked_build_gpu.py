@@ -1,5 +1,5 @@
 """The checked variant of the kernel library (``LSE_CHECK=1``: every index taken from a step's metadata is compared
-with its range, a bad one is replaced by a safe one and recorded).  It is a library of its own and is chosen when the
+with its range, a bad one is replaced by a safe one and recorded).  It is a set of libraries of its own and is chosen when the
 library is first loaded, so the checks run in a child process: a replay of mixed traces must record nothing and
 give the logits of the plain implementation; then a block table is damaged on the host (an entry of -1 inside the
 context, which the ordinary library would turn into an address) and the record must name it, with no fault."""
